@@ -3,13 +3,15 @@
 // softmax + .v + head merge, without the [b, h, t, T] score tensor).
 //
 //   persistent grid of at most 2 x SMs CTAs over the (query tile, head, sequence) work items, 192 threads,
-//   two CTAs per SM (80 KiB of shared memory and 256 TMEM columns each: while one CTA's softmax warps work,
-//   the other's products run):
-//     warp 0      TMA producer: draws the work item, loads its 128 x 64 query tile, then 64-key K and V tiles
+//   two CTAs per SM for 64-wide heads (80 KiB of shared memory and 256 TMEM columns each: while one CTA's softmax
+//   warps work, the other's products run), one for wider ones.  DQ, the width of queries and keys, and DV, that of
+//   values, are template parameters (multiples of 64; a tile is DQ / 64 or DV / 64 blocks of one 128-byte swizzle
+//   row per query or key):
+//     warp 0      TMA producer: draws the work item, loads its 128 x DQ query tile, then 64-key K and V tiles
 //                               into two-deep rings
-//     warp 1      MMA issuer:   S = Q K^T  (tcgen05.mma M128 N64 K16 x 4, both operands K-major) into one of two
-//                               TMEM score buffers; O_j = P V (M128 N64 K16 x 4, V consumed MN-major as it lies
-//                               in the cache) into one of two TMEM output buffers
+//     warp 1      MMA issuer:   S = Q K^T  (tcgen05.mma M128 N64 K16 x DQ / 16, both operands K-major) into one of
+//                               two TMEM score buffers; O_j = P V (M128 N = DV K16 x 4, V consumed MN-major as it
+//                               lies in the cache) into one of two TMEM output buffers
 //     warps 2..5  softmax:      one query row per thread (= one TMEM lane): scale, causal mask, running max and
 //                               sum without any shuffle, P rounded to bf16 into swizzled shared memory for the
 //                               second product; the rescaled sum of the O_j lives in registers
@@ -25,19 +27,28 @@ namespace {
 
 using namespace ugb_tc;
 
-constexpr int BQ = 128, BKV = 64, HD = 64;
+constexpr int BQ = 128, BKV = 64, CB = 64;    // queries and keys per tile, columns per block (one swizzle row)
 constexpr int THREADS = 192;
-constexpr int Q_BYTES = BQ * HD * 2;          // 16 KiB
-constexpr int KV_BYTES = BKV * HD * 2;        // 8 KiB per K or V tile
 constexpr int P_BYTES = BQ * BKV * 2;         // 16 KiB: 128 rows x 128 B (64 keys)
-constexpr int SMEM_BYTES = Q_BYTES + 4 * KV_BYTES + 2 * P_BYTES + 1024 /*alignment*/ + 256 /*barriers*/;
-constexpr int TMEM_COLS = 256;                // S: 2 x 64 columns, O: 2 x 64 columns
-constexpr int O_COL = 128;
-static_assert(BKV == 64 && HD == 64, "one 128-byte swizzle atom per P row and per K / V row");
+constexpr int Q_BLOCK = BQ * CB * 2;          // 16 KiB per 64 columns of the query tile
+constexpr int KV_BLOCK = BKV * CB * 2;        // 8 KiB per 64 columns of a K or V tile
+constexpr int O_COL = 128;                    // TMEM: S 2 x 64 columns, then O 2 x DV columns
+static_assert(BKV == 64, "one 128-byte swizzle atom per P row");
+template <int DQ, int DV> struct Shape {
+  static constexpr int Q_BYTES = BQ * DQ * 2, K_BYTES = BKV * DQ * 2, V_BYTES = BKV * DV * 2;
+  static constexpr int TMEM_COLS = O_COL + 2 * DV <= 256 ? 256 : 512;
+  static constexpr int CTAS_PER_SM = DQ == 64 && DV == 64 ? 2 : 1;
+  static constexpr int TILES = Q_BYTES + 2 * K_BYTES + 2 * V_BYTES + 2 * P_BYTES + 1024 /*alignment*/ + 256 /*barriers*/;
+  // a CTA that takes all 512 TMEM columns must be alone on its SM: more than half of the shared memory sees to that
+  static constexpr int SMEM_BYTES = CTAS_PER_SM == 1 && TILES < 116 * 1024 ? 116 * 1024 : TILES;
+  static_assert(DQ % CB == 0 && DV % CB == 0 && O_COL + 2 * DV <= 512 && SMEM_BYTES <= 227 * 1024, "tile shape");
+};
 
 struct Params {
   int t, pos0, n_heads, n_kv, batch;
   float scale;
+  const float *gate;   // f32 [batch * t][gate_ld]: factor per query row and head, or null
+  int gate_ld;
   __nv_bfloat16 *out;
   ugb_status_word *status;
   int *sched;   // {next item, CTAs done}: both zero between launches; null = items dealt round-robin
@@ -86,12 +97,15 @@ __device__ __forceinline__ Item item_of(int idx, const Params &p, int q_tiles) {
   return it;
 }
 
-__global__ void __launch_bounds__(THREADS, 2)
+template <int DQ, int DV>
+__global__ void __launch_bounds__(THREADS, (Shape<DQ, DV>::CTAS_PER_SM))
 prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                             const __grid_constant__ CUtensorMap tmV, Params p) {
+  using Sh = Shape<DQ, DV>;
+  constexpr int Q_BYTES = Sh::Q_BYTES, K_BYTES = Sh::K_BYTES, V_BYTES = Sh::V_BYTES, TMEM_COLS = Sh::TMEM_COLS;
   extern __shared__ uint8_t smem_raw[];
   uint8_t *smem = (uint8_t *)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
-  uint8_t *q_s = smem, *k_s = q_s + Q_BYTES, *v_s = k_s + 2 * KV_BYTES, *p_s = v_s + 2 * KV_BYTES;
+  uint8_t *q_s = smem, *k_s = q_s + Q_BYTES, *v_s = k_s + 2 * K_BYTES, *p_s = v_s + 2 * V_BYTES;
   uint64_t *bars = (uint64_t *)(p_s + 2 * P_BYTES);
   uint64_t *q_full = bars, *k_full = bars + 1, *k_empty = bars + 3, *v_full = bars + 5, *v_empty = bars + 7;
   uint64_t *s_full = bars + 9, *p_full = bars + 11, *o_full = bars + 13, *q_empty = bars + 15, *item_full = bars + 16;
@@ -147,18 +161,21 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __gri
         if (!more) break;
         const Item it = item_of(idx, p, q_tiles);
         mbar_expect_tx(smem_u32(q_full), Q_BYTES);
-        tma_load_4d(smem_u32(q_s), &tmQ, smem_u32(q_full), 0, it.head, it.q0, it.b);
+        for (int c = 0; c < DQ / CB; ++c)
+          tma_load_4d(smem_u32(q_s + c * Q_BLOCK), &tmQ, smem_u32(q_full), c * CB, it.head, it.q0, it.b);
         // the next item is drawn now, its latency hidden behind this item's tiles
         idx = p.sched ? (int)gridDim.x + atomicAdd(p.sched, 1) : idx + (int)gridDim.x;
         for (int j = 0; j < it.n_tiles; ++j, ++g) {
           const int s = g & 1;
           const uint32_t ph = (uint32_t)(g >> 1) & 1u;
           if (!mbar_wait(smem_u32(&k_empty[s]), ph ^ 1u, abort_flag, p.status, 0x41)) { alive = false; break; }
-          mbar_expect_tx(smem_u32(&k_full[s]), KV_BYTES);
-          tma_load_3d(smem_u32(k_s + s * KV_BYTES), &tmK, smem_u32(&k_full[s]), 0, j * BKV, it.b * p.n_kv + it.kvh);
+          mbar_expect_tx(smem_u32(&k_full[s]), K_BYTES);
+          for (int c = 0; c < DQ / CB; ++c)
+            tma_load_4d(smem_u32(k_s + s * K_BYTES + c * KV_BLOCK), &tmK, smem_u32(&k_full[s]), c * CB, it.kvh, j * BKV, it.b);
           if (!mbar_wait(smem_u32(&v_empty[s]), ph ^ 1u, abort_flag, p.status, 0x42)) { alive = false; break; }
-          mbar_expect_tx(smem_u32(&v_full[s]), KV_BYTES);
-          tma_load_3d(smem_u32(v_s + s * KV_BYTES), &tmV, smem_u32(&v_full[s]), 0, j * BKV, it.b * p.n_kv + it.kvh);
+          mbar_expect_tx(smem_u32(&v_full[s]), V_BYTES);
+          for (int c = 0; c < DV / CB; ++c)
+            tma_load_4d(smem_u32(v_s + s * V_BYTES + c * KV_BLOCK), &tmV, smem_u32(&v_full[s]), c * CB, it.kvh, j * BKV, it.b);
         }
       }
       if (p.sched) {
@@ -175,17 +192,17 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __gri
     // ------------------------------------------------------------------ MMA issuer --
     if (lane == 0) {
       const uint32_t idesc_s = make_idesc(BQ, BKV, false);          // Q and K both K-major (rows of 64 dims)
-      const uint32_t idesc_o = make_idesc(BQ, HD, true);            // P K-major, V MN-major ([key][dim] rows)
+      const uint32_t idesc_o = make_idesc(BQ, DV, true);            // P K-major, V MN-major ([key][dim] rows)
       bool alive = true;
       auto issue_s = [&](int g) {
         const int s = g & 1;
         if (!mbar_wait(smem_u32(&k_full[s]), (uint32_t)(g >> 1) & 1u, abort_flag, p.status, 0x44)) { alive = false; return; }
         tcgen05_fence_after();
-        const uint32_t qa = smem_u32(q_s), kb = smem_u32(k_s + s * KV_BYTES);
+        const uint32_t qa = smem_u32(q_s), kb = smem_u32(k_s + s * K_BYTES);
 #pragma unroll
-        for (int kk = 0; kk < HD / UMMA_K; ++kk)
-          umma_bf16(tmem + (uint32_t)(s * BKV), make_smem_desc(qa + kk * (UMMA_K * 2), 0, 1024),
-                    make_smem_desc(kb + kk * (UMMA_K * 2), 0, 1024), idesc_s, kk > 0 ? 1u : 0u);
+        for (int kk = 0; kk < DQ / UMMA_K; ++kk)                    // 4 steps of 16 inside a 64-column block
+          umma_bf16(tmem + (uint32_t)(s * BKV), make_smem_desc(qa + (kk / 4) * Q_BLOCK + (kk % 4) * (UMMA_K * 2), 0, 1024),
+                    make_smem_desc(kb + (kk / 4) * KV_BLOCK + (kk % 4) * (UMMA_K * 2), 0, 1024), idesc_s, kk > 0 ? 1u : 0u);
         umma_commit(smem_u32(&k_empty[s]));                         // K stage free once the products retire
         umma_commit(smem_u32(&s_full[s]));                          // scores ready for the softmax warps
       };
@@ -195,14 +212,15 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __gri
         if (!mbar_wait(smem_u32(&p_full[s]), ph, abort_flag, p.status, 0x45)) { alive = false; return; }
         if (!mbar_wait(smem_u32(&v_full[s]), ph, abort_flag, p.status, 0x46)) { alive = false; return; }
         tcgen05_fence_after();
-        const uint32_t pa = smem_u32(p_s + s * P_BYTES), vb = smem_u32(v_s + s * KV_BYTES);
+        const uint32_t pa = smem_u32(p_s + s * P_BYTES), vb = smem_u32(v_s + s * V_BYTES);
 #pragma unroll
         for (int kk = 0; kk < BKV / UMMA_K; ++kk) {
           // P: 128 rows x 128 B, a step of 16 keys moves 32 B inside the swizzled row.
-          // V: rows of 128 B per key, 8-key groups 1024 B apart; a step of 16 keys moves 16 rows.
+          // V: rows of 128 B per key, 8-key groups 1024 B apart, 64-column blocks BKV * 128 B apart; a step of
+          // 16 keys moves 16 rows.
           const uint64_t ad = make_smem_desc(pa + kk * (UMMA_K * 2), 0, 1024);
           const uint64_t bd = make_smem_desc(vb + kk * (UMMA_K * 128), BKV * 128, 1024);
-          umma_bf16(tmem + (uint32_t)(O_COL + s * HD), ad, bd, idesc_o, kk > 0 ? 1u : 0u);
+          umma_bf16(tmem + (uint32_t)(O_COL + s * DV), ad, bd, idesc_o, kk > 0 ? 1u : 0u);
         }
         umma_commit(smem_u32(&v_empty[s]));
         umma_commit(smem_u32(&o_full[s]));
@@ -247,18 +265,21 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __gri
       const int qi = it.q0 + row;
       const int reach = p.pos0 + qi;                                // last key this query attends
       float m_run = -INFINITY, l_run = 0.f, alpha_prev = 0.f;
-      float o[HD];
+      float o[DV];
 #pragma unroll
-      for (int d = 0; d < HD; ++d) o[d] = 0.f;
+      for (int d = 0; d < DV; ++d) o[d] = 0.f;
       auto fold = [&](int g, float alpha) {                         // o = o * alpha + O_g
         const int s = g & 1;
         // .aligned TMEM loads follow: the whole warp leaves together or not at all
         if (!__all_sync(0xffffffffu, mbar_wait(smem_u32(&o_full[s]), (uint32_t)(g >> 1) & 1u, abort_flag, p.status, 0x47))) { alive = false; return; }
         tcgen05_fence_after();
-        float f[HD];
-        tmem_ld64(lane_base + (uint32_t)(O_COL + s * HD), f);
 #pragma unroll
-        for (int i = 0; i < HD; ++i) o[i] = o[i] * alpha + f[i];
+        for (int c = 0; c < DV / 64; ++c) {
+          float f[64];
+          tmem_ld64(lane_base + (uint32_t)(O_COL + s * DV + c * 64), f);
+#pragma unroll
+          for (int i = 0; i < 64; ++i) o[c * 64 + i] = o[c * 64 + i] * alpha + f[i];
+        }
       };
       for (int j = 0; j < it.n_tiles && alive; ++j) {
         const int g = g0 + j, s = g & 1;
@@ -309,10 +330,11 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __gri
       }
       if (alive && it.n_tiles > 0) fold(g0 + it.n_tiles - 1, alpha_prev);
       if (alive && qi < p.t) {
-        const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
-        __nv_bfloat16 *dst = p.out + ((size_t)it.b * p.t + qi) * ((size_t)p.n_heads * HD) + (size_t)it.head * HD;
+        float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+        if (p.gate) inv *= p.gate[((size_t)it.b * p.t + qi) * p.gate_ld + it.head];
+        __nv_bfloat16 *dst = p.out + ((size_t)it.b * p.t + qi) * ((size_t)p.n_heads * DV) + (size_t)it.head * DV;
 #pragma unroll
-        for (int c = 0; c < HD / 8; ++c) {
+        for (int c = 0; c < DV / 8; ++c) {
           uint4 v;
           __nv_bfloat162 t;
           t = __floats2bfloat162_rn(o[c * 8 + 0] * inv, o[c * 8 + 1] * inv); v.x = *(uint32_t *)&t;
@@ -333,41 +355,54 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __gri
   }
 }
 
-}  // namespace
-
-int32_t ugb_prefill_attention_tc(ugb_device *dev, const __nv_bfloat16 *q, const __nv_bfloat16 *kcache,
-                                 const __nv_bfloat16 *vcache, __nv_bfloat16 *out, int batch, int t, int pos0,
-                                 int n_heads, int n_kv, int t_max, float scale, int dynamic) {
-  if (batch == 0 || t == 0) return UGB_OK;
+template <int DQ, int DV>
+int32_t launch(ugb_device *dev, const ugb_prefill_attention_args &a) {
+  using Sh = Shape<DQ, DV>;
   static bool attr_set[64] = {};
   if (!attr_set[dev->ordinal & 63]) {
-    UGB_CUDA(dev, cudaFuncSetAttribute(prefill_attention_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES));
+    UGB_CUDA(dev, cudaFuncSetAttribute(prefill_attention_tc_kernel<DQ, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, Sh::SMEM_BYTES));
     attr_set[dev->ordinal & 63] = true;
   }
   CUtensorMap tmQ, tmK, tmV;
   int32_t rc;
-  {   // q [batch, t, n_heads, 64]: dims {d, head, position, sequence}, a box is 128 positions of one head
-    const uint64_t dims[4] = {(uint64_t)HD, (uint64_t)n_heads, (uint64_t)t, (uint64_t)batch};
-    const uint64_t strides[3] = {(uint64_t)HD, (uint64_t)n_heads * HD, (uint64_t)t * n_heads * HD};
-    const uint32_t box[4] = {(uint32_t)HD, 1, (uint32_t)BQ, 1};
-    if ((rc = ugb_tc_encode_bf16(dev, &tmQ, q, 4, dims, strides, box))) return rc;
+  {   // q [batch, t, n_heads, DQ]: dims {d, head, position, sequence}, a box is 64 columns of 128 positions of one head
+    const uint64_t dims[4] = {(uint64_t)DQ, (uint64_t)a.n_heads, (uint64_t)a.t, (uint64_t)a.batch};
+    const uint64_t strides[3] = {(uint64_t)DQ, (uint64_t)a.n_heads * DQ, (uint64_t)a.t * a.n_heads * DQ};
+    const uint32_t box[4] = {(uint32_t)CB, 1, (uint32_t)BQ, 1};
+    if ((rc = ugb_tc_encode_bf16(dev, &tmQ, a.q, 4, dims, strides, box))) return rc;
   }
-  {   // caches [batch, n_kv, t_max, 64]: dims {d, position, sequence x kv head}
-    const uint64_t dims[3] = {(uint64_t)HD, (uint64_t)t_max, (uint64_t)batch * n_kv};
-    const uint64_t strides[2] = {(uint64_t)HD, (uint64_t)t_max * HD};
-    const uint32_t box[3] = {(uint32_t)HD, (uint32_t)BKV, 1};
-    if ((rc = ugb_tc_encode_bf16(dev, &tmK, kcache, 3, dims, strides, box))) return rc;
-    if ((rc = ugb_tc_encode_bf16(dev, &tmV, vcache, 3, dims, strides, box))) return rc;
-  }
+  auto kv_map = [&](CUtensorMap *m, const __nv_bfloat16 *base, int d) {   // dims {d, KV head, position, sequence}
+    const uint64_t head = a.token_major ? (uint64_t)d : (uint64_t)a.kv_rows * d;
+    const uint64_t pos = a.token_major ? (uint64_t)a.n_kv * d : (uint64_t)d;
+    const uint64_t dims[4] = {(uint64_t)d, (uint64_t)a.n_kv, (uint64_t)a.kv_rows, (uint64_t)a.batch};
+    const uint64_t strides[3] = {head, pos, (uint64_t)a.n_kv * a.kv_rows * d};
+    const uint32_t box[4] = {(uint32_t)CB, 1, (uint32_t)BKV, 1};
+    return ugb_tc_encode_bf16(dev, m, base, 4, dims, strides, box);
+  };
+  if ((rc = kv_map(&tmK, a.k, DQ)) || (rc = kv_map(&tmV, a.v, DV))) return rc;
   Params p;
-  p.t = t; p.pos0 = pos0; p.n_heads = n_heads; p.n_kv = n_kv; p.batch = batch; p.scale = scale; p.out = out;
+  p.t = a.t; p.pos0 = a.pos0; p.n_heads = a.n_heads; p.n_kv = a.n_kv; p.batch = a.batch; p.scale = a.scale; p.out = a.out;
+  p.gate = a.gate; p.gate_ld = a.gate_ld;
   p.status = dev->status_dev;
-  p.sched = dynamic ? dev->sched_dev : nullptr;
-  const long long n_items = (long long)((t + BQ - 1) / BQ) * n_heads * batch;
-  const long long slots = 2LL * dev->sm_count;                     // two CTAs per SM
+  p.sched = a.dynamic ? dev->sched_dev : nullptr;
+  const long long n_items = (long long)((a.t + BQ - 1) / BQ) * a.n_heads * a.batch;
+  const long long slots = (long long)Sh::CTAS_PER_SM * dev->sm_count;
   dim3 grid((unsigned)(n_items < slots ? n_items : slots));
-  prefill_attention_tc_kernel<<<grid, THREADS, SMEM_BYTES, dev->stream>>>(tmQ, tmK, tmV, p);
+  prefill_attention_tc_kernel<DQ, DV><<<grid, THREADS, Sh::SMEM_BYTES, dev->stream>>>(tmQ, tmK, tmV, p);
   return ugb_after_launch(dev, "prefill_attention_tc_kernel");
+}
+
+}  // namespace
+
+int ugb_prefill_attention_width(int dim) { return dim <= 64 ? 64 : (dim <= 128 ? 128 : 0); }
+
+int32_t ugb_prefill_attention_tc(ugb_device *dev, const ugb_prefill_attention_args &a) {
+  if (a.batch == 0 || a.t == 0) return UGB_OK;
+  if (a.dq == 64 && a.dv == 64) return launch<64, 64>(dev, a);
+  if (a.dq == 64 && a.dv == 128) return launch<64, 128>(dev, a);
+  if (a.dq == 128 && a.dv == 64) return launch<128, 64>(dev, a);
+  if (a.dq == 128 && a.dv == 128) return launch<128, 128>(dev, a);
+  return ugb_fail(dev, UGB_ERR_UNSUPPORTED, "prefill attention: no kernel for %d-wide keys and %d-wide values", a.dq, a.dv);
 }
 
 extern "C" int32_t ugb_causal_attention(ugb_device *dev, const ugb_slice *q, const ugb_slice *k, const ugb_slice *v,
@@ -381,15 +416,18 @@ extern "C" int32_t ugb_causal_attention(ugb_device *dev, const ugb_slice *q, con
   UGB_REQUIRE(dev, b <= 65535 && n_heads <= 65535 && t_max <= (1u << 30) && b * n_kv <= (1u << 30) &&
                        ((t + BQ - 1) / BQ) * n_heads * b <= (size_t)INT32_MAX,
               UGB_ERR_SHAPE, "causal_attention: a dimension exceeds the kernel's index range");
-  UGB_SLICE(dev, q, UGB_BF16, b * t * n_heads * HD);
-  UGB_SLICE(dev, k, UGB_BF16, b * n_kv * t_max * HD);
-  UGB_SLICE(dev, v, UGB_BF16, b * n_kv * t_max * HD);
-  UGB_SLICE(dev, out, UGB_BF16, b * t * n_heads * HD);
+  UGB_SLICE(dev, q, UGB_BF16, b * t * n_heads * 64);
+  UGB_SLICE(dev, k, UGB_BF16, b * n_kv * t_max * 64);
+  UGB_SLICE(dev, v, UGB_BF16, b * n_kv * t_max * 64);
+  UGB_SLICE(dev, out, UGB_BF16, b * t * n_heads * 64);
   if (b == 0 || t == 0) return UGB_OK;
   UGB_REQUIRE(dev, (((uintptr_t)q->ptr | (uintptr_t)k->ptr | (uintptr_t)v->ptr | (uintptr_t)out->ptr) & 15) == 0,
               UGB_ERR_UNSUPPORTED, "causal_attention: buffers must be 16-byte aligned");
   UGB_CUDA(dev, cudaSetDevice(dev->ordinal));
-  return ugb_prefill_attention_tc(dev, (const __nv_bfloat16 *)q->ptr, (const __nv_bfloat16 *)k->ptr,
-                                  (const __nv_bfloat16 *)v->ptr, (__nv_bfloat16 *)out->ptr, (int)b, (int)t, (int)pos0,
-                                  (int)n_heads, (int)n_kv, (int)t_max, 0.125f /* 64^-0.5, model.rs:236 */, 1);
+  ugb_prefill_attention_args a;
+  a.q = (const __nv_bfloat16 *)q->ptr; a.k = (const __nv_bfloat16 *)k->ptr; a.v = (const __nv_bfloat16 *)v->ptr;
+  a.out = (__nv_bfloat16 *)out->ptr;
+  a.batch = (int)b; a.t = (int)t; a.pos0 = (int)pos0; a.n_heads = (int)n_heads; a.n_kv = (int)n_kv; a.kv_rows = (int)t_max;
+  a.scale = 0.125f;   // 64^-0.5, model.rs:236
+  return ugb_prefill_attention_tc(dev, a);
 }

@@ -4,11 +4,22 @@
 
 #include "ugb_internal.h"
 
-// out[b, i, head, :] = softmax_j(scale * q[b, i, head, :] . k[b, kvh, j, :]) v[b, kvh, j, :] over the cached
-// positions j <= pos0 + i, for i in [0, t).  q bf16 [batch, t, n_heads, 64] (rope applied), caches bf16
-// [batch, n_kv, t_max, 64], out bf16 [batch, t, n_heads * 64].  All base pointers 16-byte aligned.
-// dynamic != 0: the persistent CTAs draw their work items from the device's counter (longest first);
-// 0: the items are dealt round-robin.
-int32_t ugb_prefill_attention_tc(ugb_device *dev, const __nv_bfloat16 *q, const __nv_bfloat16 *kcache,
-                                 const __nv_bfloat16 *vcache, __nv_bfloat16 *out, int batch, int t, int pos0,
-                                 int n_heads, int n_kv, int t_max, float scale, int dynamic);
+// out[b, i, head, :] = gate softmax_j(scale * q[b, i, head, :] . k[b, kvh, j, :]) v[b, kvh, j, :] over the cached
+// positions j <= pos0 + i, for i in [0, t).  All base pointers 16-byte aligned.
+struct ugb_prefill_attention_args {
+  const __nv_bfloat16 *q;          // [batch, t, n_heads, dq]
+  const __nv_bfloat16 *k, *v;      // [batch, n_kv, kv_rows, dq / dv], or token_major: [batch, kv_rows, n_kv, dq / dv]
+  __nv_bfloat16 *out;              // [batch, t, n_heads * dv]
+  int batch, t, pos0, n_heads, n_kv;
+  int kv_rows;                     // positions the k / v buffers hold per sequence (>= pos0 + t)
+  int token_major = 0;
+  int dq = 64, dv = 64;            // 64 or 128 each
+  float scale;
+  const float *gate = nullptr;     // f32 [batch * t][gate_ld]: factor per query and head
+  int gate_ld = 0;
+  int dynamic = 1;                 // the persistent CTAs draw their work items from the device's counter (longest
+                                   // first); 0: the items are dealt round-robin
+};
+// Padded head width the kernel wants for `dim` values per head, 0 when it has none.
+int ugb_prefill_attention_width(int dim);
+int32_t ugb_prefill_attention_tc(ugb_device *dev, const ugb_prefill_attention_args &a);

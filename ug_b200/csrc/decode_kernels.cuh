@@ -690,15 +690,15 @@ decode_attention_kernel_t(const __nv_bfloat16 *__restrict__ q, __nv_bfloat16 *__
 
 // next[b] = argmax_j logits[b, j] (ties -> lowest index); thread 0 of CTA 0 also
 // advances the shared position counter.  One CTA of 1024 threads per row,
-// 128-bit loads (vocab % 4 == 0).
+// 128-bit loads; rows of `vocab` values, ld elements apart (ld % 4 == 0).
 static __global__ void __launch_bounds__(1024)
-argmax_rows_kernel(const float *__restrict__ logits, int vocab, int *__restrict__ next, int *pos_p) {
+argmax_rows_kernel(const float *__restrict__ logits, int vocab, int ld, int *__restrict__ next, int *pos_p) {
   __shared__ float sv[32];
   __shared__ int si[32];
   ugb_pdl_trigger();
   ugb_pdl_wait();
   const int b = blockIdx.x;
-  const float4 *row = reinterpret_cast<const float4 *>(logits + (size_t)b * vocab);
+  const float4 *row = reinterpret_cast<const float4 *>(logits + (size_t)b * ld);
   float best = -INFINITY;
   int bi = 0x7fffffff;
   auto upd = [&](float v, int j) { if (v > best || (v == best && j < bi)) { best = v; bi = j; } };
@@ -706,6 +706,7 @@ argmax_rows_kernel(const float *__restrict__ logits, int vocab, int *__restrict_
     const float4 v = __ldcs(row + j);
     upd(v.x, 4 * j); upd(v.y, 4 * j + 1); upd(v.z, 4 * j + 2); upd(v.w, 4 * j + 3);
   }
+  if (threadIdx.x < (vocab & 3)) upd(logits[(size_t)b * ld + (vocab & ~3) + threadIdx.x], (vocab & ~3) + threadIdx.x);
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) {
     const float ov = __shfl_xor_sync(0xffffffffu, best, o);

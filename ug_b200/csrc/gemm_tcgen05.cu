@@ -61,7 +61,10 @@ template <int BM, int BN, bool PAIR = false> struct Cfg {
   static constexpr int SMEM_BYTES = STAGES * STAGE_BYTES + 1024 /*alignment slack*/ + 512 /*barriers*/;
   // pair_k (two CTAs split k and exchange sums): f32 [64][BN / 2] behind the barriers, where it fits
   static constexpr int PARK_BYTES = 64 * (BN / 2) * 4;
-  static constexpr bool PAIR_K_OK = BM == 64 && !PAIR && BN % 32 == 0 && SMEM_BYTES + PARK_BYTES <= 227 * 1024;
+  static constexpr bool PAIR_K_OK = BM == 64 && !PAIR && BN % 32 == 0;
+  static constexpr int SMEM_LIMIT = 227 * 1024;
+  static constexpr int SMEM_ATTR = PAIR_K_OK && SMEM_BYTES + PARK_BYTES > SMEM_LIMIT ? SMEM_LIMIT
+                                 : SMEM_BYTES + (PAIR_K_OK ? PARK_BYTES : 0);
 };
 
 struct Params {
@@ -80,6 +83,7 @@ struct Params {
   int pair_k;             // 1: CTAs 2c and 2c + 1 are a cluster and take the two k halves of tile c (BM = 64,
                           // UGB_EPI_SILU_MUL_BF16): rank 1 hands its sums to rank 0 through shared memory
   long long c_batch;      // output elements between batch steps
+  long long c_ld;         // output elements between rows
   long long c_split;      // output elements between split-K partials
   void *C;
   ugb_status_word *status;
@@ -87,6 +91,11 @@ struct Params {
 };
 
 using namespace ugb_tc;
+
+static __device__ __forceinline__ uint32_t relu2_bits(uint32_t bits) {
+  const float x = fmaxf(__uint_as_float(bits), 0.f);
+  return __float_as_uint(x * x);
+}
 
 // Measurement aid: CTA 0 of a launch with p.prof set records when it passed the points UGB_TC_PROF_* name.
 #define UGB_TC_STAMP(i)                                                      \
@@ -452,8 +461,12 @@ tc_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
         tmem_ld_wait();
         if (row_lane && row < p.M) {
           const int col0 = n0 + c * 32;
-          if (p.epi == UGB_EPI_BF16) {
-            __nv_bfloat16 *crow = (__nv_bfloat16 *)p.C + out_off + (long long)row * p.N + col0;
+          if (p.epi == UGB_EPI_BF16 || p.epi == UGB_EPI_RELU2_BF16) {
+            __nv_bfloat16 *crow = (__nv_bfloat16 *)p.C + out_off + (long long)row * p.c_ld + col0;
+            if (p.epi == UGB_EPI_RELU2_BF16) {
+#pragma unroll
+              for (int e = 0; e < 32; ++e) v[e] = relu2_bits(v[e]);
+            }
 #pragma unroll
             for (int q = 0; q < 4; ++q) {
               if (c * 32 + q * 8 < BN && col0 + q * 8 < p.N) {   // BN % 8 == N % 8 == 0: a chunk of 8 is all in or all out
@@ -475,14 +488,14 @@ tc_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
               }
             }
           } else if (p.epi == UGB_EPI_F32) {
-            float *crow = (float *)p.C + out_off + (long long)row * p.N + col0;
+            float *crow = (float *)p.C + out_off + (long long)row * p.c_ld + col0;
 #pragma unroll
             for (int q = 0; q < 8; ++q)
               if (c * 32 + q * 4 < BN && col0 + q * 4 < p.N)
                 *reinterpret_cast<uint4 *>(crow + q * 4) = make_uint4(v[q * 4], v[q * 4 + 1], v[q * 4 + 2], v[q * 4 + 3]);
           } else {
             // UGB_EPI_SILU_MUL_BF16: columns come in (gate, up) pairs; out [M, N/2] bf16
-            __nv_bfloat16 *crow = (__nv_bfloat16 *)p.C + out_off + (long long)row * (p.N / 2) + col0 / 2;
+            __nv_bfloat16 *crow = (__nv_bfloat16 *)p.C + out_off + (long long)row * p.c_ld + col0 / 2;
 #pragma unroll
             for (int q = 0; q < 2; ++q) {
               if (c * 32 + q * 16 < BN && col0 + q * 16 < p.N) {
@@ -538,7 +551,28 @@ tc_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
           if (row_lane && row < p.M) {
             const int col0 = pair_n0 + c * 32;
             // out [M, N/2] bf16 = silu(gate) * up over the summed (gate, up) column pairs
-            __nv_bfloat16 *crow = (__nv_bfloat16 *)p.C + (long long)row * (p.N / 2) + col0 / 2;
+            __nv_bfloat16 *crow = (__nv_bfloat16 *)p.C + (long long)row * p.c_ld + col0 / 2;
+            if (p.epi == UGB_EPI_RELU2_BF16) {                      // out [M, N] bf16 = max(sum, 0)^2
+              __nv_bfloat16 *frow = (__nv_bfloat16 *)p.C + (long long)row * p.c_ld + col0;
+#pragma unroll
+              for (int q = 0; q < 4; ++q) {
+                if (mine(2 * c + q / 2) && col0 + q * 8 < p.N) {
+                  const float4 w0 = *reinterpret_cast<const float4 *>(park + c * 32 + q * 8);
+                  const float4 w1 = *reinterpret_cast<const float4 *>(park + c * 32 + q * 8 + 4);
+                  const float wv[8] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
+                  uint32_t o[4];
+#pragma unroll
+                  for (int e = 0; e < 4; ++e) {
+                    const float s0 = fmaxf(__uint_as_float(v[q * 8 + 2 * e]) + wv[2 * e], 0.f);
+                    const float s1 = fmaxf(__uint_as_float(v[q * 8 + 2 * e + 1]) + wv[2 * e + 1], 0.f);
+                    __nv_bfloat162 t = __floats2bfloat162_rn(s0 * s0, s1 * s1);
+                    o[e] = *(uint32_t *)&t;
+                  }
+                  *reinterpret_cast<uint4 *>(frow + q * 8) = make_uint4(o[0], o[1], o[2], o[3]);
+                }
+              }
+              continue;
+            }
 #pragma unroll
             for (int q = 0; q < 2; ++q) {
               if (mine(2 * c + q) && col0 + q * 16 < p.N) {
@@ -632,7 +666,7 @@ int32_t launch_tc(ugb_device *dev, TcState *st, const ugb_tc_gemm_args &g, size_
   constexpr int slot = PAIR ? 8 : BN == 160 ? 9 : BN == 80 ? 6 : BN == 96 ? 7 : (BN == 256 ? 2 : (BN == 128 ? 1 : 0)) + (BM == 64 ? 3 : 0);
   if (!st->attr_set[slot]) {
     UGB_CUDA(dev, cudaFuncSetAttribute(tc_gemm_kernel<BM, BN, PAIR>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                       C_::SMEM_BYTES + (C_::PAIR_K_OK ? C_::PARK_BYTES : 0)));
+                                       C_::SMEM_ATTR));
 
     st->attr_set[slot] = true;
   }
@@ -654,7 +688,7 @@ int32_t launch_tc(ugb_device *dev, TcState *st, const ugb_tc_gemm_args &g, size_
   p.pair_k = 0;
   if (g.pair_k) {
     // two CTAs (a cluster) per tile, each over half of k
-    if (!C_::PAIR_K_OK || g.epi != UGB_EPI_SILU_MUL_BF16 || batch != 1 || p.k_blocks < 2 ||
+    if (!C_::PAIR_K_OK || (g.epi != UGB_EPI_SILU_MUL_BF16 && g.epi != UGB_EPI_RELU2_BF16) || batch != 1 || p.k_blocks < 2 ||
         2 * (long long)p.tiles_m * p.tiles_n > dev->sm_count)
       return UGB_ERR_UNSUPPORTED;
     p.pair_k = 1;
@@ -665,15 +699,17 @@ int32_t launch_tc(ugb_device *dev, TcState *st, const ugb_tc_gemm_args &g, size_
   // from L2 again and again, so it should be the smaller one: B (n x k) when n <= m, otherwise A.
   p.n_fast = n <= m ? 1 : 0;
   const long long out_cols = g.epi == UGB_EPI_SILU_MUL_BF16 ? (long long)n / 2 : (long long)n;
-  p.c_batch = g.c_batch ? g.c_batch : (long long)m * out_cols;
-  p.c_split = (long long)batch * m * out_cols;
+  p.c_ld = g.c_ld ? g.c_ld : out_cols;
+  p.c_batch = g.c_batch ? g.c_batch : (long long)m * p.c_ld;
+  p.c_split = (long long)batch * m * p.c_ld;
   p.C = g.out;
   p.status = dev->status_dev;
   p.rope = g.rope;
 
   CUtensorMap tmA, tmB;
+  const uint64_t a_ld = g.a_ld ? (uint64_t)g.a_ld : (uint64_t)k;
   p.stage_tx = C_::STAGE_BYTES * (PAIR ? 2 : 1);      // PAIR: one barrier counts both CTAs' stage
-  int32_t rc = encode_map(dev, st, &tmA, g.a, k, m, batch, k, batch > 1 ? (uint64_t)g.a_batch : m * k, BK, BM, g.f16);
+  int32_t rc = encode_map(dev, st, &tmA, g.a, k, m, batch, a_ld, batch > 1 ? (uint64_t)g.a_batch : m * a_ld, BK, BM, g.f16);
   if (rc) return rc;
   const uint64_t nb = p.b_batched ? batch : 1;
   const uint64_t bs = p.b_batched ? (uint64_t)g.b_batch : n * k;
@@ -691,6 +727,8 @@ int32_t launch_tc(ugb_device *dev, TcState *st, const ugb_tc_gemm_args &g, size_
     const int fit = (g.smem_kib * 1024 - 1536) / C_::STAGE_BYTES;
     stages = fit < 2 ? 2 : (fit > stages ? stages : fit);
   }
+  // with the parking area of pair_k behind the ring, a stage may have to go
+  if (p.pair_k) while (stages > 2 && stages * C_::STAGE_BYTES + 1536 + C_::PARK_BYTES > C_::SMEM_LIMIT) --stages;
   p.stages = stages;
   // pair_k: behind the barriers, the parking area the other k half writes its sums into (f32 [64][BN / 2])
   const size_t smem = (size_t)stages * C_::STAGE_BYTES + 1536 + (p.pair_k ? (size_t)C_::PARK_BYTES : 0);
@@ -739,6 +777,7 @@ int32_t ugb_tc_gemm(ugb_device *dev, const ugb_tc_gemm_args &g) {
   if (k == 0 || k % 8 != 0 || n % 8 != 0) return UGB_ERR_UNSUPPORTED;
   if (((uintptr_t)g.a | (uintptr_t)g.b | (uintptr_t)g.out) & 15) return UGB_ERR_UNSUPPORTED;
   if ((g.a_batch % 8) != 0 || (g.b_batch % 8) != 0 || g.a_batch < 0 || g.b_batch < 0) return UGB_ERR_UNSUPPORTED;
+  if (g.a_ld < 0 || g.c_ld < 0 || g.a_ld % 8 != 0 || g.c_ld % 8 != 0 || g.c_batch % 8 != 0) return UGB_ERR_UNSUPPORTED;
   if (batch > 1 && g.a_batch == 0) return UGB_ERR_UNSUPPORTED;
   if (m > (1u << 30) || n > (1u << 30) || k > (1u << 30) || batch > 65535) return UGB_ERR_UNSUPPORTED;
   if (g.epi == UGB_EPI_SILU_MUL_BF16 && n % 16 != 0) return UGB_ERR_UNSUPPORTED;
@@ -751,7 +790,7 @@ int32_t ugb_tc_gemm(ugb_device *dev, const ugb_tc_gemm_args &g) {
   if (int32_t rc = ensure_encode(dev, st)) return rc;
   // A shared B with densely stacked A batches is one tall GEMM.
   const long long dense_c = (long long)m * (long long)(g.epi == UGB_EPI_SILU_MUL_BF16 ? n / 2 : n);
-  if (batch > 1 && g.b_batch == 0 && g.a_batch == (long long)(m * k) && (g.c_batch == 0 || g.c_batch == dense_c)) {
+  if (batch > 1 && g.b_batch == 0 && g.a_ld == 0 && g.c_ld == 0 && g.a_batch == (long long)(m * k) && (g.c_batch == 0 || g.c_batch == dense_c)) {
     m *= batch;
     batch = 1;
   }

@@ -10,6 +10,7 @@ enum {
   UGB_EPI_BF16 = 0,           // out [b, m, n] in the operands' 16-bit type (bf16, or f16 with args.f16)
   UGB_EPI_F32 = 1,            // out f32 [splits, b, m, n]  (split-K partials when splits > 1)
   UGB_EPI_SILU_MUL_BF16 = 2,  // columns are (gate, up) pairs: out bf16 [b, m, n/2] = silu(gate) * up
+  UGB_EPI_RELU2_BF16 = 4,     // out bf16 [b, m, n] = max(x, 0)^2
   UGB_EPI_ROPE_QKV = 3        // columns are [q heads | k heads | v heads] of 64: rope + KV append (see ugb_tc_rope_epilogue)
 };
 
@@ -38,6 +39,7 @@ struct ugb_tc_gemm_args {
   size_t batch, m, n, k;
   long long a_batch, b_batch;   // elements between batch steps (b_batch 0 = shared operand)
   long long c_batch = 0;        // output elements between batch steps; 0 = dense (m * output columns)
+  long long a_ld = 0, c_ld = 0; // elements between the rows of A and of the output; 0 = dense (k, output columns)
   bool b_is_nk;
   int epi;              // UGB_EPI_*
   int splits;           // split-K factor (only with UGB_EPI_F32); the kernel may use fewer
@@ -46,7 +48,7 @@ struct ugb_tc_gemm_args {
   bool pdl;             // launch with programmatic stream serialization (see ugb_launch)
   int smem_kib = 0;     // cap on the shared memory of a CTA (ring depth follows); 0 = as deep as fits in 220 KiB
   bool f16 = false;     // operands (and the UGB_EPI_BF16 output) are IEEE f16 instead of bf16: same instruction, other format field
-  bool pair_k = false;  // m <= 64, UGB_EPI_SILU_MUL_BF16: two CTAs (a thread-block cluster) per tile, each over half of k; the
+  bool pair_k = false;  // m <= 64, UGB_EPI_SILU_MUL_BF16 or UGB_EPI_RELU2_BF16: two CTAs (a thread-block cluster) per tile, each over half of k; the
                         // second hands its sums to the first through distributed shared memory.  UGB_ERR_UNSUPPORTED when
                         // twice the tiles exceed the SMs
   unsigned long long *prof = nullptr;   // measurement aid, see UGB_TC_PROF_*

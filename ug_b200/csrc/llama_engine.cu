@@ -21,12 +21,14 @@
 // HBM layout per model: weights [layer]{wqkv [(h+2kv)*d, hidden], wo [hidden, h*d], wgu [2*ffn, hidden]
 // (gate row j at 2j, up row j at 2j+1), wdown [hidden, ffn]}, embedding [vocab, hidden]; KV cache K and V
 // each [layer][batch][kv_head][t_max][head_dim] bf16 (t_max rounded up to 16).
+#include <algorithm>
 #include <cmath>
 #include <cstring>
 #include <string>
 #include <vector>
 
 #include "decode_kernels.cuh"
+#include "engine_core.cuh"
 #include "gemm_tcgen05.cuh"
 #include "tp_kernels.cuh"
 #include "attention_tc.cuh"
@@ -39,16 +41,14 @@ struct LayerW {
   float *rms1 = nullptr, *rms2 = nullptr;
 };
 
-struct ugb_llama {
-  ugb_device *dev = nullptr;
+struct ugb_llama : ugb_engine {   // t_max is padded to a multiple of 16
   ugb_llama_config cfg{};         // the whole model (weight shapes, vocabulary range)
   ugb_llama_config lc{};          // this rank's share: n_heads, n_kv_heads and ffn are the local counts
-  int batch = 0, t_max = 0;       // t_max padded to a multiple of 16
   // tensor parallelism: rank tp_rank of tp_size owns query heads [q0, q0 + lc.n_heads), KV heads
   // [kv0, kv0 + lc.n_kv_heads) (a KV head is replicated when tp_size > n_kv_heads), FFN columns
   // [tp_rank * lc.ffn, ...) and logit columns [tp_rank * vl, ...).  tp == false: one rank, plain kernels.
   bool tp = false;
-  int tp_rank = 0, tp_size = 1, q0 = 0, kv0 = 0, vl = 0;
+  int tp_rank = 0, tp_size = 1, q0 = 0, kv0 = 0;
   void *tp_block = nullptr;       // exchange block of this rank (header, o / down partials, argmax pairs)
   size_t tp_off_o = 0, tp_off_down = 0, tp_off_pairs = 0, tp_block_bytes = 0, tp_part_rows = 0;
   void *tp_peer[TP_MAX] = {};     // every rank's exchange block as mapped here (own included)
@@ -62,27 +62,17 @@ struct ugb_llama {
   __nv_bfloat16 *kcache = nullptr, *vcache = nullptr;
   size_t kv_layer_stride = 0;     // elements per layer of one cache
   // activations / scratch
-  float *x = nullptr, *part = nullptr, *logits = nullptr;
+  float *x = nullptr, *part = nullptr;
   __nv_bfloat16 *xn = nullptr, *q = nullptr, *att = nullptr, *h = nullptr;
   float *att_po = nullptr, *att_pml = nullptr;
   unsigned int *att_cnt = nullptr;
-  int *tok = nullptr, *next = nullptr, *pos = nullptr;
-  int host_pos = 0;
+  int *tok = nullptr;
   // tuning
   int splits_qkv = 5, splits_o = 8, splits_down = 8, att_splits = 1, att_stages = 5;
-  int pdl = 1;                    // programmatic dependent launch between the kernels of a step
   int gemm_smem_kib = 144;        // shared-memory cap of the decode GEMM CTAs (0 = deepest ring); measured best
   int skip = 0;                   // measurement aid: bit mask of kernel types left out of the step
   int bn_qkv = 128, bn_o = 128, bn_gate_up = 128, bn_down = 128, bn_lm_head = 256;   // GEMM tile widths
   size_t part_elems = 0;
-  // graph of one step that reads `next` as its input tokens
-  cudaGraphExec_t graph = nullptr;
-  int graph_nodes = 0;
-  bool warmed = false;
-  std::vector<void *> allocs;
-  size_t loaded = 0;
-  // prefill workspace, allocated by the first ugb_llama_prefill: activations of one chunk of
-  // pf_rows = batch * pf_chunk rows (pf_chunk positions of every sequence)
   // persistent decode-step kernel (decode_step.cu): option step_kernel
   int step_kernel = 0;            // 1: a decode step is one launch of decode_step_kernel + lm_head + argmax
   bool step_ready = false;
@@ -99,35 +89,23 @@ struct ugb_llama {
   std::vector<CUtensorMap> att_kmap, att_vmap;   // per layer, for the TMA variant
   int pf_att_tc = 1;              // option prefill_attention_tc: 1 = tcgen05 / TMEM attention kernel drawing its
                                   // work items from a counter, 2 = the same dealt round-robin, 0 = mma.sync kernel
-  int pf_rows_max = 8192;         // option prefill_rows: upper bound on rows per chunk
-  int pf_rows = 0, pf_chunk = 0;
+  // prefill workspace: activations of one chunk of pf_rows rows
   float *pf_x = nullptr, *pf_f32 = nullptr;            // residual stream; f32 GEMM output (qkv, o, down)
   __nv_bfloat16 *pf_xn = nullptr, *pf_q = nullptr, *pf_att = nullptr, *pf_h = nullptr;
   int *pf_tok = nullptr;
   size_t pf_tok_cap = 0;
-  float *pf_logits = nullptr;     // [batch, pf_logits_t, vocab] when all-position logits were requested
-  int pf_logits_t = 0;
-  size_t pf_logits_cap = 0;
+
+  int position_limit() const override { return std::min(t_max, (int)cfg.max_pos); }
+  int32_t before_step() override;
+  int32_t before_prefill() override;
+  int32_t enqueue_step(const int *tok) override;
+  int32_t ensure_prefill_workspace() override;
+  int32_t enqueue_prefill_chunk(const int *tok, int t, int c0, int tc, bool all_logits) override;
+  int32_t enqueue_prefill_tail(int tc) override;
+  int32_t enqueue_head(bool after_step) override;
 };
 
 namespace {
-
-template <typename T>
-int32_t dmalloc(ugb_llama *m, T **p, size_t n, bool zero = false) {
-  ugb_device *dev = m->dev;
-  void *v = nullptr;
-  UGB_CUDA(dev, cudaMalloc(&v, n * sizeof(T) ? n * sizeof(T) : 16));
-  if (zero) UGB_CUDA(dev, cudaMemsetAsync(v, 0, n * sizeof(T), dev->stream));
-  m->allocs.push_back(v);
-  *p = (T *)v;
-  return UGB_OK;
-}
-
-__global__ void f32_to_bf16_kernel(const float *__restrict__ s, __nv_bfloat16 *__restrict__ d, size_t n,
-                                   size_t row_len, size_t dst_pitch, size_t src_pitch) {
-  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x)
-    d[(i / row_len) * dst_pitch + i % row_len] = __float2bfloat16_rn(s[(i / row_len) * src_pitch + i % row_len]);
-}
 
 // Copies rows [row0, row0 + nrows) x columns [col0, col0 + ncols) of a [rows, cols] matrix (bf16, or f32
 // rounded to bf16) into `dst` with a destination row pitch in elements (interleaving gate/up uses
@@ -135,21 +113,7 @@ __global__ void f32_to_bf16_kernel(const float *__restrict__ s, __nv_bfloat16 *_
 // a tensor-parallel rank keeps its slice only.
 int32_t put_sub(ugb_llama *m, const ugb_slice *w, __nv_bfloat16 *dst, size_t rows, size_t cols, size_t row0,
                 size_t nrows, size_t col0, size_t ncols, size_t dst_pitch, const char *name) {
-  ugb_device *dev = m->dev;
-  UGB_REQUIRE(dev, w->len == rows * cols, UGB_ERR_SHAPE, "unexpected shape for %s: %zu elements, expected (%zu, %zu)",
-              name, w->len, rows, cols);
-  const size_t off = row0 * cols + col0;
-  if (w->dtype == UGB_BF16) {
-    UGB_CUDA(dev, cudaMemcpy2DAsync(dst, dst_pitch * 2, (const __nv_bfloat16 *)w->ptr + off, cols * 2, ncols * 2, nrows,
-                                    cudaMemcpyDeviceToDevice, dev->stream));
-  } else if (w->dtype == UGB_F32) {
-    f32_to_bf16_kernel<<<dev->sm_count * 8, 256, 0, dev->stream>>>((const float *)w->ptr + off, dst, nrows * ncols, ncols,
-                                                                    dst_pitch, cols);
-    return ugb_after_launch(dev, "f32_to_bf16_kernel");
-  } else {
-    return ugb_fail(dev, UGB_ERR_DTYPE, "%s: weights must be BF16 or F32", name);
-  }
-  return UGB_OK;
+  return engine_put_matrix(m, w, dst, UGB_BF16, rows, cols, row0, nrows, col0, ncols, dst_pitch, name);
 }
 
 int32_t put_matrix(ugb_llama *m, const ugb_slice *w, __nv_bfloat16 *dst, size_t rows, size_t cols,
@@ -275,7 +239,7 @@ int32_t launch_lm_head_argmax(ugb_llama *m, bool pdl_first) {
   const bool pdl = pdl_first && m->pdl != 0;
   cudaError_t e;
   if (!m->tp) {
-    e = ugb_launch(argmax_rows_kernel, dim3(m->batch), dim3(1024), 0, st, pdl, m->logits, m->vl, m->next, m->pos);
+    e = ugb_launch(argmax_rows_kernel, dim3(m->batch), dim3(1024), 0, st, pdl, m->logits, m->vl, m->logits_ld, m->next, m->pos);
     if (e != cudaSuccess) return ugb_fail(dev, UGB_ERR_CUDA, "launch of argmax_rows_kernel failed: %s", cudaGetErrorString(e));
     return ugb_after_launch(dev, "argmax_rows_kernel");
   }
@@ -418,7 +382,7 @@ int32_t tp_in_step(ugb_llama *m) {
 }
 
 // Enqueues one decode step on the device stream; `tok` holds the input ids.
-int32_t enqueue_step(ugb_llama *m, const int *tok) {
+int32_t llama_step(ugb_llama *m, const int *tok) {
   ugb_device *dev = m->dev;
   const ugb_llama_config &c = m->lc;         // this rank's share of heads and FFN columns
   cudaStream_t st = dev->stream;
@@ -479,7 +443,7 @@ int32_t enqueue_step(ugb_llama *m, const int *tok) {
 }
 
 // Activations for one prefill chunk; allocated once, freed with the model.
-int32_t ensure_prefill_workspace(ugb_llama *m) {
+int32_t llama_prefill_workspace(ugb_llama *m) {
   if (m->pf_rows) return UGB_OK;
   const ugb_llama_config &c = m->lc;
   int rows_max = m->pf_rows_max;
@@ -502,7 +466,7 @@ int32_t ensure_prefill_workspace(ugb_llama *m) {
 
 // One chunk of a prefill: positions c0 .. c0 + tc - 1 of a block of t per sequence, cache positions
 // host_pos + c0 onwards.  Rows are ordered (sequence, position).
-int32_t enqueue_prefill_chunk(ugb_llama *m, const int *tok, int t, int c0, int tc, bool all_logits) {
+int32_t llama_prefill_chunk(ugb_llama *m, const int *tok, int t, int c0, int tc, bool all_logits) {
   ugb_device *dev = m->dev;
   const ugb_llama_config &c = m->lc;
   cudaStream_t st = dev->stream;
@@ -537,8 +501,10 @@ int32_t enqueue_prefill_chunk(ugb_llama *m, const int *tok, int t, int c0, int t
       if ((rc = ugb_after_launch(dev, "rope_append_kernel"))) return rc;
     }
     if (m->pf_att_tc) {
-      if ((rc = ugb_prefill_attention_tc(dev, m->pf_q, kc, vc, m->pf_att, B, tc, m->host_pos + c0, c.n_heads, c.n_kv_heads,
-                                         m->t_max, scale, m->pf_att_tc == 1))) return rc;
+      ugb_prefill_attention_args pa;
+      pa.q = m->pf_q; pa.k = kc; pa.v = vc; pa.out = m->pf_att; pa.batch = B; pa.t = tc; pa.pos0 = m->host_pos + c0;
+      pa.n_heads = c.n_heads; pa.n_kv = c.n_kv_heads; pa.kv_rows = m->t_max; pa.scale = scale; pa.dynamic = m->pf_att_tc == 1;
+      if ((rc = ugb_prefill_attention_tc(dev, pa))) return rc;
     } else {
       prefill_attention_kernel<<<dim3((tc + PF_BQ - 1) / PF_BQ, c.n_heads, B), 128, 0, st>>>(
           m->pf_q, kc, vc, m->pf_att, tc, m->host_pos + c0, c.n_heads, c.n_kv_heads, m->t_max, scale);
@@ -572,6 +538,30 @@ bool ends_with(const std::string &s, const char *suffix) {
 }
 
 }  // namespace
+
+int32_t ugb_llama::before_step() {
+  if (int32_t in_step = tp_in_step(this)) return in_step;
+  if (step_ready && step_timeouts != dev->wait_timeouts) {
+    // a wait gave up since the barrier words were last known good (an aborted step leaves them half counted)
+    UGB_CUDA(dev, cudaMemsetAsync(step.sync, 0, 4 * sizeof(unsigned), dev->stream));
+    step_timeouts = dev->wait_timeouts;
+  }
+  return UGB_OK;
+}
+int32_t ugb_llama::before_prefill() { return tp_in_step(this); }
+int32_t ugb_llama::enqueue_step(const int *tok_in) { return llama_step(this, tok_in); }
+int32_t ugb_llama::ensure_prefill_workspace() { return llama_prefill_workspace(this); }
+int32_t ugb_llama::enqueue_prefill_chunk(const int *tok_in, int t, int c0, int tc, bool all_logits) {
+  return llama_prefill_chunk(this, tok_in, t, c0, tc, all_logits);
+}
+// Last position of every sequence -> the decode-shaped buffers (x already holds the last down_proj output).
+int32_t ugb_llama::enqueue_prefill_tail(int tc) {
+  const size_t H = cfg.hidden;
+  UGB_CUDA(dev, cudaMemcpy2DAsync(x, H * 4, pf_x + (size_t)(tc - 1) * H, (size_t)tc * H * 4, H * 4, batch,
+                                  cudaMemcpyDeviceToDevice, dev->stream));
+  return launch_reduce(this, batch, x, xn, RED_NONE, part, 0, ln_f);
+}
+int32_t ugb_llama::enqueue_head(bool after_step) { return launch_lm_head_argmax(this, after_step); }
 
 extern "C" {
 
@@ -623,7 +613,7 @@ int32_t ugb_llama_create_tp(ugb_device *dev, const ugb_llama_config *cfg, int32_
   m->timeouts_at_create = dev->wait_timeouts;
   m->q0 = tp_rank * c.n_heads;
   m->kv0 = tp_rank * g.n_kv_heads / n_rank;
-  m->vl = g.vocab / n_rank;
+  m->vl = m->logits_ld = g.vocab / n_rank;
   m->batch = batch;
   m->t_max = (t_max + 15) / 16 * 16;
   m->qkv_dim = (c.n_heads + 2 * c.n_kv_heads) * c.head_dim;
@@ -758,11 +748,10 @@ int32_t ugb_llama_destroy(ugb_llama *m) {
   if (!m) return UGB_ERR_INVALID;
   cudaSetDevice(m->dev->ordinal);
   cudaStreamSynchronize(m->dev->stream);
-  if (m->graph) cudaGraphExecDestroy(m->graph);
+  engine_drop_graph(m);
   for (int r = 0; r < m->tp_size; ++r)
     if (r != m->tp_rank && m->tp_peer[r]) cudaIpcCloseMemHandle(m->tp_peer[r]);
-  for (void *p : m->allocs) cudaFree(p);
-  if (m->pf_logits) cudaFree(m->pf_logits);
+  engine_free(m);
   delete m;
   return UGB_OK;
 }
@@ -810,31 +799,31 @@ int32_t ugb_llama_set_option(ugb_llama *m, const char *key, int32_t value) {
   const std::string k(key);
   if (k == "measure_skip_mask") {   // measurement aid: results of a step are meaningless while it is non-zero
     m->skip = value;
-    if (m->graph) { cudaGraphExecDestroy(m->graph); m->graph = nullptr; }
+    engine_drop_graph(m);
     return UGB_OK;
   }
   if (k == "pdl") {
     m->pdl = value != 0;
-    if (m->graph) { cudaGraphExecDestroy(m->graph); m->graph = nullptr; }
+    engine_drop_graph(m);
     return UGB_OK;
   }
   if (k == "gemm_smem_kib") {
     UGB_REQUIRE(dev, value == 0 || (value >= 32 && value <= 220), UGB_ERR_INVALID, "option gemm_smem_kib: %d outside 32..220 (0 = no cap)", value);
     m->gemm_smem_kib = value;
-    if (m->graph) { cudaGraphExecDestroy(m->graph); m->graph = nullptr; }
+    engine_drop_graph(m);
     return UGB_OK;
   }
   if (k == "step_kernel") {
     UGB_REQUIRE(dev, value == 0 || value == 1, UGB_ERR_INVALID, "option step_kernel: %d is not 0 or 1", value);
     m->step_kernel = value;
-    if (m->graph) { cudaGraphExecDestroy(m->graph); m->graph = nullptr; }
+    engine_drop_graph(m);
     m->warmed = false;            // the kernel's attributes are set by its first, eager launch
     if (value && !m->tp && m->batch <= 64) return ensure_step_kernel(m);
     return UGB_OK;
   }
   if (k == "step_tune") {         // measurement aid of the persistent step kernel; non-zero values give wrong results
     m->step.tune = value;
-    if (m->graph) { cudaGraphExecDestroy(m->graph); m->graph = nullptr; }
+    engine_drop_graph(m);
     return UGB_OK;
   }
   if (k == "step_profile") {      // measurement aid: barrier time stamps of the persistent step kernel (UGB_LLAMA_STEP_PROFILE)
@@ -845,12 +834,12 @@ int32_t ugb_llama_set_option(ugb_llama *m, const char *key, int32_t value) {
       m->step.prof = buf;
     }
     if (!value) m->step.prof = nullptr;
-    if (m->graph) { cudaGraphExecDestroy(m->graph); m->graph = nullptr; }
+    engine_drop_graph(m);
     return UGB_OK;
   }
   if (k == "att_early") {
     m->att_early = value != 0;
-    if (m->graph) { cudaGraphExecDestroy(m->graph); m->graph = nullptr; }
+    engine_drop_graph(m);
     return UGB_OK;
   }
   if (k == "gemm_profile") {      // measurement aid: time stamps inside the decode projections (UGB_LLAMA_GEMM_PROFILE)
@@ -860,23 +849,23 @@ int32_t ugb_llama_set_option(ugb_llama *m, const char *key, int32_t value) {
       m->gemm_prof = buf;
     }
     if (!value) m->gemm_prof = nullptr;
-    if (m->graph) { cudaGraphExecDestroy(m->graph); m->graph = nullptr; }
+    engine_drop_graph(m);
     return UGB_OK;
   }
   if (k == "gate_up_pair") {
     m->gate_up_pair = value != 0;
-    if (m->graph) { cudaGraphExecDestroy(m->graph); m->graph = nullptr; }
+    engine_drop_graph(m);
     m->warmed = false;
     return UGB_OK;
   }
   if (k == "att_cluster") {
     m->att_cluster = value != 0;
-    if (m->graph) { cudaGraphExecDestroy(m->graph); m->graph = nullptr; }
+    engine_drop_graph(m);
     return UGB_OK;
   }
   if (k == "att_tma") {
     m->att_tma = value != 0;
-    if (m->graph) { cudaGraphExecDestroy(m->graph); m->graph = nullptr; }
+    engine_drop_graph(m);
     return UGB_OK;
   }
   if (k == "prefill_attention_tc") {
@@ -899,7 +888,7 @@ int32_t ugb_llama_set_option(ugb_llama *m, const char *key, int32_t value) {
     else if (k == "bn_down") m->bn_down = value;
     else if (k == "bn_lm_head") m->bn_lm_head = value;
     else return ugb_fail(dev, UGB_ERR_INVALID, "unknown option %s", key);
-    if (m->graph) { cudaGraphExecDestroy(m->graph); m->graph = nullptr; }
+    engine_drop_graph(m);
     m->warmed = false;   // a tile width used for the first time sets a kernel attribute: run one step eagerly
     return UGB_OK;
   }
@@ -910,111 +899,20 @@ int32_t ugb_llama_set_option(ugb_llama *m, const char *key, int32_t value) {
   else if (k == "att_splits") m->att_splits = value;
   else if (k == "att_stages") m->att_stages = value < 2 ? 2 : (value > 6 ? 6 : value);
   else return ugb_fail(dev, UGB_ERR_INVALID, "unknown option %s", key);
-  if (m->graph) { cudaGraphExecDestroy(m->graph); m->graph = nullptr; }
+  engine_drop_graph(m);
   return UGB_OK;
 }
 
-int32_t ugb_llama_reset(ugb_llama *m, int32_t pos) {
-  if (!m) return UGB_ERR_INVALID;
-  ugb_device *dev = m->dev;
-  UGB_REQUIRE(dev, pos >= 0 && pos < m->t_max, UGB_ERR_INVALID, "reset position %d outside 0..%d", pos, m->t_max - 1);
-  UGB_CUDA(dev, cudaMemcpyAsync(m->pos, &pos, 4, cudaMemcpyHostToDevice, dev->stream));
-  UGB_CUDA(dev, cudaStreamSynchronize(dev->stream));
-  m->host_pos = pos;
-  return UGB_OK;
-}
+int32_t ugb_llama_reset(ugb_llama *m, int32_t pos) { return m ? engine_reset(m, pos) : UGB_ERR_INVALID; }
 
 int32_t ugb_llama_position(const ugb_llama *m) { return m ? m->host_pos : -1; }
 
 int32_t ugb_llama_decode(ugb_llama *m, const ugb_slice *tokens, int32_t n_steps) {
-  if (!m) return UGB_ERR_INVALID;
-  ugb_device *dev = m->dev;
-  UGB_REQUIRE(dev, n_steps >= 1, UGB_ERR_INVALID, "n_steps must be >= 1");
-  UGB_REQUIRE(dev, tokens == nullptr || n_steps == 1, UGB_ERR_INVALID, "explicit tokens feed exactly one step");
-  UGB_REQUIRE(dev, m->host_pos + n_steps <= m->t_max && m->host_pos + n_steps <= m->cfg.max_pos, UGB_ERR_SHAPE,
-              "decode of %d steps from position %d exceeds the KV cache (%d positions)", n_steps, m->host_pos, m->t_max);
-  UGB_CUDA(dev, cudaSetDevice(dev->ordinal));
-  if (int32_t in_step = tp_in_step(m)) return in_step;
-  if (m->step_ready && m->step_timeouts != dev->wait_timeouts) {
-    // a wait gave up since the barrier words were last known good (an aborted step leaves them half counted)
-    UGB_CUDA(dev, cudaMemsetAsync(m->step.sync, 0, 4 * sizeof(unsigned), dev->stream));
-    m->step_timeouts = dev->wait_timeouts;
-  }
-  if (tokens) {
-    UGB_SLICE(dev, tokens, UGB_I32, (size_t)m->batch);
-    UGB_CUDA(dev, cudaMemcpyAsync(m->next, tokens->ptr, (size_t)m->batch * 4, cudaMemcpyDeviceToDevice, dev->stream));
-  }
-  int32_t rc;
-  for (int s = 0; s < n_steps; ++s) {
-    if (!m->warmed) {
-      // first step runs eagerly: it sets kernel attributes, which must not happen inside a capture
-      if ((rc = enqueue_step(m, m->next))) return rc;
-      m->warmed = true;
-    } else {
-      if (!m->graph) {
-        cudaGraph_t g = nullptr;
-        const uint64_t before = dev->launches;
-        UGB_CUDA(dev, cudaStreamBeginCapture(dev->stream, cudaStreamCaptureModeThreadLocal));
-        rc = enqueue_step(m, m->next);
-        cudaError_t e = cudaStreamEndCapture(dev->stream, &g);
-        m->graph_nodes = (int)(dev->launches - before);
-        dev->launches = before;
-        if (rc) { if (g) cudaGraphDestroy(g); return rc; }
-        if (e != cudaSuccess) return ugb_fail(dev, UGB_ERR_CUDA, "stream capture failed: %s", cudaGetErrorString(e));
-        e = cudaGraphInstantiate(&m->graph, g, 0);
-        cudaGraphDestroy(g);
-        if (e != cudaSuccess) return ugb_fail(dev, UGB_ERR_CUDA, "cudaGraphInstantiate failed: %s", cudaGetErrorString(e));
-      }
-      UGB_CUDA(dev, cudaGraphLaunch(m->graph, dev->stream));
-      dev->launches += (uint64_t)m->graph_nodes;
-    }
-    m->host_pos++;
-  }
-  return UGB_OK;
+  return m ? engine_decode(m, tokens, n_steps) : UGB_ERR_INVALID;
 }
 
 int32_t ugb_llama_prefill(ugb_llama *m, const ugb_slice *tokens, int32_t t, int32_t all_logits) {
-  if (!m) return UGB_ERR_INVALID;
-  ugb_device *dev = m->dev;
-  UGB_REQUIRE(dev, t >= 1, UGB_ERR_INVALID, "prefill of %d positions", t);
-  UGB_REQUIRE(dev, tokens != nullptr, UGB_ERR_INVALID, "ugb_llama_prefill: null tokens");
-  UGB_SLICE(dev, tokens, UGB_I32, (size_t)m->batch * t);
-  UGB_REQUIRE(dev, m->host_pos + t <= m->t_max && m->host_pos + t <= m->cfg.max_pos, UGB_ERR_SHAPE,
-              "prefill of %d positions from position %d exceeds the KV cache (%d positions)", t, m->host_pos, m->t_max);
-  UGB_CUDA(dev, cudaSetDevice(dev->ordinal));
-  if (int32_t in_step = tp_in_step(m)) return in_step;
-  const ugb_llama_config &c = m->cfg;
-  const size_t H = c.hidden;
-  int32_t rc;
-  if ((rc = ensure_prefill_workspace(m))) return rc;
-  if (all_logits) {
-    const size_t need = (size_t)m->batch * t * m->vl;
-    if (need > m->pf_logits_cap) {
-      UGB_CUDA(dev, cudaStreamSynchronize(dev->stream));
-      if (m->pf_logits) { cudaFree(m->pf_logits); m->pf_logits = nullptr; m->pf_logits_cap = 0; }
-      void *v = nullptr;
-      UGB_CUDA(dev, cudaMalloc(&v, need * sizeof(float)));
-      m->pf_logits = (float *)v;
-      m->pf_logits_cap = need;
-    }
-    m->pf_logits_t = t;
-  }
-  const int *tok = (const int *)tokens->ptr;
-  int tc = 0;
-  for (int c0 = 0; c0 < t; c0 += tc) {
-    tc = std::min(m->pf_chunk, t - c0);
-    if ((rc = enqueue_prefill_chunk(m, tok, t, c0, tc, all_logits != 0))) return rc;
-  }
-  // Last position of every sequence -> the decode-shaped buffers (x already holds the last down_proj
-  // output), final norm, lm_head, greedy choice.
-  UGB_CUDA(dev, cudaMemcpy2DAsync(m->x, H * 4, m->pf_x + (size_t)(tc - 1) * H, (size_t)tc * H * 4, H * 4, m->batch,
-                                  cudaMemcpyDeviceToDevice, dev->stream));
-  if ((rc = launch_reduce(m, m->batch, m->x, m->xn, RED_NONE, m->part, 0, m->ln_f))) return rc;
-  const int last = m->host_pos + t - 1;     // the argmax kernel advances the device-side position by one
-  UGB_CUDA(dev, cudaMemcpyAsync(m->pos, &last, 4, cudaMemcpyHostToDevice, dev->stream));
-  if ((rc = launch_lm_head_argmax(m, false))) return rc;
-  m->host_pos += t;
-  return UGB_OK;
+  return m ? engine_prefill(m, tokens, t, all_logits) : UGB_ERR_INVALID;
 }
 
 int32_t ugb_llama_read(ugb_llama *m, int32_t what, void *host_dst, size_t len) {
@@ -1164,7 +1062,7 @@ int32_t ugb_llama_tp_connect(ugb_llama *m, const void *handles, size_t handle_by
     m->tp_peer[r] = p;
   }
   m->tp_ready = true;
-  if (m->graph) { cudaGraphExecDestroy(m->graph); m->graph = nullptr; }
+  engine_drop_graph(m);
   return UGB_OK;
 }
 

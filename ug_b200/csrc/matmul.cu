@@ -216,14 +216,15 @@ f32_skinny_n_kernel(float *__restrict__ C, const float *__restrict__ A, const fl
 template <bool VEC>
 __global__ void __launch_bounds__(256, 2)
 f32_tile_kernel(float *__restrict__ C, const float *__restrict__ A, const float *__restrict__ B, int m, int n, int k,
-                long long a_rs, long long a_cs, long long a_b, long long b_rs, long long b_cs, long long b_b) {
+                long long a_rs, long long a_cs, long long a_b, long long b_rs, long long b_cs, long long b_b,
+                long long c_rs, long long c_b) {
   constexpr int BM = 128, BN = 128, BK = 8;
   __shared__ __align__(16) float As[2][BK][BM + 4];
   __shared__ __align__(16) float Bs[2][BK][BN + 4];
   const int batch = blockIdx.z, t = threadIdx.x;
   const float *Ab = A + (long long)batch * a_b;
   const float *Bb = B + (long long)batch * b_b;
-  float *Cb = C + (long long)batch * m * n;
+  float *Cb = C + (long long)batch * c_b;
   const int m0 = blockIdx.y * BM, n0 = blockIdx.x * BN;
   // one 4-element piece of each tile per thread: along the operand's contiguous direction
   const bool a_kc = a_cs == 1, b_nc = b_cs == 1;       // A: k contiguous?  B: n contiguous?
@@ -296,7 +297,7 @@ f32_tile_kernel(float *__restrict__ C, const float *__restrict__ A, const float 
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
       const int gj = n0 + h * 64 + tx * 4;
-      float *crow = Cb + (long long)gi * n + gj;
+      float *crow = Cb + (long long)gi * c_rs + gj;
       if (VEC && gj + 3 < n) {
         *reinterpret_cast<float4 *>(crow) = make_float4(acc[u][4 * h], acc[u][4 * h + 1], acc[u][4 * h + 2], acc[u][4 * h + 3]);
       } else {
@@ -340,8 +341,8 @@ int32_t launch_f32(ugb_device *dev, float *dst, const float *lhs, const float *r
   const size_t a_c = L.transposed ? m : k, a_ld = (size_t)(L.transposed ? L.cs : L.rs);
   const size_t b_c = R.transposed ? k : n, b_ld = (size_t)(R.transposed ? R.cs : R.rs);
   const bool vec = bases && a_c % 4 == 0 && a_ld % 4 == 0 && b_c % 4 == 0 && b_ld % 4 == 0 && n % 4 == 0;
-  if (vec) f32_tile_kernel<true><<<grid, 256, 0, dev->stream>>>(dst, lhs, rhs, (int)m, (int)n, (int)k, L.rs, L.cs, L.batch, R.rs, R.cs, R.batch);
-  else f32_tile_kernel<false><<<grid, 256, 0, dev->stream>>>(dst, lhs, rhs, (int)m, (int)n, (int)k, L.rs, L.cs, L.batch, R.rs, R.cs, R.batch);
+  if (vec) f32_tile_kernel<true><<<grid, 256, 0, dev->stream>>>(dst, lhs, rhs, (int)m, (int)n, (int)k, L.rs, L.cs, L.batch, R.rs, R.cs, R.batch, (long long)n, (long long)(m * n));
+  else f32_tile_kernel<false><<<grid, 256, 0, dev->stream>>>(dst, lhs, rhs, (int)m, (int)n, (int)k, L.rs, L.cs, L.batch, R.rs, R.cs, R.batch, (long long)n, (long long)(m * n));
   return ugb_after_launch(dev, "f32_tile_kernel");
 }
 
@@ -358,6 +359,24 @@ int32_t launch_simt(ugb_device *dev, void *dst, const void *lhs, const void *rhs
 }
 
 }  // namespace
+
+int32_t ugb_f32_gemm(ugb_device *dev, float *c, const float *a, const float *b, size_t batch, size_t m, size_t n, size_t k,
+                     size_t a_ld, size_t a_batch, bool b_is_nk, size_t b_batch, size_t c_ld, size_t c_batch) {
+  if (batch == 0 || m == 0 || n == 0) return UGB_OK;
+  if (batch == 1 && a_ld == k && c_ld == n && b_is_nk && k > 0) {   // a Linear: the skinny kernel takes few rows
+    const MatLayout L{(long long)k, 1, (long long)a_batch, false}, R{1, (long long)k, (long long)b_batch, true};
+    return launch_f32(dev, c, a, b, batch, m, n, k, L, R);
+  }
+  const dim3 grid((unsigned)((n + 127) / 128), (unsigned)((m + 127) / 128), (unsigned)batch);
+  UGB_REQUIRE(dev, batch <= 65535 && grid.y <= 65535 && m < (1u << 31) && n < (1u << 31) && k < (1u << 31), UGB_ERR_UNSUPPORTED,
+              "f32 product: extent too large");
+  const bool vec = al16(c) && al16(a) && al16(b) && k % 4 == 0 && n % 4 == 0 && a_ld % 4 == 0 && c_ld % 4 == 0 &&
+                   a_batch % 4 == 0 && b_batch % 4 == 0 && c_batch % 4 == 0;
+  const long long b_rs = b_is_nk ? 1 : (long long)n, b_cs = b_is_nk ? (long long)k : 1;
+  if (vec) f32_tile_kernel<true><<<grid, 256, 0, dev->stream>>>(c, a, b, (int)m, (int)n, (int)k, (long long)a_ld, 1, (long long)a_batch, b_rs, b_cs, (long long)b_batch, (long long)c_ld, (long long)c_batch);
+  else f32_tile_kernel<false><<<grid, 256, 0, dev->stream>>>(c, a, b, (int)m, (int)n, (int)k, (long long)a_ld, 1, (long long)a_batch, b_rs, b_cs, (long long)b_batch, (long long)c_ld, (long long)c_batch);
+  return ugb_after_launch(dev, "f32_tile_kernel");
+}
 
 extern "C" {
 

@@ -74,6 +74,11 @@ static inline cudaError_t ugb_malloc_async(ugb_device *dev, void **p, size_t byt
   return dev->pool ? cudaMallocFromPoolAsync(p, bytes, dev->pool, dev->stream) : cudaMallocAsync(p, bytes, dev->stream);
 }
 
+// c[b, m, n] = a[b, m, k] . w on the FP32 pipe, a row-major with row stride a_ld, w [n, k] (b_is_nk) or [k, n] row-major,
+// c with row stride c_ld; *_batch: elements between batch steps (0 = shared operand).
+int32_t ugb_f32_gemm(ugb_device *dev, float *c, const float *a, const float *b, size_t batch, size_t m, size_t n, size_t k,
+                     size_t a_ld, size_t a_batch, bool b_is_nk, size_t b_batch, size_t c_ld, size_t c_batch);
+
 // Records a formatted message on the device handle and returns `code`.
 int32_t ugb_fail(ugb_device *dev, int32_t code, const char *fmt, ...);
 // Checks the launch error of the kernel just enqueued and counts it.
