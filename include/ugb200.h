@@ -530,6 +530,120 @@ enum {
 UGB_API int32_t ugb_llama_time_kernel(ugb_llama *m, int32_t which, int32_t iters,
                                       float *ms_per_pass);
 
+/* --------------------------------------- decoders described by a list of layers */
+/* No counterpart in the reference, which has one fixed layer.  A decoder whose
+ * layers are listed one by one: each has a token mixer (a recurrence or latent
+ * attention) and optionally a feed-forward, both between two RMS norms
+ * (x += norm_b(f(conv(norm_a(x))))), the sublayer input optionally passed
+ * through a causal depthwise convolution, and the stream between layers
+ * optionally a learned average of all layer results so far.  With X_0 the
+ * normalised embedding and X_{i+1} the result of layer i, what layer i + 1
+ * reads is sum_{j <= i+1} dwa_i[j] X_j.  The step functions are those of
+ * ugb_llama: batch rows are independent sequences that share one position; a
+ * decode step is one captured CUDA graph; a prompt runs in chunks of positions
+ * and may be continued by further prompts or steps at any position.  Per
+ * sequence the engine keeps, by layer: the last taps - 1 convolution inputs of
+ * both sublayers, a f32 recurrent state, or one latent row per position. */
+typedef struct ugb_hybrid ugb_hybrid;
+
+enum { UGB_MIXER_MINGRU = 0, UGB_MIXER_LATENT_ATTENTION = 1 };
+enum { UGB_FF_NONE = 0, UGB_FF_RELU2 = 1 /* down(max(up h, 0)^2) */ };
+
+typedef struct {
+  int32_t width;           /* of the residual stream                                     */
+  int32_t vocab;
+  int32_t layers;
+  int32_t conv_taps;       /* taps of the sublayers' input convolution, 0 = none          */
+  int32_t depth_average;   /* 1: "l<i>.dwa" averages the layer results                    */
+  int32_t dtype;           /* UGB_BF16: bf16 weights and activations, f32 norms, residual
+                              stream, scores and recurrence; UGB_F32: everything f32 on the
+                              FP32 pipe                                                   */
+  float eps;               /* of every norm, inside the root                              */
+  float gain_offset;       /* gain of a stream norm = gain_offset + stored weight         */
+} ugb_hybrid_config;
+
+typedef struct {
+  int32_t mixer;           /* UGB_MIXER_*                                                 */
+  int32_t width;           /* mingru: recurrent channels                                  */
+  int32_t heads, dim, vdim, q_rank, kv_rank;   /* latent attention                        */
+  float scale;             /* latent attention: factor of the scores                      */
+  int32_t feed_forward;    /* UGB_FF_*                                                    */
+  int32_t ff;              /* feed-forward columns                                        */
+} ugb_hybrid_layer;
+
+enum { UGB_HYBRID_LOGITS = 0, UGB_HYBRID_NEXT_TOKENS = 1, UGB_HYBRID_HIDDEN = 2, UGB_HYBRID_PREFILL_LOGITS = 3,
+       UGB_HYBRID_LAYERS = 4 /* f32 [layers, batch * t, width] of the last prompt, option "keep_layers" */ };
+
+UGB_API int32_t ugb_hybrid_create(ugb_device *dev, const ugb_hybrid_config *cfg, const ugb_hybrid_layer *layers,
+                                  int32_t batch, int32_t t_max, ugb_hybrid **out);
+UGB_API int32_t ugb_hybrid_destroy(ugb_hybrid *m);
+/* One tensor by its safetensors name: "embed" [vocab, width], "embed.norm",
+ * "final.norm" [width], "head" [vocab, width]; of layer i, prefix "l<i>.":
+ * "norm1", "norm1b", "norm2", "norm2b" [width], "canon1", "canon2" [width, taps],
+ * "dwa" [i + 2], "mlp.up" [ff, width], "mlp.down" [width, ff]; mingru: "mix.z",
+ * "mix.x", "mix.g" [channels, width], "mix.z.b", "mix.x.b" [channels], "mix.o"
+ * [width, channels]; latent attention: "mix.dq" [q_rank, width], "mix.dq.norm",
+ * "mix.uq" [heads * dim, q_rank], "mix.dkv" [kv_rank, width], "mix.dkv.norm",
+ * "mix.uk" [heads * dim, kv_rank], "mix.uv" [heads * vdim, kv_rank], "mix.g"
+ * [heads, width], "mix.o" [width, heads * vdim].  BF16 or F32; f32 matrices are
+ * rounded to nearest even when the model is bf16. */
+UGB_API int32_t ugb_hybrid_load_weight(ugb_hybrid *m, const char *name, const ugb_slice *w);
+/* "pdl" (0 / 1), "prefill_rows" (16..65536, before the first prompt),
+ * "absorb_max" (blocks of at most this many positions run attention in the
+ * latent space instead of expanding keys and values, default 16), "att_splits"
+ * (slices of the cache per row in a decode step, 0 = chosen from the batch),
+ * "keep_layers" (0 / 1: keep the stream after every layer of a prompt). */
+UGB_API int32_t ugb_hybrid_set_option(ugb_hybrid *m, const char *key, int32_t value);
+/* Empties every sequence: position 0, zero convolution tails and recurrent
+ * state.  A recurrence cannot go back, so `pos` is 0 or the current position. */
+UGB_API int32_t ugb_hybrid_reset(ugb_hybrid *m, int32_t pos);
+UGB_API int32_t ugb_hybrid_position(const ugb_hybrid *m);
+UGB_API int32_t ugb_hybrid_decode(ugb_hybrid *m, const ugb_slice *tokens, int32_t n_steps);
+UGB_API int32_t ugb_hybrid_prefill(ugb_hybrid *m, const ugb_slice *tokens, int32_t t, int32_t all_logits);
+UGB_API int32_t ugb_hybrid_read(ugb_hybrid *m, int32_t what, void *host_dst, size_t len);
+/* Bytes of per-sequence state the engine keeps at `positions` cached positions. */
+UGB_API uint64_t ugb_hybrid_state_bytes(const ugb_hybrid *m, int32_t positions);
+/* Measurement aid: only the kernels of one kind of a decode step (t = 1) or of a
+ * prompt block of t positions, over all layers, replayed `iters` times from a
+ * CUDA graph; milliseconds per pass.  The model's state is scratch afterwards
+ * (reset it).  Kinds: UGB_HYBRID_K_*. */
+enum { UGB_HYBRID_K_ROWS = 0 /* residual, norms, average, fused convolution */, UGB_HYBRID_K_CONV = 1,
+       UGB_HYBRID_K_GRU_IN = 2, UGB_HYBRID_K_GRU = 3, UGB_HYBRID_K_LATENT_IN = 4, UGB_HYBRID_K_LATENT_ROWS = 5,
+       UGB_HYBRID_K_UQ = 6, UGB_HYBRID_K_ABSORB = 7 /* q W_uk, W_uv o, or the expansion of keys and values */,
+       UGB_HYBRID_K_ATTENTION = 8, UGB_HYBRID_K_OUT = 9, UGB_HYBRID_K_UP = 10, UGB_HYBRID_K_DOWN = 11,
+       UGB_HYBRID_K_HEAD = 12, UGB_HYBRID_K_ALL = 13 };
+UGB_API int32_t ugb_hybrid_time_kernel(ugb_hybrid *m, int32_t which, int32_t t, int32_t iters, float *ms_per_pass);
+
+/* The engine's mechanisms as operators on plain buffers (all F32 or, where
+ * named `T`, BF16 or F32 alike; widths multiples of 8). */
+/* out[b, i] = h[b, i] + sum_j w[j] h[b, i - (taps - 1) + j]; h, out T [b, t, width], w F32 [taps, width],
+ * tail T [b, taps - 1, width]: the rows before the block on entry, the last rows of it on return. */
+UGB_API int32_t ugb_causal_conv(ugb_device *dev, const ugb_slice *h, const ugb_slice *w, ugb_slice *tail,
+                                ugb_slice *out, size_t b, size_t t, size_t width, size_t taps);
+/* Minimal gated recurrent unit over a block: pre F32 [b, t, 3, width] (update gate, candidate and output gate
+ * before their activations), biases F32 [width], state F32 [b, width] in and out, out T [b, t, width]. */
+UGB_API int32_t ugb_min_gru(ugb_device *dev, const ugb_slice *pre, const ugb_slice *bias_z, const ugb_slice *bias_x,
+                            ugb_slice *state, ugb_slice *out, size_t b, size_t t, size_t width);
+/* Attention over cached latents, queries already in the latent space: q, out T [b, t, heads, rank], cache T
+ * [b, t_max, rank], gate F32 [b, t, heads] or null; query i attends positions 0 .. pos[0] + i (pos I32 [1], on the
+ * device); n_slices slices of the cache run as separate CTAs where the bf16 kernel takes the rank (64, 128, 256,
+ * 384, 512); cache rows of the last 32-position tile must hold finite values. */
+UGB_API int32_t ugb_latent_attend(ugb_device *dev, const ugb_slice *q, const ugb_slice *cache, const ugb_slice *gate,
+                                  const ugb_slice *pos, ugb_slice *out, size_t b, size_t t, size_t heads, size_t rank,
+                                  size_t t_max, float scale, int32_t n_slices);
+/* ugb_causal_attention for heads of 64 or 128 values (dq of queries and keys, dv of values), keys and values
+ * position-major: q BF16 [b, t, heads, dq], k / v BF16 [b, pos0 + t, heads, dq / dv], gate F32 [b, t, heads] or
+ * null, out BF16 [b, t, heads * dv]. */
+UGB_API int32_t ugb_causal_attention_wide(ugb_device *dev, const ugb_slice *q, const ugb_slice *k, const ugb_slice *v,
+                                          const ugb_slice *gate, ugb_slice *out, size_t b, size_t t, size_t pos0,
+                                          size_t heads, size_t dq, size_t dv, float scale);
+/* x += norm(y) * post_gain; bank[n] = x; x = sum_{j <= n} dwa[j] bank[j]; h = norm(x) * gain.  x, y F32 [rows, width],
+ * gains F32 [width], bank F32 [n + 1, rows, width] with the first n results on entry, dwa F32 [n + 1] (bank and dwa
+ * null: no average), h T [rows, width]. */
+UGB_API int32_t ugb_residual_update(ugb_device *dev, ugb_slice *x, const ugb_slice *y, const ugb_slice *post_gain,
+                                    ugb_slice *bank, const ugb_slice *dwa, size_t n, const ugb_slice *gain, ugb_slice *h,
+                                    size_t rows, size_t width, float eps);
+
 #ifdef __cplusplus
 }
 #endif

@@ -14,6 +14,7 @@ import numpy as np
 
 from ._lib import lib
 from .device import DType, UgError
+from .engine import EngineModel
 from .llama_config import Config, weight_names, weight_shape  # noqa: F401 (re-exported)
 
 
@@ -23,8 +24,10 @@ class _CConfig(C.Structure):
                [("rope_theta", C.c_float), ("rms_eps", C.c_float), ("rope_interleaved", C.c_int32)]
 
 
-class Model:
+class Model(EngineModel):
     """Model::new / Model::fwd for seq_len == 1 over ``batch`` independent sequences."""
+
+    PREFIX = "ugb_llama"
 
     def __init__(self, cfg, dev, batch, t_max, tp=None):
         """``tp = (rank, size)`` builds the tensor-parallel variant: this process keeps rank's share of
@@ -32,6 +35,7 @@ class Model:
         if not cfg.tie_word_embeddings:
             raise UgError(6, "tie_word_embeddings == false is not supported yet")   # model.rs:318
         self.cfg, self.dev, self.batch = cfg, dev, batch
+        self.width = cfg.hidden_size
         self.tp = tp
         cc = _CConfig(cfg.hidden_size, cfg.num_hidden_layers, cfg.num_attention_heads,
                       cfg.num_key_value_heads, cfg.head_dim(), cfg.intermediate_size, cfg.vocab_size,
@@ -87,85 +91,6 @@ class Model:
         self.dev._check(lib.ugb_llama_tp_connect(self._h, handles, 64, self.tp_size))
         self.dev.synchronize()
         group.barrier()          # nobody steps before everybody has mapped everybody
-
-    def load_weight(self, name, arr):
-        arr = np.ascontiguousarray(arr)
-        s = self.dev.slice_from_values(arr.ravel(), bf16=(arr.dtype == np.uint16))
-        self.dev._check(lib.ugb_llama_load_weight(self._h, name.encode(), s._h))
-        self.dev.synchronize()
-
-    def close(self):
-        h, self._h = self._h, None
-        if h:
-            lib.ugb_llama_destroy(h)
-
-    def __del__(self):
-        try:
-            self.close()
-        except Exception:
-            pass
-
-    def set_option(self, key, value):
-        self.dev._check(lib.ugb_llama_set_option(self._h, key.encode(), value))
-
-    def reset(self, pos=0):
-        self.dev._check(lib.ugb_llama_reset(self._h, pos))
-
-    @property
-    def position(self):
-        return lib.ugb_llama_position(self._h)
-
-    def fwd(self, tokens):
-        """Model::fwd on explicit token ids, asynchronous: int32 [batch] or [batch, 1] is one
-        decode step; [batch, t] with t > 1 appends t positions (causal prefill) and keeps the
-        logits of every position for :meth:`prefill_logits`."""
-        tokens = np.ascontiguousarray(tokens, dtype=np.int32)
-        if tokens.ndim == 2 and tokens.shape[1] > 1:
-            return self.prefill(tokens, all_logits=True)
-        s = self.dev.slice_from_values(tokens.reshape(-1))
-        self.dev._check(lib.ugb_llama_decode(self._h, s._h, 1))
-
-    def prefill(self, tokens, all_logits=False):
-        """Appends ``tokens`` (int32 [batch, t], host array or device Slice of batch*t ids) to
-        every sequence; :meth:`logits` / :meth:`next_tokens` then refer to the last position."""
-        if isinstance(tokens, np.ndarray) or not hasattr(tokens, "_h"):
-            tokens = np.ascontiguousarray(tokens, dtype=np.int32)
-            if tokens.ndim != 2 or tokens.shape[0] != self.batch:
-                raise UgError(4, f"prefill tokens must be [batch={self.batch}, t], got {tokens.shape}")
-            t = tokens.shape[1]
-            s = self.dev.slice_from_values(tokens.reshape(-1))
-        else:
-            s, t = tokens, tokens.len // self.batch
-        self.dev._check(lib.ugb_llama_prefill(self._h, s._h, t, int(all_logits)))
-        self._prefill_t = t if all_logits else getattr(self, "_prefill_t", 0)
-
-    def prefill_logits(self):
-        """f32 [batch, t, vocab] of the last ``all_logits`` prefill (what Model::fwd returns)."""
-        t = getattr(self, "_prefill_t", 0)
-        out = np.empty((self.batch, t, self.vocab_local), np.float32)
-        self.dev._check(lib.ugb_llama_read(self._h, 3, out.ctypes.data, out.size))
-        return out
-
-    def decode(self, n_steps):
-        """Greedy decoding: each step feeds the previous step's argmax; asynchronous."""
-        self.dev._check(lib.ugb_llama_decode(self._h, None, n_steps))
-
-    def logits(self):
-        """f32 [batch, vocab]; a tensor-parallel rank returns its columns
-        [vocab_offset, vocab_offset + vocab_local)."""
-        out = np.empty((self.batch, self.vocab_local), np.float32)
-        self.dev._check(lib.ugb_llama_read(self._h, 0, out.ctypes.data, out.size))
-        return out
-
-    def next_tokens(self):
-        out = np.empty(self.batch, np.int32)
-        self.dev._check(lib.ugb_llama_read(self._h, 1, out.ctypes.data, out.size))
-        return out
-
-    def hidden(self):
-        out = np.empty((self.batch, self.cfg.hidden_size), np.float32)
-        self.dev._check(lib.ugb_llama_read(self._h, 2, out.ctypes.data, out.size))
-        return out
 
     def kv_cache(self, layer, which):
         """bf16 bit patterns [batch, n_kv_heads, kv_positions, head_dim] of K (0) or V (1)."""

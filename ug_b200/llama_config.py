@@ -29,7 +29,10 @@ class Config:
         """A Hugging Face ``config.json`` (what ug-llama deserialises into Config, main.rs:105-122)."""
         import json
         with open(path) as f:
-            d = json.load(f)
+            return Config.from_dict(json.load(f))
+
+    @staticmethod
+    def from_dict(d):
         keys = ("hidden_size", "intermediate_size", "max_position_embeddings", "num_attention_heads",
                 "num_key_value_heads", "num_hidden_layers", "vocab_size", "rms_norm_eps", "rope_theta",
                 "rope_interleaved", "tie_word_embeddings")
