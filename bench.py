@@ -1057,11 +1057,151 @@ class PrefillWorkload(DecodeWorkload):
                 "l2": "inputs larger than L2 (2.07 GB of weights read per step vs 126 MB L2)"}
 
 
+class KabidraWorkload:
+    """The Kabidra decoder at the layer sizes of the 1.1B Llama benchmark model, beside that model: decode steps of 64
+    and 8 sequences at 2048 cached positions, prompts of 8 x 512 and 1 x 4096 tokens, every kind of kernel of a pass
+    timed alone (graph replays of that kind over all layers).  Random weights, one set per tensor shape."""
+    unit = "tokens/s"
+    dtype = "bf16"
+    metric = "tokens/s, Kabidra decode (64 sequences, 2048 cached positions)"
+    name = ("Kabidra, width 2048, 22 layers (every fourth latent attention with 16 heads of 128 over a latent of 512, the "
+            "others minimal GRUs of 2048 channels), feed-forward 5632, vocab 32000, bf16; beside the Llama-1.1B shape")
+    DECODE = ((64, 2048), (8, 2048))
+    PREFILL = ((8, 512), (1, 4096))
+
+    def __init__(self, rank=0):
+        from ug_b200.kabidra_config import Config
+        self.cfg = Config.like_llama_1b()
+
+    def setup(self, dev):
+        from ug_b200 import synth
+        from ug_b200.kabidra_config import weight_shapes
+        shapes = weight_shapes(self.cfg)
+        first = {}
+        for n, shape in shapes.items():
+            first.setdefault((n.split(".", 1)[-1], shape), n)
+        from concurrent.futures import ThreadPoolExecutor
+        with ThreadPoolExecutor(max_workers=min(16, os.cpu_count() or 1)) as ex:
+            made = dict(zip(first, ex.map(lambda n: synth.kabidra_tensor(300, n, shapes[n]), first.values())))
+        self.weights = {n: made[(n.split(".", 1)[-1], shape)] for n, shape in shapes.items()}
+        self.counts = {"attention": sum(l.type == "latent_attention" for l in self.cfg.layers)}
+        self.counts["gru"] = len(self.cfg.layers) - self.counts["attention"]
+
+    def work(self, rows, batch, t, depth):
+        """Per kind of kernel: (launches, bytes moved at least once, flops) of one pass over all layers."""
+        c, na, ng = self.cfg, self.counts["attention"], self.counts["gru"]
+        L, w, decode = len(c.layers), c.width, t == 1
+        a = next(l.mixer for l in c.layers if l.type == "latent_attention")
+        u = next(l.mixer["width"] for l in c.layers if l.type == "mingru")
+        ff, H, d, v, q, r = c.layers[0].ff, a["heads"], a["dim"], a["vdim"], a["q_rank"], a["kv_rank"]
+        mm = lambda n, k, out: (2 * n * k + rows * (2 * k + out * n), 2 * rows * n * k)      # weights + rows in + rows out
+        f = lambda n, x: (n, n * x[0], n * x[1])
+        k = {"gru_in": f(ng, mm(3 * u, w, 4)), "gru": (ng, ng * rows * (12 * u + 2 * u), 0),
+             "latent_in": f(na, mm(q + r + H, w, 4)), "uq": f(na, mm(H * d, q, 2)),
+             "up": f(L, mm(ff, w, 2)), "down": f(L, mm(w, ff, 4)),
+             "out": (L, ng * mm(w, u, 4)[0] + na * mm(w, H * v, 4)[0], ng * mm(w, u, 4)[1] + na * mm(w, H * v, 4)[1]),
+             # residual in and out, product in, h out; the bank: one row written and i + 1 read in layer i
+             "rows": (2 * L + 1, rows * w * ((2 * L + 1) * 14 + 4 * (L + L * (L + 1) // 2)), 0),
+             "latent_rows": (na, na * rows * (4 * (q + r + H) + 2 * (q + r) + 4 * H), 0)}
+        if decode:
+            k["absorb"] = (2 * na, na * (2 * H * (d + v) * r + rows * H * (2 * d + 4 * r + 2 * v)), na * 2 * rows * H * r * (d + v))
+            k["attention"] = (na, na * batch * depth * r * 2, na * batch * depth * H * 4 * r)
+        else:
+            pairs = batch * (depth * t + t * (t + 1) // 2)
+            k["conv"] = (2 * L, 2 * L * rows * w * 4, 0)
+            k["absorb"] = (2 * na, na * (2 * H * (d + v) * r + batch * (depth + t) * (2 * r + 2 * H * (d + v))), na * 2 * batch * (depth + t) * H * r * (d + v))
+            k["attention"] = (na, na * rows * H * (4 * d + 4 * v), na * pairs * H * 2 * (d + v))
+        return k
+
+    def kernels(self, model, rows, batch, t, depth, peaks):
+        out = {}
+        for name, (n, nbytes, flops) in self.work(rows, batch, t, depth).items():
+            ms = model.time_kernel(name, t, 20)
+            t_hbm, t_tc = nbytes / peaks["hbm"] / 1e6, flops / peaks["bf16"] / 1e9
+            out[name] = {"ms": round(ms, 4), "launches": n, "us_per_launch": round(1e3 * ms / n, 2),
+                         "bound": "hbm" if t_hbm >= t_tc else "tensor", "frac": round(max(t_hbm, t_tc) / ms, 3)}
+        return out
+
+    def timed(self, dev, f, warmup, steps):
+        for _ in range(warmup):
+            f()
+        dev.synchronize()
+        dev.timer_begin()
+        for _ in range(steps):
+            f()
+        dev.timer_end()
+        return dev.timer_elapsed_ms() / steps
+
+    def record(self, dev, warmup, steps, peaks):
+        from ug_b200 import kabidra, llama, synth
+        from ug_b200.llama_config import Config as LlamaConfig
+        lc = LlamaConfig.llama_1b()
+        lw = _weights(lc)
+        sampler = ClockSampler(0)
+        sampler.start()
+        rec = {"workload": self.name, "metric": self.metric, "unit": self.unit, "dtype": self.dtype, "steps": steps,
+               "data": "synthetic (random weights and tokens)", "peak_source": peaks["source"], "decode": {}, "prefill": {}}
+        for batch, depth in self.DECODE:
+            t_max = depth + warmup + steps + 64
+            prompts = synth.tokens(8, (batch, depth), self.cfg.vocab)
+            r = {}
+            for key, make in (("kabidra", lambda: kabidra.Model.new(self.cfg, self.weights, dev, batch, t_max)),
+                              ("llama", lambda: llama.Model.new(lc, lw, dev, batch, t_max))):
+                m = make()
+                m.prefill(prompts)
+                ms = self.timed(dev, lambda: m.decode(1), max(warmup, 3), steps)
+                r[key] = {"tokens_per_s": round(1e3 * batch / ms, 1), "ms_per_step": round(ms, 4)}
+                at = m.position
+                if key == "kabidra":
+                    r[key]["state_bytes_per_sequence"] = m.state_bytes(at)
+                    r[key]["kernels"] = self.kernels(m, batch, batch, 1, at, peaks)
+                    r[key]["kernels"]["head"] = {"ms": round(m.time_kernel("head"), 4), "launches": 1}
+                else:
+                    kv = 2 * lc.num_hidden_layers * 2 * lc.num_key_value_heads * lc.head_dim() * at * batch
+                    h, ffn, n = lc.hidden_size, lc.intermediate_size, lc.num_hidden_layers
+                    kvd = lc.num_key_value_heads * lc.head_dim()
+                    nb = {"qkv_gemm": 2 * h * (h + 2 * kvd) * n, "decode_attention": kv, "o_gemm": 2 * h * h * n,
+                          "gate_up_gemm": 4 * h * ffn * n, "down_gemm": 2 * h * ffn * n, "lm_head_gemm": 2 * h * lc.vocab_size}
+                    r[key]["kernels"] = {}
+                    for name in m.KERNELS:
+                        kms, cnt = m.time_kernel(name, 20), 1 if name == "lm_head_gemm" else n
+                        r[key]["kernels"][name] = {"ms": round(kms, 4), "launches": cnt, "us_per_launch": round(1e3 * kms / cnt, 2),
+                                                   "bound": "hbm", "frac": round(nb[name] / peaks["hbm"] / 1e6 / kms, 3)}
+                m.close()
+            rec["decode"]["%d x %d" % (batch, depth)] = r
+        for batch, t in self.PREFILL:
+            prompts = dev.slice_from_values(synth.tokens(9, (batch, t), self.cfg.vocab).reshape(-1))
+            r = {}
+            for key, make in (("kabidra", lambda: kabidra.Model.new(self.cfg, self.weights, dev, batch, t + 32)),
+                              ("llama", lambda: llama.Model.new(lc, lw, dev, batch, t))):
+                m = make()
+
+                def step():
+                    m.reset()
+                    m.prefill(prompts)
+                ms = self.timed(dev, step, max(warmup, 3), max(3, steps // 5))
+                r[key] = {"tokens_per_s": round(1e3 * batch * t / ms, 1), "ms_per_step": round(ms, 4)}
+                if key == "kabidra":
+                    m.reset()
+                    m.decode(1)
+                    m.reset()
+                    r[key]["kernels"] = self.kernels(m, batch * t, batch, t, 0, peaks)
+                m.close()
+            rec["prefill"]["%d x %d" % (batch, t)] = r
+        rec["clocks"] = sampler.stop()
+        rec["value"] = rec["decode"]["64 x 2048"]["kabidra"]["tokens_per_s"]
+        return rec
+
+    def config(self):
+        return {"workload": self.name}
+
+
 WORKLOADS = {"rms_silu": RmsSiluWorkload, "softmax": SoftmaxWorkload, "softmax_c1": SoftmaxC1Workload,
              "gemm": GemmWorkload, "decode": DecodeWorkload, "prefill": PrefillWorkload,
              "graph_softmax": lambda r: GraphRowWorkload("softmax"), "graph_rms_norm": lambda r: GraphRowWorkload("rms_norm"),
              "gemm_f32": lambda r: F32MatmulWorkload("gemm_f32"), "gemv_f32": lambda r: F32MatmulWorkload("gemv_f32"),
-             "graph_decode": GraphDecodeWorkload, "llama_ops": LlamaOpsWorkload}
+             "graph_decode": GraphDecodeWorkload, "llama_ops": LlamaOpsWorkload,
+             "kabidra": KabidraWorkload}
 DEFAULT_WORKLOAD = "decode"
 
 # DRAM traffic of the decode step's kernels, from ncu captures of single launches (dram__bytes_read.sum +

@@ -276,3 +276,27 @@ class Device:
         """Fused grouped-query attention for one new position per sequence (model.rs:231-245)."""
         self._check(lib.ugb_decode_attention(self._h, q._h, k._h, v._h, pos._h, out._h, b, n_heads, n_kv,
                                              t_max, n_slices))
+
+    # ---- mechanisms of the layer-list engine, each alone ---------------------
+    def causal_conv(self, h, w, tail, out, b, t, width, taps):
+        """h + depthwise causal convolution over time; ``tail`` (the rows before the block) is moved on."""
+        self._check(lib.ugb_causal_conv(self._h, h._h, w._h, tail._h, out._h, b, t, width, taps))
+
+    def min_gru(self, pre, bias_z, bias_x, state, out, b, t, width):
+        """Minimal gated recurrent unit over a block of t positions; ``state`` is moved on."""
+        self._check(lib.ugb_min_gru(self._h, pre._h, bias_z._h, bias_x._h, state._h, out._h, b, t, width))
+
+    def latent_attend(self, q, cache, gate, pos, out, b, t, heads, rank, t_max, scale, n_slices=1):
+        """Attention of latent-space queries over a cache of latents shared by all heads."""
+        self._check(lib.ugb_latent_attend(self._h, q._h, cache._h, gate._h if gate else None, pos._h, out._h, b, t, heads,
+                                          rank, t_max, scale, n_slices))
+
+    def causal_attention_wide(self, q, k, v, gate, out, b, t, pos0, heads, dq, dv, scale):
+        """Causal attention of a block, heads of 64 or 128 values, keys and values position-major."""
+        self._check(lib.ugb_causal_attention_wide(self._h, q._h, k._h, v._h, gate._h if gate else None, out._h, b, t, pos0,
+                                                  heads, dq, dv, scale))
+
+    def residual_update(self, x, y, post_gain, bank, dwa, n, gain, h, rows, width, eps):
+        """x += norm(y) post_gain; with a bank of n earlier results, x becomes their weighted sum; h = norm(x) gain."""
+        self._check(lib.ugb_residual_update(self._h, x._h, y._h, post_gain._h, bank._h if bank else None,
+                                            dwa._h if dwa else None, n, gain._h, h._h, rows, width, eps))

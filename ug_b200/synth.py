@@ -73,6 +73,43 @@ def llama_weights(cfg, seed_base=100):
         return dict(ex.map(one, enumerate(weight_names(cfg))))
 
 
+def kabidra_tensor(seed, name, shape):
+    """One random tensor of a Kabidra model as bf16 bit patterns.  Matrices ~ N(0, 1 / columns), so that every sublayer's
+    output has the size of its input; norm weights, biases and convolution taps are spread widely enough that a model
+    without them computes something else; the depth average keeps most of the newest result."""
+    tail = name.split(".", 1)[-1]
+    x = normal(seed, shape)
+    if tail == "dwa":
+        x = np.float32(0.3) * x
+        x[-1] += np.float32(0.8)
+    elif tail in ("mix.dq.norm", "mix.dkv.norm"):
+        x = np.float32(1.0) + np.float32(0.2) * x
+    elif tail in ("canon1", "canon2"):
+        x = np.float32(0.35) * x
+    elif tail == "mix.z.b":
+        x = x - np.float32(1.5)            # recurrent channels that forget slowly
+    elif len(shape) == 1 and not tail.endswith(".b"):
+        x = np.float32(0.2) * x
+    elif len(shape) == 2 and name != "embed":
+        x = x * np.float32(shape[1] ** -0.5)
+    return to_bf16_bits(x)
+
+
+def kabidra_weights(cfg, seed_base=300):
+    """All tensors of a Kabidra model, name -> uint16 array; seed = seed_base + index of the tensor in load order."""
+    import os
+    from concurrent.futures import ThreadPoolExecutor
+
+    from .kabidra_config import weight_shapes
+
+    def one(item):
+        i, (name, shape) = item
+        return name, kabidra_tensor(seed_base + i, name, shape)
+
+    with ThreadPoolExecutor(max_workers=min(16, os.cpu_count() or 1)) as ex:
+        return dict(ex.map(one, enumerate(weight_shapes(cfg).items())))
+
+
 def llama_weights_f32(weights):
-    """The f32 view of bf16 weights that load_with_cast BF16 -> F32 produces."""
+    """The f32 view of bf16 weights that load_with_cast BF16 -> F32 produces (any model's)."""
     return {k: (bf16_bits_to_f32(v) if v.dtype == np.uint16 else v) for k, v in weights.items()}
