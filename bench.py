@@ -1096,13 +1096,19 @@ class KabidraWorkload:
         ff, H, d, v, q, r = c.layers[0].ff, a["heads"], a["dim"], a["vdim"], a["q_rank"], a["kv_rank"]
         mm = lambda n, k, out: (2 * n * k + rows * (2 * k + out * n), 2 * rows * n * k)      # weights + rows in + rows out
         f = lambda n, x: (n, n * x[0], n * x[1])
-        k = {"gru_in": f(ng, mm(3 * u, w, 4)), "gru": (ng, ng * rows * (12 * u + 2 * u), 0),
-             "latent_in": f(na, mm(q + r + H, w, 4)), "uq": f(na, mm(H * d, q, 2)),
-             "up": f(L, mm(ff, w, 2)), "down": f(L, mm(w, ff, 4)),
-             "out": (L, ng * mm(w, u, 4)[0] + na * mm(w, H * v, 4)[0], ng * mm(w, u, 4)[1] + na * mm(w, H * v, 4)[1]),
-             # residual in and out, product in, h out; the bank: one row written and i + 1 read in layer i
-             "rows": (2 * L + 1, rows * w * ((2 * L + 1) * 14 + 4 * (L + L * (L + 1) // 2)), 0),
-             "latent_rows": (na, na * rows * (4 * (q + r + H) + 2 * (q + r) + 4 * H), 0)}
+        # a step's split products reach their consumer as f32 partials, a block's recurrent projections as bf16
+        parts = {"gru_in": 3, "latent_in": 8, "out": 8, "down": 8} if decode and batch <= 64 else {}
+        pn = lambda name: parts.get(name, 1)
+        pre = 4 * pn("gru_in") if decode else 2
+        k = {"gru_in": f(ng, mm(3 * u, w, pre)), "gru": (ng, ng * rows * u * (3 * pre + 2 + (8 if decode else 0)), 0),
+             "latent_in": f(na, mm(q + r + H, w, 4 * pn("latent_in"))), "uq": f(na, mm(H * d, q, 2)),
+             "up": f(L, mm(ff, w, 2)), "down": f(L, mm(w, ff, 4 * pn("down"))),
+             "out": (L, ng * mm(w, u, 4 * pn("out"))[0] + na * mm(w, H * v, 4 * pn("out"))[0], ng * mm(w, u, 4)[1] + na * mm(w, H * v, 4)[1]),
+             # residual in and out, product partials in, h out, in a step the convolution tail in and out; the bank: one
+             # row written and i + 1 read in layer i
+             "rows": (2 * L + 1, rows * w * ((2 * L + 1) * (10 + (4 * (c.taps - 1) if decode else 0)) +
+                                             L * 4 * (pn("out") + pn("down")) + 4 * (L + L * (L + 1) // 2)), 0),
+             "latent_rows": (na, na * rows * (4 * pn("latent_in") * (q + r + H) + 2 * (q + r) + 4 * H), 0)}
         if decode:
             k["absorb"] = (2 * na, na * (2 * H * (d + v) * r + rows * H * (2 * d + 4 * r + 2 * v)), na * 2 * rows * H * r * (d + v))
             k["attention"] = (na, na * batch * depth * r * 2, na * batch * depth * H * 4 * r)

@@ -620,7 +620,7 @@ UGB_API int32_t ugb_hybrid_time_kernel(ugb_hybrid *m, int32_t which, int32_t t, 
  * tail T [b, taps - 1, width]: the rows before the block on entry, the last rows of it on return. */
 UGB_API int32_t ugb_causal_conv(ugb_device *dev, const ugb_slice *h, const ugb_slice *w, ugb_slice *tail,
                                 ugb_slice *out, size_t b, size_t t, size_t width, size_t taps);
-/* Minimal gated recurrent unit over a block: pre F32 [b, t, 3, width] (update gate, candidate and output gate
+/* Minimal gated recurrent unit over a block: pre F32 (or BF16, with t > 1 and a BF16 result) [b, t, 3, width] (update gate, candidate and output gate
  * before their activations), biases F32 [width], state F32 [b, width] in and out, out T [b, t, width]. */
 UGB_API int32_t ugb_min_gru(ugb_device *dev, const ugb_slice *pre, const ugb_slice *bias_z, const ugb_slice *bias_x,
                             ugb_slice *state, ugb_slice *out, size_t b, size_t t, size_t width);

@@ -88,6 +88,27 @@ def test_min_gru(dev, bf16, width, batch, cuts):
         assert close(st.to_vec().reshape(batch, width).astype(np.float64), S[:, at - 1], 2e-5)
 
 
+@pytest.mark.parametrize("width,batch,cuts", [(8, 2, (2, 3, 64, 65)), (72, 1, (511, 512, 513)), (2048, 2, (700,))])
+def test_min_gru_on_bf16_projections(dev, width, batch, cuts):
+    """A block whose pre-activations were rounded to bf16: the recurrence itself stays in 32 bits."""
+    B, t = Buf(dev, True), sum(cuts)
+    pre = synth.normal(3, (batch, t, 3, width), 1.5)
+    pre[:, :, 0] -= 3.0
+    bz, bx = synth.normal(4, (width,)), synth.normal(5, (width,))
+    st, zs, xs, at = B.f32(np.zeros((batch, width))), B.f32(bz), B.f32(bx), 0
+    S0 = np.zeros((batch, width))
+    for n in cuts:
+        ps, pv = B.act(pre[:, at:at + n])
+        out = B.out(batch * n * width)
+        dev.min_gru(ps, zs, xs, st, out, batch, n, width)
+        z, c = K.sigmoid(pv[:, :, 0] + bz), K.gru_candidate(pv[:, :, 1] + bx)
+        S = np.stack([K.min_gru(z[b], c[b], S0[b])[0] for b in range(batch)])
+        S0 = S[:, -1]
+        assert close(B.read(out, (batch, n, width)), S * K.silu(pv[:, :, 2]), B.tol)
+        assert close(st.to_vec().reshape(batch, width).astype(np.float64), S0, 2e-5)
+        at += n
+
+
 def test_min_gru_remembers_the_first_token(dev):
     """With the gate shut after position 0 the state is the first candidate for as long as anyone looks."""
     B, n, width = Buf(dev, False), 3000, 40

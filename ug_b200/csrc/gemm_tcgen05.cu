@@ -77,6 +77,7 @@ struct Params {
   int stage_tx;           // bytes one pipeline stage receives (A box + B box)
   int n_fast;             // tile order: 1 = n-tiles vary fastest (a wave re-reads B, the smaller operand)
   int b_static;           // 1: no kernel on the stream writes B (weights): it may be fetched before ugb_pdl_wait
+  int late_trigger;       // see ugb_tc_gemm_args
   int stages;             // depth of the shared-memory ring in use (2 .. Cfg::STAGES)
   int f16;                // operands and 16-bit output are IEEE f16 (0: bf16)
   unsigned long long *prof;   // measurement aid (or null): %globaltimer stamps of CTA 0, see UGB_TC_PROF_* in the header
@@ -204,7 +205,7 @@ tc_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
   if constexpr (PAIR) cluster_sync_all();    // both CTAs' barriers exist before either signals the other's
   tcgen05_fence_after();
   const uint32_t tmem_base = *tmem_slot;
-  if (threadIdx.x == 0) ugb_pdl_trigger();   // the next kernel on the stream may begin its preamble
+  if (threadIdx.x == 0 && !p.late_trigger) ugb_pdl_trigger();   // the next kernel on the stream may begin its preamble
 
   if (warp == 0) {
     // ------------------------------------------------------ TMA producer --
@@ -235,6 +236,7 @@ tc_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
           }
         }
         ugb_pdl_wait();
+        if (p.late_trigger) ugb_pdl_trigger();
         UGB_TC_STAMP(UGB_TC_PROF_DEP);
         for (int i = 0; i < pre; ++i)
           load3(smem_u32(smem + i * STAGE_BYTES), &tmA, PAIR ? mapa_u32(smem_u32(&full[i]), 0) : smem_u32(&full[i]),
@@ -684,6 +686,7 @@ int32_t launch_tc(ugb_device *dev, TcState *st, const ugb_tc_gemm_args &g, size_
   p.epi = g.epi;
   p.b_static = g.b_static ? 1 : 0;
   p.f16 = g.f16 ? 1 : 0;
+  p.late_trigger = g.late_trigger ? 1 : 0;
   p.prof = g.prof;
   p.pair_k = 0;
   if (g.pair_k) {

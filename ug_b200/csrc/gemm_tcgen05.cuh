@@ -46,6 +46,9 @@ struct ugb_tc_gemm_args {
   int bn;               // tile width: 64, 128, 256 (80, 96, 160 too when m <= 64 and b_is_nk), or 0 = choose from m
   bool b_static;        // no kernel on the stream writes b (weights): fetch it before waiting for the predecessor
   bool pdl;             // launch with programmatic stream serialization (see ugb_launch)
+  bool late_trigger = false;   // let the next kernel start only once the wait for the preceding one has returned: a kernel
+                               // of a stream whose kernels all do so may read what the kernels before its predecessor wrote
+                               // ahead of its own wait
   int smem_kib = 0;     // cap on the shared memory of a CTA (ring depth follows); 0 = as deep as fits in 220 KiB
   bool f16 = false;     // operands (and the UGB_EPI_BF16 output) are IEEE f16 instead of bf16: same instruction, other format field
   bool pair_k = false;  // m <= 64, UGB_EPI_SILU_MUL_BF16 or UGB_EPI_RELU2_BF16: two CTAs (a thread-block cluster) per tile, each over half of k; the

@@ -83,8 +83,6 @@ struct ugb_hybrid : ugb_engine {
   size_t tail_bytes = 0;
   Work dec, pf;
   void *kx = nullptr, *vx = nullptr;                       // expanded keys / values of one layer
-  float *att_o = nullptr, *att_ml = nullptr;
-  unsigned *att_cnt = nullptr;
   int att_splits_opt = 0, absorb_max = 16, keep_layers = 0;
   float *layer_out = nullptr;
   size_t layer_cap = 0;
@@ -136,7 +134,7 @@ int32_t matmul(ugb_hybrid *m, const Mat &x) {
   g.a_ld = x.a_ld == x.k ? 0 : (long long)x.a_ld; g.c_ld = x.c_ld == x.n ? 0 : (long long)x.c_ld;
   g.b_is_nk = x.nk;
   g.epi = x.relu2 ? UGB_EPI_RELU2_BF16 : (x.f32_out ? UGB_EPI_F32 : UGB_EPI_BF16);
-  g.splits = x.splits; g.bn = x.bn; g.b_static = true; g.pdl = m->pdl != 0;
+  g.splits = x.splits; g.bn = x.bn; g.b_static = true; g.pdl = m->pdl != 0; g.late_trigger = true;
   g.smem_kib = x.m <= 64 ? 144 : 0;
   if (x.relu2 && x.m <= 64) {
     // the two k halves of a tile on a pair of CTAs, with the narrowest tile that fits the SMs
@@ -161,47 +159,59 @@ int32_t matmul(ugb_hybrid *m, const Mat &x) {
 struct Tiling { int bn, splits; };
 Tiling tiling(const ugb_hybrid *m, size_t n, size_t k) {
   if (m->f32 || m->batch > 64) return {0, 1};
+  // A CTA's time goes with its k blocks and hardly with its tile width (an MMA of 64 rows costs the same up to 160
+  // columns), so: the fewest k blocks per CTA over widths and splits that fit one wave, then the fewest partials,
+  // then the narrowest tile.
   const int sms = m->dev->sm_count, kb = (int)((k + 63) / 64);
-  const int bn = (n + 63) / 64 > (size_t)sms ? 128 : 64;
-  const int tiles = (int)((n + bn - 1) / bn);
-  const int s = std::max(1, std::min({8, sms / tiles, kb / 2}));
-  return {bn, ugb_tc_gemm_effective_splits(k, s)};
+  Tiling best{128, 1};
+  int best_kb = kb + 1;
+  for (int s = 1; s <= std::min(8, kb); ++s)
+    for (int bn : {64, 80, 96, 128, 160}) {
+      const int tiles = (int)((n + bn - 1) / bn), per = (kb + s - 1) / s;
+      if (tiles * s > sms || per >= best_kb) continue;
+      best = {bn, s};
+      best_kb = per;
+    }
+  if (best_kb > kb) return {256, 1};           // more tiles than SMs whatever the width
+  return {best.bn, ugb_tc_gemm_effective_splits(k, best.splits)};
 }
 constexpr int MAX_SPLITS = 8;
 
-template <typename T> int32_t launch_rows(ugb_hybrid *m, RowArgs<T> &a, int rows) {
+template <typename T> int32_t launch_rows(ugb_hybrid *m, RowArgs<T> &a, int rows, bool early) {
   if (!m->on(UGB_HYBRID_K_ROWS)) return UGB_OK;
+  a.early = early ? 1 : 0;
   a.ld = m->wl; a.inv_width = 1.0f / (float)m->cfg.width; a.eps = m->cfg.eps; a.status = m->dev->status_dev;
   const int nvec = m->wl / 4;
   cudaStream_t st = m->dev->stream;
   const bool pdl = m->pdl != 0;
-  cudaError_t e;
-  if (nvec <= 256) e = ugb_launch(row_update_kernel<T, 1>, dim3(rows), dim3(256), 0, st, pdl, a);
-  else if (nvec <= 512) e = ugb_launch(row_update_kernel<T, 2>, dim3(rows), dim3(256), 0, st, pdl, a);
-  else if (nvec <= 1024) e = ugb_launch(row_update_kernel<T, 4>, dim3(rows), dim3(256), 0, st, pdl, a);
-  else e = ugb_launch(row_update_kernel<T, 8>, dim3(rows), dim3(256), 0, st, pdl, a);
+  const bool step = rows <= m->dev->sm_count;
+  auto *k = nvec <= 256    ? (step ? row_update_kernel<T, 1, true> : row_update_kernel<T, 1, false>)
+            : nvec <= 512  ? (step ? row_update_kernel<T, 2, true> : row_update_kernel<T, 2, false>)
+            : nvec <= 1024 ? (step ? row_update_kernel<T, 4, true> : row_update_kernel<T, 4, false>)
+                           : row_update_kernel<T, 8, false>;
+  const cudaError_t e = ugb_launch(k, dim3(rows), dim3(256), 0, st, pdl, a);
   if (e != cudaSuccess) return ugb_fail(m->dev, UGB_ERR_CUDA, "launch of row_update_kernel failed: %s", cudaGetErrorString(e));
   return ugb_after_launch(m->dev, "row_update_kernel");
 }
 
 template <typename T>
 int32_t launch_conv(ugb_device *dev, const T *h, const float *w, const T *tail_in, T *tail_out, T *out, int b, int t, int taps, int ld) {
-  const dim3 grid((unsigned)((t + CONV_STRIP - 1) / CONV_STRIP), (unsigned)((ld / 4 + 255) / 256), (unsigned)b);
-  causal_conv_kernel<T><<<grid, 256, 0, dev->stream>>>(h, w, tail_in, tail_out, out, t, taps, ld);
+  const dim3 grid((unsigned)((t + CONV_STRIP - 1) / CONV_STRIP), (unsigned)((ld / 8 + 127) / 128), (unsigned)b);
+  auto *k = causal_conv_kernel<T, 0>;
+  if (taps == 2) k = causal_conv_kernel<T, 2>;
+  else if (taps == 3) k = causal_conv_kernel<T, 3>;
+  else if (taps == 4) k = causal_conv_kernel<T, 4>;
+  k<<<grid, 128, 0, dev->stream>>>(h, w, tail_in, tail_out, out, t, taps, ld);
   return ugb_after_launch(dev, "causal_conv_kernel");
 }
 
-// CTAs of a scan cluster: enough pieces of time to fill the SMs twice, no more than the block has
-int scan_cluster(const ugb_device *dev, int b, int t, int ld) {
-  const int pieces = (t + SCAN_BLOCK - 1) / SCAN_BLOCK, columns = b * ((ld + 31) / 32);
+template <typename TI, typename T>
+int32_t launch_scan(ugb_device *dev, const TI *pre, const float *bz, const float *bu, float *state, T *out, int b, int t, int ld) {
+  // CTAs of a cluster: enough pieces of time to fill the SMs twice, no more than the block has
+  const int columns = (ld + Scan<TI>::COLUMNS - 1) / Scan<TI>::COLUMNS;
   int c = 1;
-  while (c < 8 && c * 2 <= pieces && c * columns < 2 * dev->sm_count) c *= 2;
-  return c;
-}
-template <typename T>
-int32_t launch_scan(ugb_device *dev, const float *pre, const float *bz, const float *bu, float *state, T *out, int b, int t, int ld) {
-  const int c = scan_cluster(dev, b, t, ld);
-  cudaError_t e = ugb_launch_cluster(min_gru_scan_kernel<float, T>, dim3((unsigned)c, (unsigned)((ld + 31) / 32), (unsigned)b),
+  while (c < 8 && c * Scan<TI>::BLOCK < t && 2 * c * b * columns <= 2 * dev->sm_count) c *= 2;
+  cudaError_t e = ugb_launch_cluster(min_gru_scan_kernel<TI, T>, dim3((unsigned)c, (unsigned)columns, (unsigned)b),
                                      dim3(SCAN_WARPS * 32), 0, dev->stream, false, c, pre, bz, bu, state, out, t, ld);
   if (e != cudaSuccess) return ugb_fail(dev, UGB_ERR_CUDA, "launch of min_gru_scan_kernel failed: %s", cudaGetErrorString(e));
   return ugb_after_launch(dev, "min_gru_scan_kernel");
@@ -214,6 +224,9 @@ int32_t run_layers(ugb_hybrid *m, Work &w, const int *tok, int t_block, int off,
   ugb_device *dev = m->dev;
   cudaStream_t st = dev->stream;
   const bool pdl = m->pdl != 0;
+  // In a bf16 decode step every kernel lets its successor start only after its own wait, and at least two kernels lie
+  // between one row kernel and the next: what earlier row kernels wrote is complete when a row kernel starts.
+  const bool early = decode && pdl && !m->f32;
   const int B = m->batch, rows = B * t, wl = m->wl, taps = m->cfg.conv_taps;
   const size_t bank_stride = (size_t)w.rows * wl, n_tail = taps > 1 ? (size_t)B * (taps - 1) * wl : 0;
   int32_t rc;
@@ -242,7 +255,7 @@ int32_t run_layers(ugb_hybrid *m, Work &w, const int *tok, int t_block, int off,
     a.gain = m->layers.empty() ? m->final_gain : m->layers[0].norm1;
     a.h = (T *)w.h;
     if (!m->layers.empty()) fuse_conv(a, m->layers[0].conv1, 0, 0);
-    if ((rc = launch_rows<T>(m, a, rows))) return rc;
+    if ((rc = launch_rows<T>(m, a, rows, early))) return rc;
   }
   const int n_layers = (int)m->layers.size();
   for (int i = 0; i < n_layers; ++i) {
@@ -255,6 +268,7 @@ int32_t run_layers(ugb_hybrid *m, Work &w, const int *tok, int t_block, int off,
       if (m->on(UGB_HYBRID_K_GRU_IN)) {
         Mat g{w.pre, in, L.w_in, (size_t)rows, 3 * (size_t)L.ul, (size_t)wl};
         g.splits = ti.splits; g.bn = ti.bn;
+        g.f32_out = decode || m->f32;            // a block's projection is rounded to T, a step's partials are summed in f32
         if ((rc = matmul(m, g))) return rc;
       }
       if (m->on(UGB_HYBRID_K_GRU)) {
@@ -263,7 +277,7 @@ int32_t run_layers(ugb_hybrid *m, Work &w, const int *tok, int t_block, int off,
                          (size_t)rows * 3 * L.ul, L.bz, L.bu, L.state, (T *)w.mid, L.ul);
           if (e != cudaSuccess) return ugb_fail(dev, UGB_ERR_CUDA, "launch of min_gru_step_kernel failed: %s", cudaGetErrorString(e));
           if ((rc = ugb_after_launch(dev, "min_gru_step_kernel"))) return rc;
-        } else if ((rc = launch_scan<T>(dev, w.pre, L.bz, L.bu, L.state, (T *)w.mid, B, t, L.ul))) {
+        } else if ((rc = launch_scan<T, T>(dev, (const T *)w.pre, L.bz, L.bu, L.state, (T *)w.mid, B, t, L.ul))) {
           return rc;
         }
       }
@@ -324,7 +338,7 @@ int32_t run_layers(ugb_hybrid *m, Work &w, const int *tok, int t_block, int off,
           a.q = w.ql; a.cache = L.cache; a.out = w.ol; a.gate = w.gate; a.f32 = m->f32; a.rows = rows; a.t = t;
           a.pos_p = m->pos; a.pos_off = off; a.heads = H; a.ld = L.cl; a.t_max = m->t_max; a.gate_ld = L.gl; a.scale = L.d.scale;
           a.splits = decode ? m->att_splits() : 1;
-          a.part_o = m->att_o; a.part_ml = m->att_ml; a.counters = m->att_cnt; a.pdl = pdl;
+          a.pdl = pdl; a.early = early;
           if ((rc = ugb_latent_attention(dev, a))) return rc;
         }
         if (m->on(UGB_HYBRID_K_ABSORB)) {
@@ -356,7 +370,7 @@ int32_t run_layers(ugb_hybrid *m, Work &w, const int *tok, int t_block, int off,
     a.post_gain = L.norm1b; a.x = w.x; a.h = (T *)w.h;
     if (L.d.feed_forward == UGB_FF_NONE) layer_end(a);
     else { a.gain = L.norm2; fuse_conv(a, L.conv2, i, 1); }
-    if ((rc = launch_rows<T>(m, a, rows))) return rc;
+    if ((rc = launch_rows<T>(m, a, rows, early))) return rc;
     if (L.d.feed_forward != UGB_FF_NONE) {
       if ((rc = input_of(L.conv2, i, 1, &in))) return rc;
       if (m->on(UGB_HYBRID_K_UP)) {
@@ -374,7 +388,7 @@ int32_t run_layers(ugb_hybrid *m, Work &w, const int *tok, int t_block, int off,
       f.part = w.pre; f.n_part = td.splits; f.part_stride = (size_t)rows * wl;
       f.post_gain = L.norm2b; f.x = w.x; f.h = (T *)w.h;
       layer_end(f);
-      if ((rc = launch_rows<T>(m, f, rows))) return rc;
+      if ((rc = launch_rows<T>(m, f, rows, early))) return rc;
     }
     if (!decode && m->keep_layers && m->layer_out) {     // rows (b, off + i) of [layer][batch * t_block][wl]
       for (int b = 0; b < B; ++b)
@@ -595,18 +609,6 @@ int32_t ugb_hybrid_create(ugb_device *dev, const ugb_hybrid_config *cfg, const u
   TRY(dmalloc(m, &m->next, batch, true));
   TRY(dmalloc(m, &m->pos, 1, true));
   TRY(alloc_work(m, m->dec, batch, true));
-  {
-    size_t so = 1, sm = 1, sc = 1;
-    for (const Layer &L : m->layers)
-      if (L.d.heads > 0) {
-        so = std::max(so, ugb_latent_scratch_o(batch, L.d.heads, L.cl, UGB_LATENT_MAX_SPLITS));
-        sm = std::max(sm, ugb_latent_scratch_ml(batch, L.d.heads, UGB_LATENT_MAX_SPLITS));
-        sc = std::max(sc, (size_t)batch * ((L.d.heads + 15) / 16));
-      }
-    TRY(dmalloc(m, &m->att_o, so));
-    TRY(dmalloc(m, &m->att_ml, sm));
-    TRY(dmalloc(m, &m->att_cnt, sc, true));
-  }
   TRY(ugb_latent_attention_prepare(dev));
 #undef TRY
 #undef CHECK
@@ -864,7 +866,10 @@ int32_t ugb_min_gru(ugb_device *dev, const ugb_slice *pre, const ugb_slice *bias
   if (!dev) return UGB_ERR_INVALID;
   if (int32_t rc = act_dtype(dev, out, out, "min_gru")) return rc;
   UGB_REQUIRE(dev, width % 8 == 0 && b <= 65535 && 3 * b * t * width < (1ull << 31), UGB_ERR_SHAPE, "min_gru: unsupported shape");
-  UGB_SLICE(dev, pre, UGB_F32, 3 * b * t * width);
+  if (int32_t rc = act_dtype(dev, pre, pre, "min_gru")) return rc;
+  const bool half = pre->dtype == UGB_BF16;
+  UGB_REQUIRE(dev, !half || (t > 1 && out->dtype == UGB_BF16), UGB_ERR_DTYPE, "min_gru: bf16 pre-activations want a block and a bf16 result");
+  UGB_SLICE(dev, pre, pre->dtype, 3 * b * t * width);
   UGB_SLICE(dev, bias_z, UGB_F32, width);
   UGB_SLICE(dev, bias_x, UGB_F32, width);
   UGB_SLICE(dev, state, UGB_F32, b * width);
@@ -875,10 +880,11 @@ int32_t ugb_min_gru(ugb_device *dev, const ugb_slice *pre, const ugb_slice *bias
   float *s = (float *)state->ptr;
   const dim3 grid((unsigned)b, (unsigned)((width / 4 + 127) / 128));
   if (out->dtype == UGB_F32) {
-    if (t > 1) return launch_scan<float>(dev, p, bz, bx, s, (float *)out->ptr, (int)b, (int)t, (int)width);
+    if (t > 1) return launch_scan<float, float>(dev, p, bz, bx, s, (float *)out->ptr, (int)b, (int)t, (int)width);
     min_gru_step_kernel<float><<<grid, 128, 0, dev->stream>>>(p, 1, 0, bz, bx, s, (float *)out->ptr, (int)width);
   } else {
-    if (t > 1) return launch_scan<__nv_bfloat16>(dev, p, bz, bx, s, (__nv_bfloat16 *)out->ptr, (int)b, (int)t, (int)width);
+    if (half) return launch_scan<__nv_bfloat16, __nv_bfloat16>(dev, (const __nv_bfloat16 *)p, bz, bx, s, (__nv_bfloat16 *)out->ptr, (int)b, (int)t, (int)width);
+    if (t > 1) return launch_scan<float, __nv_bfloat16>(dev, p, bz, bx, s, (__nv_bfloat16 *)out->ptr, (int)b, (int)t, (int)width);
     min_gru_step_kernel<__nv_bfloat16><<<grid, 128, 0, dev->stream>>>(p, 1, 0, bz, bx, s, (__nv_bfloat16 *)out->ptr, (int)width);
   }
   return ugb_after_launch(dev, "min_gru_step_kernel");
@@ -903,15 +909,7 @@ int32_t ugb_latent_attend(ugb_device *dev, const ugb_slice *q, const ugb_slice *
   a.q = q->ptr; a.cache = cache->ptr; a.out = out->ptr; a.gate = gate ? (const float *)gate->ptr : nullptr; a.f32 = q->dtype == UGB_F32;
   a.rows = (int)(b * t); a.t = (int)t; a.pos_p = (const int *)pos->ptr; a.heads = (int)heads; a.ld = (int)rank; a.t_max = (int)t_max;
   a.gate_ld = (int)heads; a.scale = scale; a.splits = n_slices;
-  const size_t so = ugb_latent_scratch_o(a.rows, a.heads, a.ld, n_slices) * 4, sm = ugb_latent_scratch_ml(a.rows, a.heads, n_slices) * 4;
-  const size_t sc = (size_t)a.rows * ((heads + 15) / 16) * 4;
-  void *tmp = nullptr;
-  UGB_CUDA(dev, ugb_malloc_async(dev, &tmp, so + sm + sc));
-  a.part_o = (float *)tmp; a.part_ml = (float *)((char *)tmp + so); a.counters = (unsigned *)((char *)tmp + so + sm);
-  if (cudaMemsetAsync(a.counters, 0, sc, dev->stream) != cudaSuccess) rc = ugb_fail(dev, UGB_ERR_CUDA, "latent_attend: clearing the counters failed");
-  if (!rc) rc = ugb_latent_attention(dev, a);
-  cudaFreeAsync(tmp, dev->stream);
-  return rc;
+  return ugb_latent_attention(dev, a);
 }
 
 int32_t ugb_causal_attention_wide(ugb_device *dev, const ugb_slice *q, const ugb_slice *k, const ugb_slice *v, const ugb_slice *gate,
@@ -965,12 +963,12 @@ int32_t ugb_residual_update(ugb_device *dev, ugb_slice *x, const ugb_slice *y, c
     RowArgs<float> a;
     fill(a);
     a.h = (float *)h->ptr;
-    return launch_rows<float>(&m, a, (int)rows);
+    return launch_rows<float>(&m, a, (int)rows, false);
   }
   RowArgs<__nv_bfloat16> a;
   fill(a);
   a.h = (__nv_bfloat16 *)h->ptr;
-  return launch_rows<__nv_bfloat16>(&m, a, (int)rows);
+  return launch_rows<__nv_bfloat16>(&m, a, (int)rows, false);
 }
 
 }  // extern "C"

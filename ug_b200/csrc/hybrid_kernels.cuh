@@ -33,10 +33,15 @@ template <> struct Act<__nv_bfloat16> {
   static __device__ __forceinline__ float round(float v) { return __bfloat162float(__float2bfloat16_rn(v)); }
 };
 
-__device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf(-x)); }
-__device__ __forceinline__ float silu_f(float x) { return x / (1.0f + expf(-x)); }
+// Gate functions in fp32; EXACT: correctly rounded division and full-precision exp (models that run in 32 bits), otherwise
+// the hardware's exp2 and reciprocal (about 1e-6 relative), which the block scan of a bf16 model is bound by.
+template <bool EXACT> __device__ __forceinline__ float over_1_exp(float num, float x) {   // num / (1 + e^-x)
+  return EXACT ? num / (1.0f + expf(-x)) : __fdividef(num, 1.0f + __expf(-x));
+}
+__device__ __forceinline__ float sigmoid_f(float x) { return over_1_exp<true>(1.0f, x); }
+__device__ __forceinline__ float silu_f(float x) { return over_1_exp<true>(x, x); }
 // candidate of the minimal gated recurrent unit: u + 1/2 for u >= 0, sigmoid(u) below
-__device__ __forceinline__ float gru_candidate(float u) { return u >= 0.0f ? u + 0.5f : sigmoid_f(u); }
+template <bool EXACT> __device__ __forceinline__ float gru_candidate(float u) { return u >= 0.0f ? u + 0.5f : over_1_exp<EXACT>(1.0f, u); }
 
 __device__ __forceinline__ float block_sum_256(float v, float *sm) {   // sm: 8 floats; all 256 threads
 #pragma unroll
@@ -81,66 +86,115 @@ template <typename T> struct RowArgs {
   T *tail = nullptr;                   // [rows][taps - 1][ld]
   int ld = 0;
   float inv_width = 0.f, eps = 0.f;
+  int early = 0;                       // 1: x, bank and tail may be read before the wait for the preceding kernel
   ugb_status_word *status = nullptr;
 };
 
-template <typename T, int VPT>
-__global__ void __launch_bounds__(256)
+// Taps of a fused convolution whose tail rows are held in registers from before the wait; longer ones are read late.
+constexpr int ROW_TAPS = 4;
+
+// STEP: few rows (a decode step), everything that can be requested early is; otherwise many rows, whose CTAs hide one
+// another's latencies, and registers count.
+template <typename T, int VPT, bool STEP>
+__global__ void __launch_bounds__(256, (STEP || VPT > 2 ? 1 : 4))
 row_update_kernel(RowArgs<T> a) {
   __shared__ float sm[8];
-  ugb_pdl_trigger();
-  // gains and taps are weights: fetched before the wait for the preceding kernel
   const int r = blockIdx.x, nvec = a.ld >> 2;
-  float4 pg[VPT], g2[VPT];
+  const size_t row0 = (size_t)r * a.ld;
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  float4 *xr = reinterpret_cast<float4 *>(a.x + row0);
+  float4 v[VPT], pg[VPT], acc[VPT];
+  float4 tl[STEP ? ROW_TAPS - 1 : 1][VPT];
+  const bool short_conv = STEP && a.conv != nullptr && a.taps <= ROW_TAPS;
+  // Weights, and what kernels before the predecessor wrote -- the residual row, the layer bank, the convolution tail --
+  // are read ahead of the wait: every kernel of the chain lets its successor start only after its own wait has returned,
+  // so when this kernel runs, everything up to its predecessor's predecessor is complete.
+  if (!a.early) { ugb_pdl_wait(); ugb_pdl_trigger(); }
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
     const int c = threadIdx.x + i * 256;
     pg[i] = make_float4(1.f, 1.f, 1.f, 1.f);
-    g2[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    v[i] = acc[i] = zero;
     if (c < nvec) {
+      if (a.add_x) v[i] = xr[c];
       if (a.post_gain) pg[i] = __ldg(reinterpret_cast<const float4 *>(a.post_gain) + c);
-      g2[i] = __ldg(reinterpret_cast<const float4 *>(a.gain) + c);
+      if (STEP && short_conv) {
+#pragma unroll
+        for (int j = 0; j < (STEP ? ROW_TAPS - 1 : 1); ++j)
+          tl[j][i] = j < a.taps - 1 ? Act<T>::ld4(a.tail + ((size_t)r * (a.taps - 1) + j) * a.ld + 4 * c) : zero;
+      }
     }
   }
-  ugb_pdl_wait();
-  float4 v[VPT], y[VPT];
-  float4 *xr = reinterpret_cast<float4 *>(a.x + (size_t)r * a.ld);
-  const T *erow = nullptr;
+  if (a.dwa) {
+    constexpr int U = STEP ? (VPT <= 2 ? 8 : (VPT <= 4 ? 4 : 2)) : (VPT <= 2 ? 4 : 2);  // bank rows in flight
+    for (int j = 0; j < a.n_avg; j += U) {
+      float4 q[U][VPT];
+      float w[U];
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const bool on = j + u < a.n_avg;
+        w[u] = on ? __ldg(a.dwa + j + u) : 0.f;
+#pragma unroll
+        for (int i = 0; i < VPT; ++i) {
+          const int c = threadIdx.x + i * 256;
+          q[u][i] = zero;
+          if (on && c < nvec) q[u][i] = __ldcg(reinterpret_cast<const float4 *>(a.bank + (size_t)(j + u) * a.bank_stride + row0) + c);
+        }
+      }
+#pragma unroll
+      for (int u = 0; u < U; ++u)
+#pragma unroll
+        for (int i = 0; i < VPT; ++i) {
+          acc[i].x = fmaf(w[u], q[u][i].x, acc[i].x); acc[i].y = fmaf(w[u], q[u][i].y, acc[i].y);
+          acc[i].z = fmaf(w[u], q[u][i].z, acc[i].z); acc[i].w = fmaf(w[u], q[u][i].w, acc[i].w);
+        }
+    }
+  }
+  if (a.early) { ugb_pdl_wait(); ugb_pdl_trigger(); }
+  float4 y[VPT];
   if (a.tok) {
     const int id = a.tok[(size_t)(r / a.t) * a.tok_stride + a.tok_off + r % a.t];
     if (id < 0 || id >= a.vocab) {
       if (threadIdx.x == 0 && atomicCAS(&a.status->code, 0u, (unsigned)UGB_ERR_INVALID) == 0u) a.status->detail = r;
       return;
     }
-    erow = a.embed + (size_t)id * a.ld;
-  }
 #pragma unroll
-  for (int i = 0; i < VPT; ++i) {
-    const int c = threadIdx.x + i * 256;
-    v[i] = y[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (c < nvec) {
-      if (a.add_x) v[i] = xr[c];
-      if (erow) y[i] = Act<T>::ld4(erow + 4 * c);
-      else y[i] = __ldcs(reinterpret_cast<const float4 *>(a.part + (size_t)r * a.ld) + c);
+    for (int i = 0; i < VPT; ++i) {
+      const int c = threadIdx.x + i * 256;
+      y[i] = c < nvec ? Act<T>::ld4(a.embed + (size_t)id * a.ld + 4 * c) : zero;
     }
-  }
-  if (!erow && a.n_part > 1) {
-    for (int s = 1; s < a.n_part; s += 4) {               // split-K partials in order, four round trips in flight
-      float4 q[4][VPT];
+  } else if (a.n_part == 1) {
 #pragma unroll
-      for (int u = 0; u < 4; ++u)
+    for (int i = 0; i < VPT; ++i) {
+      const int c = threadIdx.x + i * 256;
+      y[i] = c < nvec ? __ldcs(reinterpret_cast<const float4 *>(a.part + row0) + c) : zero;
+    }
+  } else {
+    constexpr int U = STEP ? (VPT <= 2 ? 8 : 4) : 1;      // split-K partials, added in order, U round trips in flight
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) y[i] = zero;
+    for (int s = 0; s < a.n_part; s += U) {
+      float4 q[U][VPT];
+#pragma unroll
+      for (int u = 0; u < U; ++u)
 #pragma unroll
         for (int i = 0; i < VPT; ++i) {
           const int c = threadIdx.x + i * 256;
-          q[u][i] = make_float4(0.f, 0.f, 0.f, 0.f);
+          q[u][i] = zero;
           if (c < nvec && s + u < a.n_part)
-            q[u][i] = __ldcs(reinterpret_cast<const float4 *>(a.part + (size_t)(s + u) * a.part_stride + (size_t)r * a.ld) + c);
+            q[u][i] = __ldcs(reinterpret_cast<const float4 *>(a.part + (size_t)(s + u) * a.part_stride + row0) + c);
         }
 #pragma unroll
-      for (int u = 0; u < 4; ++u)
+      for (int u = 0; u < U; ++u)
 #pragma unroll
         for (int i = 0; i < VPT; ++i) { y[i].x += q[u][i].x; y[i].y += q[u][i].y; y[i].z += q[u][i].z; y[i].w += q[u][i].w; }
     }
+  }
+  float4 g2[VPT];
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = threadIdx.x + i * 256;
+    g2[i] = c < nvec ? __ldg(reinterpret_cast<const float4 *>(a.gain) + c) : zero;
   }
   float inv = 1.f;
   if (a.post_gain) {
@@ -155,7 +209,7 @@ row_update_kernel(RowArgs<T> a) {
     v[i].z += y[i].z * inv * pg[i].z; v[i].w += y[i].w * inv * pg[i].w;
   }
   if (a.bank_out) {
-    float4 *bo = reinterpret_cast<float4 *>(a.bank_out + (size_t)r * a.ld);
+    float4 *bo = reinterpret_cast<float4 *>(a.bank_out + row0);
 #pragma unroll
     for (int i = 0; i < VPT; ++i) {
       const int c = threadIdx.x + i * 256;
@@ -164,32 +218,6 @@ row_update_kernel(RowArgs<T> a) {
   }
   if (a.dwa) {
     const float own = __ldg(a.dwa + a.n_avg);
-    float4 acc[VPT];
-#pragma unroll
-    for (int i = 0; i < VPT; ++i) acc[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-    constexpr int U = VPT <= 2 ? 8 : (VPT <= 4 ? 4 : 2);  // bank rows in flight
-    for (int j = 0; j < a.n_avg; j += U) {
-      float4 q[U][VPT];
-      float w[U];
-#pragma unroll
-      for (int u = 0; u < U; ++u) {
-        const bool on = j + u < a.n_avg;
-        w[u] = on ? __ldg(a.dwa + j + u) : 0.f;
-#pragma unroll
-        for (int i = 0; i < VPT; ++i) {
-          const int c = threadIdx.x + i * 256;
-          q[u][i] = make_float4(0.f, 0.f, 0.f, 0.f);
-          if (on && c < nvec) q[u][i] = __ldcg(reinterpret_cast<const float4 *>(a.bank + (size_t)(j + u) * a.bank_stride + (size_t)r * a.ld) + c);
-        }
-      }
-#pragma unroll
-      for (int u = 0; u < U; ++u)
-#pragma unroll
-        for (int i = 0; i < VPT; ++i) {
-          acc[i].x = fmaf(w[u], q[u][i].x, acc[i].x); acc[i].y = fmaf(w[u], q[u][i].y, acc[i].y);
-          acc[i].z = fmaf(w[u], q[u][i].z, acc[i].z); acc[i].w = fmaf(w[u], q[u][i].w, acc[i].w);
-        }
-    }
 #pragma unroll
     for (int i = 0; i < VPT; ++i) {
       v[i].x = fmaf(own, v[i].x, acc[i].x); v[i].y = fmaf(own, v[i].y, acc[i].y);
@@ -204,6 +232,9 @@ row_update_kernel(RowArgs<T> a) {
     ss += sq4(v[i]);
   }
   const float inv2 = 1.0f / sqrtf(block_sum_256(ss, sm) * a.inv_width + a.eps);
+  auto fma4 = [](float4 w, float4 q, float4 &s) {
+    s.x = fmaf(w.x, q.x, s.x); s.y = fmaf(w.y, q.y, s.y); s.z = fmaf(w.z, q.z, s.z); s.w = fmaf(w.w, q.w, s.w);
+  };
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
     const int c = threadIdx.x + i * 256;
@@ -212,50 +243,129 @@ row_update_kernel(RowArgs<T> a) {
     if (a.conv) {
       // what the convolution sees, now and later, is the rounded h
       h = make_float4(Act<T>::round(h.x), Act<T>::round(h.y), Act<T>::round(h.z), Act<T>::round(h.w));
-      T *tl = a.tail + (size_t)r * (a.taps - 1) * a.ld + 4 * c;
-      float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
-      for (int j = 0; j < a.taps; ++j) {
-        const float4 w = __ldg(reinterpret_cast<const float4 *>(a.conv + (size_t)j * a.ld) + c);
-        const float4 q = j + 1 < a.taps ? Act<T>::ld4(tl + (size_t)j * a.ld) : h;
-        if (j > 0) Act<T>::st4(tl + (size_t)(j - 1) * a.ld, q);
-        s.x = fmaf(w.x, q.x, s.x); s.y = fmaf(w.y, q.y, s.y); s.z = fmaf(w.z, q.z, s.z); s.w = fmaf(w.w, q.w, s.w);
+      T *tp = a.tail + (size_t)r * (a.taps - 1) * a.ld + 4 * c;
+      const float4 *cw = reinterpret_cast<const float4 *>(a.conv) + c;
+      float4 s = zero;
+      if (STEP && short_conv) {
+        float4 w[ROW_TAPS];
+#pragma unroll
+        for (int j = 0; j < ROW_TAPS; ++j) w[j] = j < a.taps ? __ldg(cw + (size_t)j * (a.ld >> 2)) : zero;
+#pragma unroll
+        for (int j = 0; j < ROW_TAPS; ++j) {
+          if (j < a.taps - 1) {
+            const float4 q = tl[STEP && j < ROW_TAPS - 1 ? j : 0][i];
+            fma4(w[j], q, s);
+            if (j > 0) Act<T>::st4(tp + (size_t)(j - 1) * a.ld, q);
+          } else if (j == a.taps - 1) {
+            fma4(w[j], h, s);
+            if (j > 0) Act<T>::st4(tp + (size_t)(j - 1) * a.ld, h);
+          }
+        }
+      } else {
+        for (int j = 0; j < a.taps; ++j) {
+          const float4 q = j + 1 < a.taps ? Act<T>::ld4(tp + (size_t)j * a.ld) : h;
+          if (j > 0) Act<T>::st4(tp + (size_t)(j - 1) * a.ld, q);
+          fma4(__ldg(cw + (size_t)j * (a.ld >> 2)), q, s);
+        }
       }
       h.x += s.x; h.y += s.y; h.z += s.z; h.w += s.w;
     }
-    Act<T>::st4(a.h + (size_t)r * a.ld + 4 * c, h);
+    Act<T>::st4(a.h + row0 + 4 * c, h);
   }
 }
 
 // ------------------------------------------------- causal input convolution ---
 // out[b, i] = h[b, i] + sum_j w[j] h[b, i - (taps - 1) + j] over a block of t positions per sequence, rows before the
 // block from tail_in [b][taps - 1][ld]; the block's own last taps - 1 rows go to tail_out (a different buffer).
-// One thread per 4 channels and CONV_STRIP positions: a row of h is fetched once per tap from L1.
+// One thread per 8 channels and CONV_STRIP positions; with TAPS > 0 (the tap count, when it is small) the rows of the
+// strip slide through registers, all of them requested before the first is used; TAPS = 0 takes any tap count.
 constexpr int CONV_STRIP = 8;
+constexpr int CONV_TAPS = 4;
 
-template <typename T>
-__global__ void __launch_bounds__(256)
+template <typename T> struct Row8 { float v[8]; };
+struct alignas(16) Raw32 { uint4 a, b; };
+template <typename T> struct RawRow8 { using type = uint4; };
+template <> struct RawRow8<float> { using type = Raw32; };
+template <typename T> __device__ __forceinline__ Row8<T> ld8(const T *p) {
+  Row8<T> r;
+  if constexpr (sizeof(T) == 2) {
+    const uint4 u = *reinterpret_cast<const uint4 *>(p);
+    const __nv_bfloat162 *h = reinterpret_cast<const __nv_bfloat162 *>(&u);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) { const float2 f = __bfloat1622float2(h[e]); r.v[2 * e] = f.x; r.v[2 * e + 1] = f.y; }
+  } else {
+    const float4 a = Act<T>::ld4(p), b = Act<T>::ld4(p + 4);
+    r.v[0] = a.x; r.v[1] = a.y; r.v[2] = a.z; r.v[3] = a.w; r.v[4] = b.x; r.v[5] = b.y; r.v[6] = b.z; r.v[7] = b.w;
+  }
+  return r;
+}
+template <typename T> __device__ __forceinline__ void st8(T *p, const Row8<T> &r) {
+  if constexpr (sizeof(T) == 2) {
+    uint4 u;
+    uint32_t *w = reinterpret_cast<uint32_t *>(&u);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) { __nv_bfloat162 b = __floats2bfloat162_rn(r.v[2 * e], r.v[2 * e + 1]); w[e] = *(uint32_t *)&b; }
+    *reinterpret_cast<uint4 *>(p) = u;
+  } else {
+    Act<T>::st4(p, make_float4(r.v[0], r.v[1], r.v[2], r.v[3]));
+    Act<T>::st4(p + 4, make_float4(r.v[4], r.v[5], r.v[6], r.v[7]));
+  }
+}
+
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(128)
 causal_conv_kernel(const T *__restrict__ h, const float *__restrict__ w, const T *__restrict__ tail_in, T *__restrict__ tail_out,
-                   T *__restrict__ out, int t, int taps, int ld) {
+                   T *__restrict__ out, int t, int taps_any, int ld) {
+  const int taps = TAPS > 0 ? TAPS : taps_any;
   const int c = blockIdx.y * blockDim.x + threadIdx.x, b = blockIdx.z;
-  if (c >= ld >> 2) return;
-  const T *hb = h + (size_t)b * t * ld + 4 * c;
-  const T *ti = tail_in + (size_t)b * (taps - 1) * ld + 4 * c;
-  T *to = tail_out + (size_t)b * (taps - 1) * ld + 4 * c;
-  auto row = [&](int i) { return i >= 0 ? Act<T>::ld4(hb + (size_t)i * ld) : Act<T>::ld4(ti + (size_t)(i + taps - 1) * ld); };
+  if (c >= ld >> 3) return;
+  const T *hb = h + (size_t)b * t * ld + 8 * c;
+  const T *ti = tail_in + (size_t)b * (taps - 1) * ld + 8 * c;
+  T *to = tail_out + (size_t)b * (taps - 1) * ld + 8 * c;
+  T *ob = out + (size_t)b * t * ld + 8 * c;
+  auto row = [&](int i) { return i >= 0 ? ld8<T>(hb + (size_t)i * ld) : ld8<T>(ti + (size_t)(i + taps - 1) * ld); };
   const int i0 = blockIdx.x * CONV_STRIP, i1 = min(i0 + CONV_STRIP, t);
-#pragma unroll 4
-  for (int i = i0; i < i1; ++i) {
-    float4 own = make_float4(0.f, 0.f, 0.f, 0.f), s = own;
-    for (int j = 0; j < taps; ++j) {
-      const float4 q = row(i - (taps - 1) + j);
-      const float4 wv = __ldg(reinterpret_cast<const float4 *>(w + (size_t)j * ld) + c);
-      s.x = fmaf(wv.x, q.x, s.x); s.y = fmaf(wv.y, q.y, s.y); s.z = fmaf(wv.z, q.z, s.z); s.w = fmaf(wv.w, q.w, s.w);
-      own = q;                                             // the last tap is position i itself
+  if constexpr (TAPS > 0) {
+    using Raw = typename RawRow8<T>::type;                 // rows wait as they are stored and are widened when used
+    Raw q[CONV_STRIP + TAPS - 1];
+#pragma unroll
+    for (int k = 0; k < CONV_STRIP + TAPS - 1; ++k) {
+      const int i = i0 - (TAPS - 1) + k;
+      if (i < i1) q[k] = *reinterpret_cast<const Raw *>(i >= 0 ? hb + (size_t)i * ld : ti + (size_t)(i + TAPS - 1) * ld);
     }
-    Act<T>::st4(out + ((size_t)b * t + i) * ld + 4 * c, make_float4(own.x + s.x, own.y + s.y, own.z + s.z, own.w + s.w));
+    Row8<float> wv[TAPS];
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) wv[j] = ld8<float>(w + (size_t)j * ld + 8 * c);
+#pragma unroll
+    for (int k = 0; k < CONV_STRIP; ++k) {
+      if (i0 + k >= i1) break;
+      Row8<T> o{}, x;
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) {
+        x = ld8<T>(reinterpret_cast<const T *>(&q[k + j]));
+#pragma unroll
+        for (int e = 0; e < 8; ++e) o.v[e] = fmaf(wv[j].v[e], x.v[e], o.v[e]);
+      }
+#pragma unroll
+      for (int e = 0; e < 8; ++e) o.v[e] += x.v[e];        // the last tap is the position itself
+      st8<T>(ob + (size_t)(i0 + k) * ld, o);
+    }
+  } else {
+    for (int i = i0; i < i1; ++i) {
+      Row8<T> own{}, o{};
+      for (int j = 0; j < taps; ++j) {
+        own = row(i - (taps - 1) + j);
+        const Row8<float> wv = ld8<float>(w + (size_t)j * ld + 8 * c);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) o.v[e] = fmaf(wv.v[e], own.v[e], o.v[e]);
+      }
+#pragma unroll
+      for (int e = 0; e < 8; ++e) o.v[e] += own.v[e];
+      st8<T>(ob + (size_t)i * ld, o);
+    }
   }
   if (i1 == t)
-    for (int j = 0; j < taps - 1; ++j) Act<T>::st4(to + (size_t)j * ld, row(t - (taps - 1) + j));
+    for (int j = 0; j < taps - 1; ++j) st8<T>(to + (size_t)j * ld, row(t - (taps - 1) + j));
 }
 
 // ---------------------------------------------------------- minimal GRU -----
@@ -266,7 +376,6 @@ template <typename T>
 __global__ void __launch_bounds__(128)
 min_gru_step_kernel(const float *__restrict__ pre, int n_part, size_t part_stride, const float *__restrict__ bz,
                     const float *__restrict__ bu, float *__restrict__ state, T *__restrict__ out, int ld) {
-  ugb_pdl_trigger();
   const int r = blockIdx.x, c = blockIdx.y * blockDim.x + threadIdx.x;
   const bool on = c < ld >> 2;
   float4 z = make_float4(0.f, 0.f, 0.f, 0.f), u = z, g = z;
@@ -274,10 +383,13 @@ min_gru_step_kernel(const float *__restrict__ pre, int n_part, size_t part_strid
     z = __ldg(reinterpret_cast<const float4 *>(bz) + c);
     u = __ldg(reinterpret_cast<const float4 *>(bu) + c);
   }
+  // the state was written a step ago, by a kernel that is certainly complete (see row_update_kernel)
+  float4 S = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (on) S = *reinterpret_cast<const float4 *>(state + (size_t)r * ld + 4 * c);
   ugb_pdl_wait();
+  ugb_pdl_trigger();
   if (!on) return;
   const float *row = pre + (size_t)r * 3 * ld + 4 * c;
-  float4 S = *reinterpret_cast<const float4 *>(state + (size_t)r * ld + 4 * c);
   auto add = [](float4 &d, float4 s) { d.x += s.x; d.y += s.y; d.z += s.z; d.w += s.w; };
   for (int s = 0; s < n_part; s += 4) {
     float4 q[4][3];
@@ -293,7 +405,7 @@ min_gru_step_kernel(const float *__restrict__ pre, int n_part, size_t part_strid
   }
   auto step = [](float S0, float zp, float up) {
     const float zz = sigmoid_f(zp);
-    return (1.0f - zz) * S0 + zz * gru_candidate(up);
+    return (1.0f - zz) * S0 + zz * gru_candidate<true>(up);
   };
   S = make_float4(step(S.x, z.x, u.x), step(S.y, z.y, u.y), step(S.z, z.z, u.z), step(S.w, z.w, u.w));
   *reinterpret_cast<float4 *>(state + (size_t)r * ld + 4 * c) = S;
@@ -305,83 +417,144 @@ min_gru_step_kernel(const float *__restrict__ pre, int n_part, size_t part_strid
 // composes its positions into one affine map S -> A S + B held in registers, the maps meet in shared memory (warps)
 // and distributed shared memory (CTAs), and every warp then replays its positions from its own incoming state.  The
 // cluster walks the sequence in rounds of SCAN_BLOCK * gridDim.x positions; all CTAs run every round.
-constexpr int SCAN_WARPS = 16, SCAN_STEPS = 8, SCAN_BLOCK = SCAN_WARPS * SCAN_STEPS;
+// bf16 pre-activations: a lane takes two adjacent channels, so a warp reads 128 bytes of a row either way.
+constexpr int SCAN_WARPS = 16;
+template <typename TI> struct Scan {
+  static constexpr int V = sizeof(TI) == 2 ? 2 : 1;        // channels per lane
+  static constexpr int STEPS = 4;                          // positions per warp and round
+  static constexpr int BLOCK = SCAN_WARPS * STEPS, COLUMNS = 32 * V;
+};
 
-template <typename TI> __device__ __forceinline__ float scan_load(const TI *p) { return (float)*p; }
+// a lane's channels of one pre-activation row, as stored (32 bits either way)
+template <int V> __device__ __forceinline__ void scan_widen(uint32_t raw, float (&f)[V]) {
+  if constexpr (V == 2) {
+    const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&raw));
+    f[0] = x.x; f[1] = x.y;
+  } else f[0] = __uint_as_float(raw);
+}
 
 template <typename TI, typename T>
-__global__ void __launch_bounds__(SCAN_WARPS * 32)
+__global__ void __launch_bounds__(SCAN_WARPS * 32, 2)
 min_gru_scan_kernel(const TI *__restrict__ pre, const float *__restrict__ bz, const float *__restrict__ bu,
                     float *__restrict__ state, T *__restrict__ out, int t, int ld) {
-  __shared__ float agg_a[SCAN_WARPS][32], agg_b[SCAN_WARPS][32];
-  __shared__ float tot[2][2][32];                          // [round parity][A, B][channel], read by the cluster
+  constexpr int V = Scan<TI>::V, STEPS = Scan<TI>::STEPS, BLOCK = Scan<TI>::BLOCK, COLS = Scan<TI>::COLUMNS;
+  constexpr bool EXACT = sizeof(T) == 4;
+  __shared__ float agg_a[SCAN_WARPS][COLS], agg_b[SCAN_WARPS][COLS];
+  __shared__ float tot[2][2][COLS];                        // [round parity][A, B][channel], read by the cluster
+  __shared__ float enter[COLS], carry[COLS];               // state entering this CTA's piece, state before the round
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int rank = blockIdx.x, n_cta = gridDim.x, b = blockIdx.z;
-  const int c = blockIdx.y * 32 + lane;
+  const int c = blockIdx.y * COLS + lane * V;              // ld is a multiple of 8: a lane's channels are all in or all out
   const bool on = c < ld;
-  const float zb = on ? bz[c] : 0.f, ub = on ? bu[c] : 0.f;
-  const size_t base = (size_t)b * t;
-  float carry = on ? state[(size_t)b * ld + c] : 0.f;      // state before this round (every warp of every CTA keeps it)
-  int round = 0;
-  for (int t0 = 0; t0 < t; t0 += SCAN_BLOCK * n_cta, ++round) {
-    const int i0 = t0 + rank * SCAN_BLOCK + warp * SCAN_STEPS;
-    float a[SCAN_STEPS], bb[SCAN_STEPS], sg[SCAN_STEPS];
+  float zb[V], ub[V];
 #pragma unroll
-    for (int s = 0; s < SCAN_STEPS; ++s) {
-      a[s] = bb[s] = sg[s] = 0.f;
+  for (int e = 0; e < V; ++e) {
+    zb[e] = on ? bz[c + e] : 0.f;
+    ub[e] = on ? bu[c + e] : 0.f;
+  }
+  if (threadIdx.x < COLS) {
+    const int k = blockIdx.y * COLS + threadIdx.x;
+    carry[threadIdx.x] = k < ld ? state[(size_t)b * ld + k] : 0.f;
+  }
+  const size_t base = (size_t)b * t;
+  uint32_t nz[STEPS], nu[STEPS], ng[STEPS];                // the coming round's rows, requested a round ahead
+  auto fetch = [&](int i0) {
+#pragma unroll
+    for (int s = 0; s < STEPS; ++s) {
+      nz[s] = nu[s] = ng[s] = 0u;
       if (on && i0 + s < t) {
         const TI *row = pre + (base + i0 + s) * (size_t)(3 * ld) + c;
-        a[s] = scan_load(row); bb[s] = scan_load(row + ld); sg[s] = scan_load(row + 2 * ld);
+        nz[s] = __ldcs(reinterpret_cast<const uint32_t *>(row));
+        nu[s] = __ldcs(reinterpret_cast<const uint32_t *>(row + ld));
+        ng[s] = __ldcs(reinterpret_cast<const uint32_t *>(row + 2 * ld));
       }
     }
-    float A = 1.f, B = 0.f;
+  };
+  fetch(rank * BLOCK + warp * STEPS);
+  int round = 0;
+  for (int t0 = 0; t0 < t; t0 += BLOCK * n_cta, ++round) {
+    const int i0 = t0 + rank * BLOCK + warp * STEPS;
+    float a[STEPS][V], bb[STEPS][V], sg[STEPS][V];
 #pragma unroll
-    for (int s = 0; s < SCAN_STEPS; ++s) {
-      if (on && i0 + s < t) {
-        const float z = sigmoid_f(a[s] + zb);
-        a[s] = 1.0f - z;
-        bb[s] = z * gru_candidate(bb[s] + ub);
-        sg[s] = silu_f(sg[s]);
-      } else { a[s] = 1.f; bb[s] = 0.f; sg[s] = 0.f; }
-      A *= a[s];
-      B = fmaf(a[s], B, bb[s]);
+    for (int s = 0; s < STEPS; ++s) { scan_widen<V>(nz[s], a[s]); scan_widen<V>(nu[s], bb[s]); scan_widen<V>(ng[s], sg[s]); }
+    fetch(i0 + BLOCK * n_cta);
+    float A[V], B[V];
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      A[e] = 1.f; B[e] = 0.f;
+#pragma unroll
+      for (int s = 0; s < STEPS; ++s) {
+        if (on && i0 + s < t) {
+          const float z = over_1_exp<EXACT>(1.0f, a[s][e] + zb[e]);
+          a[s][e] = 1.0f - z;
+          bb[s][e] = z * gru_candidate<EXACT>(bb[s][e] + ub[e]);
+          sg[s][e] = over_1_exp<EXACT>(sg[s][e], sg[s][e]);
+        } else { a[s][e] = 1.f; bb[s][e] = 0.f; sg[s][e] = 0.f; }
+        A[e] *= a[s][e];
+        B[e] = fmaf(a[s][e], B[e], bb[s][e]);
+      }
+      agg_a[warp][lane * V + e] = A[e]; agg_b[warp][lane * V + e] = B[e];
     }
-    agg_a[warp][lane] = A; agg_b[warp][lane] = B;
     __syncthreads();
-    if (warp == 0) {                                       // this CTA's map
+    if (threadIdx.x < COLS) {                              // this CTA's map, a thread per channel
       float TA = 1.f, TB = 0.f;
 #pragma unroll
-      for (int w = 0; w < SCAN_WARPS; ++w) { TB = fmaf(agg_a[w][lane], TB, agg_b[w][lane]); TA *= agg_a[w][lane]; }
-      tot[round & 1][0][lane] = TA; tot[round & 1][1][lane] = TB;
+      for (int w = 0; w < SCAN_WARPS; ++w) { TB = fmaf(agg_a[w][threadIdx.x], TB, agg_b[w][threadIdx.x]); TA *= agg_a[w][threadIdx.x]; }
+      tot[round & 1][0][threadIdx.x] = TA; tot[round & 1][1][threadIdx.x] = TB;
     }
     // the parity of `tot` alternates, so one barrier per round separates a round's writes from the reads of the
     // round before the last
-    ugb_tc::cluster_sync_all();
-    float in = carry, S = carry;
-    for (int q = 0; q < n_cta; ++q) {
-      const uint32_t ra = ugb_tc::mapa_u32(ugb_tc::smem_u32(&tot[round & 1][0][lane]), (uint32_t)q);
-      const uint32_t rb = ugb_tc::mapa_u32(ugb_tc::smem_u32(&tot[round & 1][1][lane]), (uint32_t)q);
-      float va, vb;
-      asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(va) : "r"(ra) : "memory");
-      asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(vb) : "r"(rb) : "memory");
-      if (q == rank) in = S;                               // state entering this CTA's piece
-      S = fmaf(va, S, vb);
-    }
-    carry = S;
-    S = in;
-    for (int w = 0; w < warp; ++w) S = fmaf(agg_a[w][lane], S, agg_b[w][lane]);
+    if (n_cta > 1) ugb_tc::cluster_sync_all();
+    if (threadIdx.x < COLS) {
+      float in = carry[threadIdx.x], R = in;
+      const uint32_t pa = ugb_tc::smem_u32(&tot[round & 1][0][threadIdx.x]), pb = ugb_tc::smem_u32(&tot[round & 1][1][threadIdx.x]);
+      float va[8], vb[8];                                  // every CTA's map is requested before the first is used
 #pragma unroll
-    for (int s = 0; s < SCAN_STEPS; ++s) {
-      S = fmaf(a[s], S, bb[s]);
+      for (int q = 0; q < 8; ++q) {
+        va[q] = 1.f; vb[q] = 0.f;
+        if (q < n_cta) {
+          asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(va[q]) : "r"(ugb_tc::mapa_u32(pa, (uint32_t)q)) : "memory");
+          asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(vb[q]) : "r"(ugb_tc::mapa_u32(pb, (uint32_t)q)) : "memory");
+        }
+      }
+#pragma unroll
+      for (int q = 0; q < 8; ++q) {
+        if (q == rank) in = R;                             // state entering this CTA's piece
+        R = fmaf(va[q], R, vb[q]);
+      }
+      carry[threadIdx.x] = R;
+      enter[threadIdx.x] = in;
+    }
+    __syncthreads();
+    float S[V];
+#pragma unroll
+    for (int e = 0; e < V; ++e) S[e] = enter[lane * V + e];
+    for (int w = 0; w < warp; ++w)
+#pragma unroll
+      for (int e = 0; e < V; ++e) S[e] = fmaf(agg_a[w][lane * V + e], S[e], agg_b[w][lane * V + e]);
+#pragma unroll
+    for (int s = 0; s < STEPS; ++s) {
+#pragma unroll
+      for (int e = 0; e < V; ++e) S[e] = fmaf(a[s][e], S[e], bb[s][e]);
       if (on && i0 + s < t) {
-        if constexpr (sizeof(T) == 4) out[(base + i0 + s) * (size_t)ld + c] = S * sg[s];
-        else out[(base + i0 + s) * (size_t)ld + c] = __float2bfloat16_rn(S * sg[s]);
+        T *o = out + (base + i0 + s) * (size_t)ld + c;
+        if constexpr (sizeof(T) == 4) {
+#pragma unroll
+          for (int e = 0; e < V; ++e) o[e] = S[e] * sg[s][e];
+        } else if constexpr (V == 2) {
+          *reinterpret_cast<__nv_bfloat162 *>(o) = __floats2bfloat162_rn(S[0] * sg[s][0], S[1] * sg[s][1]);
+        } else {
+          *o = __float2bfloat16_rn(S[0] * sg[s][0]);
+        }
       }
     }
     __syncthreads();                                       // agg_a / agg_b are free
   }
   ugb_tc::cluster_sync_all();                              // no CTA leaves (or writes the state) while a peer still reads
-  if (on && rank == 0 && warp == 0) state[(size_t)b * ld + c] = carry;
+  if (rank == 0 && threadIdx.x < COLS) {
+    const int k = blockIdx.y * COLS + threadIdx.x;
+    if (k < ld) state[(size_t)b * ld + k] = carry[threadIdx.x];
+  }
 }
 
 // ------------------------------------------------- latent attention inputs ---
@@ -395,30 +568,45 @@ latent_inputs_kernel(const float *__restrict__ pre, int n_part, size_t part_stri
                      const int *__restrict__ pos_p, int pos_off, int t, int t_max, int q_ld, int c_ld, int g_ld,
                      float inv_q, float inv_c, float eps, ugb_status_word *status) {
   extern __shared__ __align__(16) float row_s[];
-  __shared__ float sm[8];
-  ugb_pdl_trigger();
-  ugb_pdl_wait();
+  __shared__ float sm[2][8];
   const int r = blockIdx.x, n = q_ld + c_ld + g_ld, tid = threadIdx.x;
+  const int b = r / t;
+  ugb_pdl_wait();
+  ugb_pdl_trigger();
+  const int pos = *pos_p + pos_off + r % t;
   float sq = 0.f, sc = 0.f;
   for (int c = tid; c < n >> 2; c += 256) {
+    const float *src = pre + (size_t)r * n + 4 * c;
     float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
-    for (int s = 0; s < n_part; s += 4) {
-      float4 q[4];
+    if (n_part == 1) {
+      y = __ldcs(reinterpret_cast<const float4 *>(src));
+    } else {
+      for (int s = 0; s < n_part; s += 8) {               // split-K partials, added in order
+        float4 q[8];
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        q[e] = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (s + e < n_part) q[e] = __ldcs(reinterpret_cast<const float4 *>(pre + (size_t)(s + e) * part_stride + (size_t)r * n) + c);
+        for (int e = 0; e < 8; ++e) {
+          q[e] = make_float4(0.f, 0.f, 0.f, 0.f);
+          if (s + e < n_part) q[e] = __ldcs(reinterpret_cast<const float4 *>(src + (size_t)(s + e) * part_stride));
+        }
+#pragma unroll
+        for (int e = 0; e < 8; ++e) { y.x += q[e].x; y.y += q[e].y; y.z += q[e].z; y.w += q[e].w; }
       }
-#pragma unroll
-      for (int e = 0; e < 4; ++e) { y.x += q[e].x; y.y += q[e].y; y.z += q[e].z; y.w += q[e].w; }
     }
-    reinterpret_cast<float4 *>(row_s)[c] = y;
+    reinterpret_cast<float4 *>(row_s)[c] = y;              // read back by the same thread
     if (4 * c < q_ld) sq += sq4(y);                        // the segments are multiples of 8 wide
     else if (4 * c < q_ld + c_ld) sc += sq4(y);
   }
-  const float rq = 1.0f / sqrtf(block_sum_256(sq, sm) * inv_q + eps);
-  const float rc = 1.0f / sqrtf(block_sum_256(sc, sm) * inv_c + eps);   // its barriers also publish row_s
-  const int b = r / t, pos = *pos_p + pos_off + r % t;
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    sq += __shfl_xor_sync(0xffffffffu, sq, o);
+    sc += __shfl_xor_sync(0xffffffffu, sc, o);
+  }
+  if ((tid & 31) == 0) { sm[0][tid >> 5] = sq; sm[1][tid >> 5] = sc; }
+  __syncthreads();
+  sq = sc = 0.f;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) { sq += sm[0][i]; sc += sm[1][i]; }
+  const float rq = 1.0f / sqrtf(sq * inv_q + eps), rc = 1.0f / sqrtf(sc * inv_c + eps);
   const bool ok = pos >= 0 && pos < t_max;
   if (!ok && tid == 0 && atomicCAS(&status->code, 0u, (unsigned)UGB_ERR_INVALID) == 0u) status->detail = (unsigned)pos;
   for (int c = tid; c < n >> 2; c += 256) {

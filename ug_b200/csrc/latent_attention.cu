@@ -16,16 +16,17 @@ using ugb_decode::cp_async16;
 using ugb_decode::cp_async_commit;
 using ugb_decode::mma_bf16_16x8x16;
 using ugb_decode::pack_bf16;
+using ugb_tc::cluster_sync_all;
+using ugb_tc::mapa_u32;
+using ugb_tc::smem_u32;
 
 struct Params {
   const void *q, *cache;
   void *out;
   const float *gate;
-  int t, pos_off, heads, ld, t_max, gate_ld, splits;
+  int t, pos_off, heads, ld, t_max, gate_ld, splits, early;
   const int *pos_p;
   float scale;
-  float *part_o, *part_ml;
-  unsigned *counters;
   ugb_status_word *status;
 };
 
@@ -49,10 +50,10 @@ __device__ __forceinline__ int keys_of(const Params &p, int r) {
 // grid (splits, head groups of 16, rows), 256 threads, cache rows of 64 NT elements.
 // A 32-key tile lies in shared memory as rows of NT 128-byte pieces, the 16-byte chunks of a piece XORed with the key
 // (the 128-byte swizzle): ldmatrix over 8 keys of one chunk column is conflict-free, plain and transposed.
-//   scores   warp w: keys 8 (w & 3) .. + 7 over half (w >> 2) of the latent; the halves meet in shared memory
+//   scores   warp w: keys 16 (w & 1) .. + 15 over quarter w >> 1 of the latent; the quarters meet in shared memory
 //   softmax  every warp for itself, straight in the A-fragment layout of the second product (fp32, online)
 //   sums     warp w: latent columns 8 NT w .. + 8 NT - 1
-// The scores of tile j + 1 are formed before the sums of tile j, so one CTA barrier per tile suffices.
+// The ring matters more than the arithmetic: of STAGES tiles one is worked on, the others are in flight.
 constexpr int KT = 32;
 constexpr int WARPS = 8;
 template <int NT> struct Ring {
@@ -67,16 +68,19 @@ __global__ void __launch_bounds__(WARPS * 32, 2)
 latent_attention_mma_kernel(Params p) {
   using R = Ring<NT>;
   extern __shared__ __align__(128) uint8_t ring[];
-  __shared__ float sc[2][2][16][KT + 2];                   // [tile parity][latent half][head][key]
-  __shared__ int is_last;
-  ugb_pdl_trigger();
-  ugb_pdl_wait();
+  __shared__ float sc[4][16][KT + 8];                      // [latent quarter][head][key]; the pitch keeps 8-byte reads conflict-free
+  __shared__ float2 ml[16];                                // (max, sum) of this slice per head
+  __shared__ float fac[16][UGB_LATENT_MAX_SPLITS];         // weight of a slice's sums, gate and 1 / sum included
+  if (!p.early) { ugb_pdl_wait(); ugb_pdl_trigger(); }
   const int sp = blockIdx.x, hg = blockIdx.y, r = blockIdx.z, b = r / p.t;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, tq = lane & 3;
   constexpr int LD = NT * 64;
   const int head0 = hg * 16, n_heads = min(16, p.heads - head0);
   const int T = keys_of(p, r);
-  if (T == 0) return;                                      // the whole grid row leaves: no counter is touched
+  if (T == 0) {                                            // the whole cluster leaves
+    if (p.early) { ugb_pdl_wait(); ugb_pdl_trigger(); }
+    return;
+  }
   const int n_tiles = (T + KT - 1) / KT, per = (n_tiles + p.splits - 1) / p.splits;
   const int tile0 = sp * per, tile1 = min(n_tiles, tile0 + per);
   const __nv_bfloat16 *cache = (const __nv_bfloat16 *)p.cache + (size_t)b * p.t_max * LD;
@@ -95,17 +99,24 @@ latent_attention_mma_kernel(Params p) {
     }
     cp_async_commit();
   };
+  // early: only the newest position's row (in the last tile) comes from a kernel that may still be running
+  const int pre = p.early ? max(0, min(R::STAGES - 1, n_tiles - 1 - tile0)) : 0;
 #pragma unroll
-  for (int s = 0; s < R::STAGES - 1; ++s) issue(tile0 + s);
+  for (int s = 0; s < R::STAGES - 1; ++s)
+    if (s < pre) issue(tile0 + s);
+  if (p.early) { ugb_pdl_wait(); ugb_pdl_trigger(); }
+#pragma unroll
+  for (int s = 0; s < R::STAGES - 1; ++s)
+    if (s >= pre) issue(tile0 + s);
 
-  // queries of this warp's half of the latent: A fragments, rows = heads g and g + 8
-  const int half = warp >> 2, nt = warp & 3;
-  uint32_t qa[2 * NT][4];
+  // queries of this warp's quarter of the latent: A fragments, rows = heads g and g + 8
+  const int quarter = warp >> 1, kp = warp & 1;
+  uint32_t qa[NT][4];
   {
-    const __nv_bfloat16 *q = (const __nv_bfloat16 *)p.q + ((size_t)r * p.heads + head0) * LD + half * (LD / 2);
+    const __nv_bfloat16 *q = (const __nv_bfloat16 *)p.q + ((size_t)r * p.heads + head0) * LD + quarter * (LD / 4);
     auto ld2 = [&](int h, int col) -> uint32_t { return h < n_heads ? *reinterpret_cast<const uint32_t *>(q + (size_t)h * LD + col) : 0u; };
 #pragma unroll
-    for (int k = 0; k < 2 * NT; ++k) {
+    for (int k = 0; k < NT; ++k) {
       qa[k][0] = ld2(g, 16 * k + 2 * tq);
       qa[k][1] = ld2(g + 8, 16 * k + 2 * tq);
       qa[k][2] = ld2(g, 16 * k + 8 + 2 * tq);
@@ -116,19 +127,34 @@ latent_attention_mma_kernel(Params p) {
   auto scores = [&](int tile) {
     const uint32_t base = ring_u + (uint32_t)((tile - tile0) % R::STAGES) * R::TILE;
     float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f};
+    const int key = 16 * kp + 8 * (mi >> 1) + ri;
+    const uint32_t row = base + key * R::ROW;
+    constexpr int G = NT < 4 ? NT : 4;                     // operand loads issued ahead of their products
 #pragma unroll
-    for (int k = 0; k < NT; ++k) {                         // two k steps of 16 per ldmatrix.x4
-      const int key = 8 * nt + ri, ch = half * (NT * 4) + 4 * k + mi;
-      uint32_t b0, b1, b2, b3;
-      asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-                   : "=r"(b0), "=r"(b1), "=r"(b2), "=r"(b3)
-                   : "r"(base + key * R::ROW + (((ch & ~7) | ((ch ^ key) & 7)) << 4)));
-      mma_bf16_16x8x16(s0, qa[2 * k][0], qa[2 * k][1], qa[2 * k][2], qa[2 * k][3], b0, b1);
-      mma_bf16_16x8x16(s1, qa[2 * k + 1][0], qa[2 * k + 1][1], qa[2 * k + 1][2], qa[2 * k + 1][3], b2, b3);
+    for (int k0 = 0; k0 < NT; k0 += G) {
+      uint32_t bf[G][4];
+#pragma unroll
+      for (int k = 0; k < G; ++k) {
+        if (k0 + k >= NT) continue;
+        const int ch = quarter * (NT * 2) + 2 * (k0 + k) + (mi & 1);
+        asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+                     : "=r"(bf[k][0]), "=r"(bf[k][1]), "=r"(bf[k][2]), "=r"(bf[k][3])
+                     : "r"(row + (((ch & ~7) | ((ch ^ key) & 7)) << 4)));
+      }
+#pragma unroll
+      for (int k = 0; k < G; ++k) {
+        if (k0 + k >= NT) continue;
+        const uint32_t (&a)[4] = qa[k0 + k];
+        mma_bf16_16x8x16(s0, a[0], a[1], a[2], a[3], bf[k][0], bf[k][1]);
+        mma_bf16_16x8x16(s1, a[0], a[1], a[2], a[3], bf[k][2], bf[k][3]);
+      }
     }
-    float (*dst)[KT + 2] = sc[(tile - tile0) & 1][half];
-    *reinterpret_cast<float2 *>(&dst[g][8 * nt + 2 * tq]) = make_float2(s0[0] + s1[0], s0[1] + s1[1]);
-    *reinterpret_cast<float2 *>(&dst[g + 8][8 * nt + 2 * tq]) = make_float2(s0[2] + s1[2], s0[3] + s1[3]);
+    float (*dst)[KT + 8] = sc[quarter];
+#pragma unroll
+    for (int rr = 0; rr < 2; ++rr) {
+      *reinterpret_cast<float2 *>(&dst[g + 8 * rr][16 * kp + 2 * tq]) = make_float2(s0[2 * rr], s0[2 * rr + 1]);
+      *reinterpret_cast<float2 *>(&dst[g + 8 * rr][16 * kp + 8 + 2 * tq]) = make_float2(s1[2 * rr], s1[2 * rr + 1]);
+    }
   };
 
   const float scl = p.scale * 1.4426950408889634f;
@@ -138,18 +164,13 @@ latent_attention_mma_kernel(Params p) {
   for (int d = 0; d < NT; ++d) o[d][0] = o[d][1] = o[d][2] = o[d][3] = 0.f;
   const int chunk0 = warp * NT;                            // first 16-byte chunk of this warp's columns
 
-  if (tile0 < tile1) {
+  for (int j = tile0; j < tile1; ++j) {
+    // tile j has landed, and nobody works on tile j - 1 any more
     asm volatile("cp.async.wait_group %0;" ::"n"(R::STAGES - 2) : "memory");
     __syncthreads();
-    scores(tile0);
-  }
-  for (int j = tile0; j < tile1; ++j) {
-    // tile j + 1 has landed, the scores of tile j are visible, nobody reads tile j - 1 any more
-    asm volatile("cp.async.wait_group %0;" ::"n"(R::STAGES - 3) : "memory");
-    __syncthreads();
     issue(j + R::STAGES - 1);
-    if (j + 1 < tile1) scores(j + 1);
-    const float (*s0)[KT + 2] = sc[(j - tile0) & 1][0], (*s1)[KT + 2] = sc[(j - tile0) & 1][1];
+    scores(j);
+    __syncthreads();
     uint32_t pa[2][4];
 #pragma unroll
     for (int rr = 0; rr < 2; ++rr) {
@@ -158,11 +179,12 @@ latent_attention_mma_kernel(Params p) {
       float mx = -INFINITY;
 #pragma unroll
       for (int e = 0; e < 4; ++e) {                        // keys 8 e + 2 tq, + 1
-        const float2 x = *reinterpret_cast<const float2 *>(&s0[row][8 * e + 2 * tq]);
-        const float2 y = *reinterpret_cast<const float2 *>(&s1[row][8 * e + 2 * tq]);
+        float2 x[4];
+#pragma unroll
+        for (int q = 0; q < 4; ++q) x[q] = *reinterpret_cast<const float2 *>(&sc[q][row][8 * e + 2 * tq]);
         const int key = j * KT + 8 * e + 2 * tq;
-        f[2 * e] = key < T ? (x.x + y.x) * scl : -INFINITY;
-        f[2 * e + 1] = key + 1 < T ? (x.y + y.y) * scl : -INFINITY;
+        f[2 * e] = key < T ? ((x[0].x + x[1].x) + (x[2].x + x[3].x)) * scl : -INFINITY;
+        f[2 * e + 1] = key + 1 < T ? ((x[0].y + x[1].y) + (x[2].y + x[3].y)) * scl : -INFINITY;
         mx = fmaxf(mx, fmaxf(f[2 * e], f[2 * e + 1]));
       }
       mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
@@ -184,15 +206,18 @@ latent_attention_mma_kernel(Params p) {
     for (int kk = 0; kk < 2; ++kk) {
       const int key = 16 * kk + ri + 8 * (mi & 1);
       if constexpr (NT % 2 == 0) {
+        uint32_t bf[NT / 2][4];
 #pragma unroll
-        for (int d = 0; d < NT; d += 2) {
-          const int ch = chunk0 + d + (mi >> 1);
-          uint32_t b0, b1, b2, b3;
+        for (int d = 0; d < NT / 2; ++d) {
+          const int ch = chunk0 + 2 * d + (mi >> 1);
           asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-                       : "=r"(b0), "=r"(b1), "=r"(b2), "=r"(b3)
+                       : "=r"(bf[d][0]), "=r"(bf[d][1]), "=r"(bf[d][2]), "=r"(bf[d][3])
                        : "r"(base + key * R::ROW + (((ch & ~7) | ((ch ^ key) & 7)) << 4)));
-          mma_bf16_16x8x16(o[d], pa[kk][0], pa[kk][1], pa[kk][2], pa[kk][3], b0, b1);
-          mma_bf16_16x8x16(o[d + 1], pa[kk][0], pa[kk][1], pa[kk][2], pa[kk][3], b2, b3);
+        }
+#pragma unroll
+        for (int d = 0; d < NT / 2; ++d) {
+          mma_bf16_16x8x16(o[2 * d], pa[kk][0], pa[kk][1], pa[kk][2], pa[kk][3], bf[d][0], bf[d][1]);
+          mma_bf16_16x8x16(o[2 * d + 1], pa[kk][0], pa[kk][1], pa[kk][2], pa[kk][3], bf[d][2], bf[d][3]);
         }
       } else {
 #pragma unroll
@@ -225,61 +250,62 @@ latent_attention_mma_kernel(Params p) {
     }
     return;
   }
-  const size_t group = (size_t)r * gridDim.y + hg, slot = group * p.splits + sp;
+  // The slices of a (row, head group) are the CTAs of one cluster.  Every slice leaves its sums and its (max, sum) in its
+  // own shared memory (the ring is idle now); after one cluster barrier each CTA combines its share of the elements,
+  // in slice order, reading the peers' shared memory.
+  __syncthreads();
+  float *os = reinterpret_cast<float *>(ring);             // [16][LD], exactly one ring stage
 #pragma unroll
   for (int rr = 0; rr < 2; ++rr) {
-    const int h = g + 8 * rr;
-    if (h >= n_heads) continue;
-    float *po = p.part_o + (slot * 16 + h) * LD;
+    float *po = os + (g + 8 * rr) * LD;
 #pragma unroll
     for (int d = 0; d < NT; ++d) *reinterpret_cast<float2 *>(po + (chunk0 + d) * 8 + 2 * tq) = make_float2(o[d][2 * rr], o[d][2 * rr + 1]);
-    if (warp == 0 && tq == 0) { p.part_ml[(slot * 16 + h) * 2] = m[rr]; p.part_ml[(slot * 16 + h) * 2 + 1] = l[rr]; }
+    if (warp == 0 && tq == 0) ml[g + 8 * rr] = make_float2(m[rr], l[rr]);
   }
-  __threadfence();
-  __syncthreads();
-  if (threadIdx.x == 0) {
-    const unsigned prev = atomicAdd(&p.counters[group], 1u);
-    is_last = prev == (unsigned)p.splits - 1u;
-    if (is_last) p.counters[group] = 0u;                   // ready for the next launch
-  }
-  __syncthreads();
-  if (!is_last) return;
-  __threadfence();
-  // the last slice to finish combines all of them in slice order; every partial of an element is requested before the
-  // first is used
-  float *fac = reinterpret_cast<float *>(ring);            // [16][splits]: weight of a slice, gate and 1 / l included
-  for (int h = threadIdx.x; h < n_heads; h += WARPS * 32) {
+  cluster_sync_all();
+  if (threadIdx.x < 16) {
+    const int h = threadIdx.x;
+    const uint32_t addr = smem_u32(&ml[h]);
+    float2 v[UGB_LATENT_MAX_SPLITS];
     float mm = -INFINITY;
-    for (int s = 0; s < p.splits; ++s) mm = fmaxf(mm, __ldcg(&p.part_ml[((group * p.splits + s) * 16 + h) * 2]));
-    float ll = 0.f;
-    for (int s = 0; s < p.splits; ++s) {
-      const float ms = __ldcg(&p.part_ml[((group * p.splits + s) * 16 + h) * 2]);
-      const float f = ms == -INFINITY ? 0.f : ex2(ms - mm);
-      fac[h * UGB_LATENT_MAX_SPLITS + s] = f;
-      ll += f * __ldcg(&p.part_ml[((group * p.splits + s) * 16 + h) * 2 + 1]);
+#pragma unroll
+    for (int s = 0; s < UGB_LATENT_MAX_SPLITS; ++s) {
+      v[s] = make_float2(-INFINITY, 0.f);
+      if (s < p.splits)
+        asm volatile("ld.shared::cluster.v2.f32 {%0, %1}, [%2];" : "=f"(v[s].x), "=f"(v[s].y) : "r"(mapa_u32(addr, (uint32_t)s)) : "memory");
     }
-    const float k = (p.gate ? p.gate[(size_t)r * p.gate_ld + head0 + h] : 1.f) / ll;
-    for (int s = 0; s < p.splits; ++s) fac[h * UGB_LATENT_MAX_SPLITS + s] *= k;
+#pragma unroll
+    for (int s = 0; s < UGB_LATENT_MAX_SPLITS; ++s) mm = fmaxf(mm, v[s].x);
+    float ll = 0.f;
+#pragma unroll
+    for (int s = 0; s < UGB_LATENT_MAX_SPLITS; ++s) {
+      v[s].x = v[s].x == -INFINITY ? 0.f : ex2(v[s].x - mm);
+      ll += v[s].x * v[s].y;
+    }
+    const float k = h < n_heads ? (p.gate ? p.gate[(size_t)r * p.gate_ld + head0 + h] : 1.f) / ll : 0.f;
+#pragma unroll
+    for (int s = 0; s < UGB_LATENT_MAX_SPLITS; ++s) fac[h][s] = v[s].x * k;
   }
   __syncthreads();
-  for (int idx = threadIdx.x; idx < n_heads * (LD / 4); idx += WARPS * 32) {
+  for (int idx = sp * (WARPS * 32) + threadIdx.x; idx < n_heads * (LD / 4); idx += p.splits * (WARPS * 32)) {
     const int h = idx / (LD / 4), c = (idx % (LD / 4)) * 4;
-    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
-    for (int s0 = 0; s0 < p.splits; s0 += 4) {
-      float4 v[4];
+    const uint32_t addr = smem_u32(os + h * LD + c);
+    float4 v[UGB_LATENT_MAX_SPLITS], acc = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        v[e] = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (s0 + e < p.splits) v[e] = __ldcg(reinterpret_cast<const float4 *>(p.part_o + ((group * p.splits + s0 + e) * 16 + h) * LD + c));
-      }
+    for (int s = 0; s < UGB_LATENT_MAX_SPLITS; ++s) {
+      v[s] = acc;
+      if (s < p.splits)
+        asm volatile("ld.shared::cluster.v4.f32 {%0, %1, %2, %3}, [%4];"
+                     : "=f"(v[s].x), "=f"(v[s].y), "=f"(v[s].z), "=f"(v[s].w) : "r"(mapa_u32(addr, (uint32_t)s)) : "memory");
+    }
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const float f = s0 + e < p.splits ? fac[h * UGB_LATENT_MAX_SPLITS + s0 + e] : 0.f;
-        acc.x = fmaf(f, v[e].x, acc.x); acc.y = fmaf(f, v[e].y, acc.y); acc.z = fmaf(f, v[e].z, acc.z); acc.w = fmaf(f, v[e].w, acc.w);
-      }
+    for (int s = 0; s < UGB_LATENT_MAX_SPLITS; ++s) {
+      const float f = s < p.splits ? fac[h][s] : 0.f;
+      acc.x = fmaf(f, v[s].x, acc.x); acc.y = fmaf(f, v[s].y, acc.y); acc.z = fmaf(f, v[s].z, acc.z); acc.w = fmaf(f, v[s].w, acc.w);
     }
     *reinterpret_cast<uint2 *>(out + (size_t)h * LD + c) = make_uint2(pack_bf16(acc.x, acc.y), pack_bf16(acc.z, acc.w));
   }
+  cluster_sync_all();                                      // no CTA leaves while a peer may still read its shared memory
 }
 
 // ------------------------------------------------------------- generic ------
@@ -291,8 +317,8 @@ latent_attention_generic_kernel(Params p, int kt) {
   extern __shared__ float gsm[];
   const int ld = p.ld, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   float *qs = gsm, *os = qs + 8 * ld, *ks = os + 8 * ld;
-  ugb_pdl_trigger();
   ugb_pdl_wait();
+  ugb_pdl_trigger();
   const int r = blockIdx.x, head = blockIdx.y * 8 + warp, b = r / p.t;
   const bool on = head < p.heads;
   const int n = keys_of(p, r);
@@ -356,7 +382,7 @@ template <int NT> int32_t prepare_one(ugb_device *dev) {
   return UGB_OK;
 }
 template <int NT> cudaError_t launch_one(dim3 grid, cudaStream_t st, bool pdl, const Params &p) {
-  return ugb_launch(latent_attention_mma_kernel<NT>, grid, dim3(WARPS * 32), Ring<NT>::BYTES, st, pdl, p);
+  return ugb_launch_cluster(latent_attention_mma_kernel<NT>, grid, dim3(WARPS * 32), Ring<NT>::BYTES, st, pdl, p.splits, p);
 }
 
 }  // namespace
@@ -366,10 +392,6 @@ int ugb_latent_row_width(int rank) {
     if (rank <= nt * 64) return nt * 64;
   return 0;
 }
-size_t ugb_latent_scratch_o(int rows, int heads, int ld, int splits) {
-  return (size_t)rows * ((heads + 15) / 16) * splits * 16 * ld;
-}
-size_t ugb_latent_scratch_ml(int rows, int heads, int splits) { return (size_t)rows * ((heads + 15) / 16) * splits * 16 * 2; }
 
 int32_t ugb_latent_attention_prepare(ugb_device *dev) {
   int32_t rc;
@@ -386,7 +408,7 @@ int32_t ugb_latent_attention(ugb_device *dev, const ugb_latent_attention_args &a
   Params p;
   p.q = a.q; p.cache = a.cache; p.out = a.out; p.gate = a.gate; p.t = a.t; p.pos_off = a.pos_off; p.heads = a.heads;
   p.ld = a.ld; p.t_max = a.t_max; p.gate_ld = a.gate_ld; p.splits = a.splits; p.pos_p = a.pos_p; p.scale = a.scale;
-  p.part_o = a.part_o; p.part_ml = a.part_ml; p.counters = a.counters; p.status = dev->status_dev;
+  p.early = a.early && a.pdl ? 1 : 0; p.status = dev->status_dev;
   cudaError_t e;
   if (!a.f32 && ugb_latent_row_width(a.ld) == a.ld) {
     UGB_REQUIRE(dev, a.splits >= 1 && a.splits <= UGB_LATENT_MAX_SPLITS, UGB_ERR_INVALID, "latent attention: %d slices", a.splits);

@@ -18,17 +18,14 @@ struct ugb_latent_attention_args {
   int heads, ld, t_max, gate_ld;
   float scale;
   int splits;              // slices of the cached positions per row that run as separate CTAs (bf16 fast path)
-  float *part_o, *part_ml; // scratch of the slices: ugb_latent_attention_scratch elements each
-  unsigned *counters;      // zeroed, one per (row, group of 16 heads)
   bool pdl;
+  bool early;              // with pdl, t == 1: the position and every cache row but the newest were written by kernels that
+                           // are complete when this one starts, and may be read before the wait for the preceding one
 };
 
 // Row width (elements) the bf16 fast path wants for a latent of `rank` values, or 0 when it has no kernel for it.
 int ugb_latent_row_width(int rank);
-constexpr int UGB_LATENT_MAX_SPLITS = 16;
-// Elements of part_o / part_ml for `rows` rows.
-size_t ugb_latent_scratch_o(int rows, int heads, int ld, int splits);
-size_t ugb_latent_scratch_ml(int rows, int heads, int splits);
+constexpr int UGB_LATENT_MAX_SPLITS = 8;   // CTAs of a cluster
 // Sets the kernels' shared-memory attributes (must not happen inside a stream capture).
 int32_t ugb_latent_attention_prepare(ugb_device *dev);
 int32_t ugb_latent_attention(ugb_device *dev, const ugb_latent_attention_args &a);
