@@ -29,8 +29,9 @@ def _stale(out, deps):
     return any(os.path.getmtime(d) > t for d in deps)
 
 
-def build(force=False, verbose=False):
-    """Compile and link; returns the path of the shared library."""
+def build(force=False, verbose=False, host=True):
+    """Compile and link; returns the path of the shared library.  ``host=False`` leaves the host layer
+    (libughost.so: lazy graph, scheduler) out: the fused engines do not use it."""
     os.makedirs(OBJ, exist_ok=True)
     srcs = sorted(glob.glob(os.path.join(CSRC, "*.cu")))
     hdrs = glob.glob(os.path.join(CSRC, "*.h")) + glob.glob(os.path.join(CSRC, "*.cuh")) + \
@@ -63,7 +64,8 @@ def build(force=False, verbose=False):
             raise RuntimeError(f"link failed:\n{r.stdout}\n{r.stderr}")
         if verbose:
             print(f"linked {LIB}")
-    build_host(force=force or bool(jobs), verbose=verbose)
+    if host:
+        build_host(force=force or bool(jobs), verbose=verbose)
     return LIB
 
 

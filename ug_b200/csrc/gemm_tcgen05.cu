@@ -554,7 +554,8 @@ tc_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
             const int col0 = pair_n0 + c * 32;
             // out [M, N/2] bf16 = silu(gate) * up over the summed (gate, up) column pairs
             __nv_bfloat16 *crow = (__nv_bfloat16 *)p.C + (long long)row * p.c_ld + col0 / 2;
-            if (p.epi == UGB_EPI_RELU2_BF16) {                      // out [M, N] bf16 = max(sum, 0)^2
+            if (p.epi != UGB_EPI_SILU_MUL_BF16) {                   // out [M, N] bf16 = sum, or max(sum, 0)^2
+              const bool relu2 = p.epi == UGB_EPI_RELU2_BF16;
               __nv_bfloat16 *frow = (__nv_bfloat16 *)p.C + (long long)row * p.c_ld + col0;
 #pragma unroll
               for (int q = 0; q < 4; ++q) {
@@ -565,9 +566,10 @@ tc_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
                   uint32_t o[4];
 #pragma unroll
                   for (int e = 0; e < 4; ++e) {
-                    const float s0 = fmaxf(__uint_as_float(v[q * 8 + 2 * e]) + wv[2 * e], 0.f);
-                    const float s1 = fmaxf(__uint_as_float(v[q * 8 + 2 * e + 1]) + wv[2 * e + 1], 0.f);
-                    __nv_bfloat162 t = __floats2bfloat162_rn(s0 * s0, s1 * s1);
+                    float s0 = __uint_as_float(v[q * 8 + 2 * e]) + wv[2 * e];
+                    float s1 = __uint_as_float(v[q * 8 + 2 * e + 1]) + wv[2 * e + 1];
+                    if (relu2) { s0 = fmaxf(s0, 0.f); s1 = fmaxf(s1, 0.f); s0 *= s0; s1 *= s1; }
+                    __nv_bfloat162 t = __floats2bfloat162_rn(s0, s1);
                     o[e] = *(uint32_t *)&t;
                   }
                   *reinterpret_cast<uint4 *>(frow + q * 8) = make_uint4(o[0], o[1], o[2], o[3]);
@@ -691,7 +693,7 @@ int32_t launch_tc(ugb_device *dev, TcState *st, const ugb_tc_gemm_args &g, size_
   p.pair_k = 0;
   if (g.pair_k) {
     // two CTAs (a cluster) per tile, each over half of k
-    if (!C_::PAIR_K_OK || (g.epi != UGB_EPI_SILU_MUL_BF16 && g.epi != UGB_EPI_RELU2_BF16) || batch != 1 || p.k_blocks < 2 ||
+    if (!C_::PAIR_K_OK || (g.epi != UGB_EPI_SILU_MUL_BF16 && g.epi != UGB_EPI_RELU2_BF16 && g.epi != UGB_EPI_BF16) || g.f16 || batch != 1 || p.k_blocks < 2 ||
         2 * (long long)p.tiles_m * p.tiles_n > dev->sm_count)
       return UGB_ERR_UNSUPPORTED;
     p.pair_k = 1;

@@ -51,7 +51,7 @@ struct ugb_tc_gemm_args {
                                // ahead of its own wait
   int smem_kib = 0;     // cap on the shared memory of a CTA (ring depth follows); 0 = as deep as fits in 220 KiB
   bool f16 = false;     // operands (and the UGB_EPI_BF16 output) are IEEE f16 instead of bf16: same instruction, other format field
-  bool pair_k = false;  // m <= 64, UGB_EPI_SILU_MUL_BF16 or UGB_EPI_RELU2_BF16: two CTAs (a thread-block cluster) per tile, each over half of k; the
+  bool pair_k = false;  // m <= 64, an epilogue that writes bf16 columns: two CTAs (a thread-block cluster) per tile, each over half of k; the
                         // second hands its sums to the first through distributed shared memory.  UGB_ERR_UNSUPPORTED when
                         // twice the tiles exceed the SMs
   unsigned long long *prof = nullptr;   // measurement aid, see UGB_TC_PROF_*

@@ -136,8 +136,8 @@ int32_t matmul(ugb_hybrid *m, const Mat &x) {
   g.epi = x.relu2 ? UGB_EPI_RELU2_BF16 : (x.f32_out ? UGB_EPI_F32 : UGB_EPI_BF16);
   g.splits = x.splits; g.bn = x.bn; g.b_static = true; g.pdl = m->pdl != 0; g.late_trigger = true;
   g.smem_kib = x.m <= 64 ? 144 : 0;
-  if (x.relu2 && x.m <= 64) {
-    // the two k halves of a tile on a pair of CTAs, with the narrowest tile that fits the SMs
+  if (!x.f32_out && x.batch == 1 && x.nk && x.m <= 64 && x.k >= 256) {
+    // a T result cannot be split into partials: the two k halves of a tile on a pair of CTAs, with the narrowest tile that fits the SMs
     for (int bn : {64, 96, 128, 160})
       if ((x.n + bn - 1) / bn * 2 <= (size_t)dev->sm_count) {
         g.bn = bn;
@@ -296,7 +296,10 @@ int32_t run_layers(ugb_hybrid *m, Work &w, const int *tok, int t_block, int off,
         if ((rc = matmul(m, g))) return rc;
       }
       if (m->on(UGB_HYBRID_K_LATENT_ROWS)) {
-        e = ugb_launch(latent_inputs_kernel<T>, dim3(rows), dim3(256), (size_t)n_in * 4, st, pdl, w.pre, ti.splits, (size_t)rows * n_in,
+        const int threads = decode ? 512 : 256, per = (n_in / 4 + threads - 1) / threads;
+        auto *k = decode ? (per <= 1 ? latent_inputs_kernel<T, 1, 8> : per <= 2 ? latent_inputs_kernel<T, 2, 8> : latent_inputs_kernel<T, 16, 1>)
+                         : (per <= 2 ? latent_inputs_kernel<T, 2, 1> : per <= 4 ? latent_inputs_kernel<T, 4, 1> : latent_inputs_kernel<T, 16, 1>);
+        e = ugb_launch(k, dim3(rows), dim3(threads), 0, st, pdl, w.pre, ti.splits, (size_t)rows * n_in,
                        L.q_gain, L.c_gain, (T *)w.cq, (T *)L.cache, w.gate, m->pos, off, t, m->t_max, L.ql, L.cl, L.gl,
                        1.0f / (float)L.d.q_rank, 1.0f / (float)L.d.kv_rank, m->cfg.eps, dev->status_dev);
         if (e != cudaSuccess) return ugb_fail(dev, UGB_ERR_CUDA, "launch of latent_inputs_kernel failed: %s", cudaGetErrorString(e));
@@ -587,7 +590,7 @@ int32_t ugb_hybrid_create(ugb_device *dev, const ugb_hybrid_config *cfg, const u
       L.expand = !m->f32 && dp && vp && d.scale > 0.f;
       L.dp = L.expand ? dp : (int)up8(d.dim);
       L.vp = L.expand ? vp : (int)up8(d.vdim);
-      CHECK((size_t)(L.ql + L.cl + L.gl) * 4 <= 48 * 1024 - 64, UGB_ERR_UNSUPPORTED, "layer %d: latents of %d + %d values", i, d.q_rank, d.kv_rank);
+      CHECK(L.ql + L.cl + L.gl <= 16 * 4 * 256, UGB_ERR_UNSUPPORTED, "layer %d: latents of %d + %d values", i, d.q_rank, d.kv_rank);
       TRY(alloc_bytes(m, &L.w_in, (size_t)(L.ql + L.cl + L.gl) * wl * es, true));
       TRY(alloc_bytes(m, &L.w_uq, (size_t)d.heads * L.dp * L.ql * es, true));
       TRY(alloc_bytes(m, &L.w_uk, (size_t)d.heads * L.dp * L.cl * es, true));

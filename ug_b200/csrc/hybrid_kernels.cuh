@@ -33,15 +33,19 @@ template <> struct Act<__nv_bfloat16> {
   static __device__ __forceinline__ float round(float v) { return __bfloat162float(__float2bfloat16_rn(v)); }
 };
 
-// Gate functions in fp32; EXACT: correctly rounded division and full-precision exp (models that run in 32 bits), otherwise
-// the hardware's exp2 and reciprocal (about 1e-6 relative), which the block scan of a bf16 model is bound by.
-template <bool EXACT> __device__ __forceinline__ float over_1_exp(float num, float x) {   // num / (1 + e^-x)
-  return EXACT ? num / (1.0f + expf(-x)) : __fdividef(num, 1.0f + __expf(-x));
+// Gate functions in fp32; EXACT: correctly rounded division and full-precision exp, otherwise the hardware's exp2 and
+// reciprocal (about 1e-6 relative): the block scan of a bf16 model is bound by the instructions of its gates.
+template <bool EXACT> __device__ __forceinline__ float sigmoid_t(float x) {
+  if constexpr (EXACT) return 1.0f / (1.0f + expf(-x));
+  float e, r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(x * -1.4426950408889634f));
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));   // e = inf gives 0
+  return r;
 }
-__device__ __forceinline__ float sigmoid_f(float x) { return over_1_exp<true>(1.0f, x); }
-__device__ __forceinline__ float silu_f(float x) { return over_1_exp<true>(x, x); }
+__device__ __forceinline__ float sigmoid_f(float x) { return sigmoid_t<true>(x); }
+__device__ __forceinline__ float silu_f(float x) { return x / (1.0f + expf(-x)); }
 // candidate of the minimal gated recurrent unit: u + 1/2 for u >= 0, sigmoid(u) below
-template <bool EXACT> __device__ __forceinline__ float gru_candidate(float u) { return u >= 0.0f ? u + 0.5f : over_1_exp<EXACT>(1.0f, u); }
+template <bool EXACT> __device__ __forceinline__ float gru_candidate(float u) { return u >= 0.0f ? u + 0.5f : sigmoid_t<EXACT>(u); }
 
 __device__ __forceinline__ float block_sum_256(float v, float *sm) {   // sm: 8 floats; all 256 threads
 #pragma unroll
@@ -441,7 +445,8 @@ min_gru_scan_kernel(const TI *__restrict__ pre, const float *__restrict__ bz, co
   constexpr bool EXACT = sizeof(T) == 4;
   __shared__ float agg_a[SCAN_WARPS][COLS], agg_b[SCAN_WARPS][COLS];
   __shared__ float tot[2][2][COLS];                        // [round parity][A, B][channel], read by the cluster
-  __shared__ float enter[COLS], carry[COLS];               // state entering this CTA's piece, state before the round
+  __shared__ float enter[SCAN_WARPS][COLS];                // state entering each warp's positions
+  __shared__ float carry[COLS];                            // state before the round
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int rank = blockIdx.x, n_cta = gridDim.x, b = blockIdx.z;
   const int c = blockIdx.y * COLS + lane * V;              // ld is a multiple of 8: a lane's channels are all in or all out
@@ -457,13 +462,14 @@ min_gru_scan_kernel(const TI *__restrict__ pre, const float *__restrict__ bz, co
     carry[threadIdx.x] = k < ld ? state[(size_t)b * ld + k] : 0.f;
   }
   const size_t base = (size_t)b * t;
+  const TI *mine = pre + base * (size_t)(3 * ld) + c;
   uint32_t nz[STEPS], nu[STEPS], ng[STEPS];                // the coming round's rows, requested a round ahead
   auto fetch = [&](int i0) {
 #pragma unroll
     for (int s = 0; s < STEPS; ++s) {
       nz[s] = nu[s] = ng[s] = 0u;
       if (on && i0 + s < t) {
-        const TI *row = pre + (base + i0 + s) * (size_t)(3 * ld) + c;
+        const TI *row = mine + (size_t)(i0 + s) * (3 * ld);
         nz[s] = __ldcs(reinterpret_cast<const uint32_t *>(row));
         nu[s] = __ldcs(reinterpret_cast<const uint32_t *>(row + ld));
         ng[s] = __ldcs(reinterpret_cast<const uint32_t *>(row + 2 * ld));
@@ -474,6 +480,7 @@ min_gru_scan_kernel(const TI *__restrict__ pre, const float *__restrict__ bz, co
   int round = 0;
   for (int t0 = 0; t0 < t; t0 += BLOCK * n_cta, ++round) {
     const int i0 = t0 + rank * BLOCK + warp * STEPS;
+    const bool whole = i0 + STEPS <= t;
     float a[STEPS][V], bb[STEPS][V], sg[STEPS][V];
 #pragma unroll
     for (int s = 0; s < STEPS; ++s) { scan_widen<V>(nz[s], a[s]); scan_widen<V>(nu[s], bb[s]); scan_widen<V>(ng[s], sg[s]); }
@@ -484,15 +491,15 @@ min_gru_scan_kernel(const TI *__restrict__ pre, const float *__restrict__ bz, co
       A[e] = 1.f; B[e] = 0.f;
 #pragma unroll
       for (int s = 0; s < STEPS; ++s) {
-        if (on && i0 + s < t) {
-          const float z = over_1_exp<EXACT>(1.0f, a[s][e] + zb[e]);
-          a[s][e] = 1.0f - z;
-          bb[s][e] = z * gru_candidate<EXACT>(bb[s][e] + ub[e]);
-          sg[s][e] = over_1_exp<EXACT>(sg[s][e], sg[s][e]);
-        } else { a[s][e] = 1.f; bb[s][e] = 0.f; sg[s][e] = 0.f; }
+        const float z = sigmoid_t<EXACT>(a[s][e] + zb[e]);
+        const bool live = whole || i0 + s < t;             // positions behind the block leave the state alone
+        a[s][e] = live ? 1.0f - z : 1.0f;
+        bb[s][e] = live ? z * gru_candidate<EXACT>(bb[s][e] + ub[e]) : 0.0f;
+        sg[s][e] = sg[s][e] * sigmoid_t<EXACT>(sg[s][e]);
         A[e] *= a[s][e];
         B[e] = fmaf(a[s][e], B[e], bb[s][e]);
       }
+      // (the round before has left these arrays: all read them before its last barrier)
       agg_a[warp][lane * V + e] = A[e]; agg_b[warp][lane * V + e] = B[e];
     }
     __syncthreads();
@@ -523,20 +530,21 @@ min_gru_scan_kernel(const TI *__restrict__ pre, const float *__restrict__ bz, co
         R = fmaf(va[q], R, vb[q]);
       }
       carry[threadIdx.x] = R;
-      enter[threadIdx.x] = in;
+#pragma unroll
+      for (int w = 0; w < SCAN_WARPS; ++w) {
+        enter[w][threadIdx.x] = in;
+        in = fmaf(agg_a[w][threadIdx.x], in, agg_b[w][threadIdx.x]);
+      }
     }
     __syncthreads();
     float S[V];
 #pragma unroll
-    for (int e = 0; e < V; ++e) S[e] = enter[lane * V + e];
-    for (int w = 0; w < warp; ++w)
-#pragma unroll
-      for (int e = 0; e < V; ++e) S[e] = fmaf(agg_a[w][lane * V + e], S[e], agg_b[w][lane * V + e]);
+    for (int e = 0; e < V; ++e) S[e] = enter[warp][lane * V + e];
 #pragma unroll
     for (int s = 0; s < STEPS; ++s) {
 #pragma unroll
       for (int e = 0; e < V; ++e) S[e] = fmaf(a[s][e], S[e], bb[s][e]);
-      if (on && i0 + s < t) {
+      if (on && (whole || i0 + s < t)) {
         T *o = out + (base + i0 + s) * (size_t)ld + c;
         if constexpr (sizeof(T) == 4) {
 #pragma unroll
@@ -548,7 +556,6 @@ min_gru_scan_kernel(const TI *__restrict__ pre, const float *__restrict__ bz, co
         }
       }
     }
-    __syncthreads();                                       // agg_a / agg_b are free
   }
   ugb_tc::cluster_sync_all();                              // no CTA leaves (or writes the state) while a peer still reads
   if (rank == 0 && threadIdx.x < COLS) {
@@ -560,41 +567,51 @@ min_gru_scan_kernel(const TI *__restrict__ pre, const float *__restrict__ bz, co
 // ------------------------------------------------- latent attention inputs ---
 // pre [n_part][rows][q_ld + c_ld + g_ld]: query latent, key/value latent and head gates of one projection.
 //   cq[r] = norm(query latent) * q_gain   cache[b][pos] = norm(kv latent) * c_gain   gate[r] = sigmoid(head gate)
-// row r = (b, i) = (r / t, r % t), pos = *pos_p + pos_off + i.  One CTA of 256 threads per row.
-template <typename T>
-__global__ void __launch_bounds__(256)
+// row r = (b, i) = (r / t, r % t), pos = *pos_p + pos_off + i.  One CTA of 256 or 512 threads per row, PER groups of 4
+// columns per thread (the segments are multiples of 8 wide), U split-K partials in flight.
+template <typename T, int PER, int U>
+__global__ void __launch_bounds__(512)
 latent_inputs_kernel(const float *__restrict__ pre, int n_part, size_t part_stride, const float *__restrict__ q_gain,
                      const float *__restrict__ c_gain, T *__restrict__ cq, T *__restrict__ cache, float *__restrict__ gate,
                      const int *__restrict__ pos_p, int pos_off, int t, int t_max, int q_ld, int c_ld, int g_ld,
                      float inv_q, float inv_c, float eps, ugb_status_word *status) {
-  extern __shared__ __align__(16) float row_s[];
-  __shared__ float sm[2][8];
-  const int r = blockIdx.x, n = q_ld + c_ld + g_ld, tid = threadIdx.x;
-  const int b = r / t;
+  __shared__ float sm[2][16];
+  const int r = blockIdx.x, n = q_ld + c_ld + g_ld, tid = threadIdx.x, bd = blockDim.x;
+  const int b = r / t, off = pos_off + r % t;
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  float4 y[PER], w[PER];
+#pragma unroll
+  for (int i = 0; i < PER; ++i) {
+    const int c = 4 * (tid + i * bd);
+    y[i] = w[i] = zero;
+    if (c < q_ld) w[i] = __ldg(reinterpret_cast<const float4 *>(q_gain + c));
+    else if (c < q_ld + c_ld) w[i] = __ldg(reinterpret_cast<const float4 *>(c_gain + c - q_ld));
+  }
   ugb_pdl_wait();
   ugb_pdl_trigger();
-  const int pos = *pos_p + pos_off + r % t;
-  float sq = 0.f, sc = 0.f;
-  for (int c = tid; c < n >> 2; c += 256) {
-    const float *src = pre + (size_t)r * n + 4 * c;
-    float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (n_part == 1) {
-      y = __ldcs(reinterpret_cast<const float4 *>(src));
-    } else {
-      for (int s = 0; s < n_part; s += 8) {               // split-K partials, added in order
-        float4 q[8];
+  const int pos = *pos_p + off;
+  for (int s = 0; s < n_part; s += U) {                    // the partials are added in order
+    float4 q[U][PER];
 #pragma unroll
-        for (int e = 0; e < 8; ++e) {
-          q[e] = make_float4(0.f, 0.f, 0.f, 0.f);
-          if (s + e < n_part) q[e] = __ldcs(reinterpret_cast<const float4 *>(src + (size_t)(s + e) * part_stride));
-        }
+    for (int e = 0; e < U; ++e)
 #pragma unroll
-        for (int e = 0; e < 8; ++e) { y.x += q[e].x; y.y += q[e].y; y.z += q[e].z; y.w += q[e].w; }
+      for (int i = 0; i < PER; ++i) {
+        const int c = tid + i * bd;
+        q[e][i] = zero;
+        if (s + e < n_part && c < n >> 2)
+          q[e][i] = __ldcs(reinterpret_cast<const float4 *>(pre + (size_t)(s + e) * part_stride + (size_t)r * n) + c);
       }
-    }
-    reinterpret_cast<float4 *>(row_s)[c] = y;              // read back by the same thread
-    if (4 * c < q_ld) sq += sq4(y);                        // the segments are multiples of 8 wide
-    else if (4 * c < q_ld + c_ld) sc += sq4(y);
+#pragma unroll
+    for (int e = 0; e < U; ++e)
+#pragma unroll
+      for (int i = 0; i < PER; ++i) { y[i].x += q[e][i].x; y[i].y += q[e][i].y; y[i].z += q[e][i].z; y[i].w += q[e][i].w; }
+  }
+  float sq = 0.f, sc = 0.f;
+#pragma unroll
+  for (int i = 0; i < PER; ++i) {
+    const int c = 4 * (tid + i * bd);
+    if (c < q_ld) sq += sq4(y[i]);
+    else if (c < q_ld + c_ld) sc += sq4(y[i]);
   }
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) {
@@ -604,23 +621,21 @@ latent_inputs_kernel(const float *__restrict__ pre, int n_part, size_t part_stri
   if ((tid & 31) == 0) { sm[0][tid >> 5] = sq; sm[1][tid >> 5] = sc; }
   __syncthreads();
   sq = sc = 0.f;
-#pragma unroll
-  for (int i = 0; i < 8; ++i) { sq += sm[0][i]; sc += sm[1][i]; }
+  for (int i = 0; i < bd >> 5; ++i) { sq += sm[0][i]; sc += sm[1][i]; }
   const float rq = 1.0f / sqrtf(sq * inv_q + eps), rc = 1.0f / sqrtf(sc * inv_c + eps);
   const bool ok = pos >= 0 && pos < t_max;
   if (!ok && tid == 0 && atomicCAS(&status->code, 0u, (unsigned)UGB_ERR_INVALID) == 0u) status->detail = (unsigned)pos;
-  for (int c = tid; c < n >> 2; c += 256) {
-    const float4 y = reinterpret_cast<const float4 *>(row_s)[c];
-    if (4 * c < q_ld) {
-      const float4 w = __ldg(reinterpret_cast<const float4 *>(q_gain) + c);
-      Act<T>::st4(cq + (size_t)r * q_ld + 4 * c, make_float4(y.x * rq * w.x, y.y * rq * w.y, y.z * rq * w.z, y.w * rq * w.w));
-    } else if (4 * c < q_ld + c_ld) {
-      const int k = 4 * c - q_ld;
-      const float4 w = __ldg(reinterpret_cast<const float4 *>(c_gain + k));
-      if (ok) Act<T>::st4(cache + ((size_t)b * t_max + pos) * c_ld + k, make_float4(y.x * rc * w.x, y.y * rc * w.y, y.z * rc * w.z, y.w * rc * w.w));
-    } else {
-      const int k = 4 * c - q_ld - c_ld;
-      *reinterpret_cast<float4 *>(gate + (size_t)r * g_ld + k) = make_float4(sigmoid_f(y.x), sigmoid_f(y.y), sigmoid_f(y.z), sigmoid_f(y.w));
+#pragma unroll
+  for (int i = 0; i < PER; ++i) {
+    const int c = 4 * (tid + i * bd);
+    if (c < q_ld) {
+      Act<T>::st4(cq + (size_t)r * q_ld + c, make_float4(y[i].x * rq * w[i].x, y[i].y * rq * w[i].y, y[i].z * rq * w[i].z, y[i].w * rq * w[i].w));
+    } else if (c < q_ld + c_ld) {
+      if (ok) Act<T>::st4(cache + ((size_t)b * t_max + pos) * c_ld + c - q_ld,
+                          make_float4(y[i].x * rc * w[i].x, y[i].y * rc * w[i].y, y[i].z * rc * w[i].z, y[i].w * rc * w[i].w));
+    } else if (c < n) {
+      *reinterpret_cast<float4 *>(gate + (size_t)r * g_ld + c - q_ld - c_ld) =
+          make_float4(sigmoid_f(y[i].x), sigmoid_f(y[i].y), sigmoid_f(y[i].z), sigmoid_f(y[i].w));
     }
   }
 }

@@ -51,7 +51,7 @@ __device__ __forceinline__ int keys_of(const Params &p, int r) {
 // A 32-key tile lies in shared memory as rows of NT 128-byte pieces, the 16-byte chunks of a piece XORed with the key
 // (the 128-byte swizzle): ldmatrix over 8 keys of one chunk column is conflict-free, plain and transposed.
 //   scores   warp w: keys 16 (w & 1) .. + 15 over quarter w >> 1 of the latent; the quarters meet in shared memory
-//   softmax  every warp for itself, straight in the A-fragment layout of the second product (fp32, online)
+//   softmax  warp w: heads w and w + 8, a lane per key (fp32, online); probabilities to shared memory as bf16
 //   sums     warp w: latent columns 8 NT w .. + 8 NT - 1
 // The ring matters more than the arithmetic: of STAGES tiles one is worked on, the others are in flight.
 constexpr int KT = 32;
@@ -68,7 +68,9 @@ __global__ void __launch_bounds__(WARPS * 32, 2)
 latent_attention_mma_kernel(Params p) {
   using R = Ring<NT>;
   extern __shared__ __align__(128) uint8_t ring[];
-  __shared__ float sc[4][16][KT + 8];                      // [latent quarter][head][key]; the pitch keeps 8-byte reads conflict-free
+  __shared__ float sc[4][16][KT + 8];                      // [latent quarter][head][key]; the pitch keeps 8-byte accesses conflict-free
+  __shared__ __align__(16) __nv_bfloat16 pr[16][KT + 8];   // probabilities; pitch of 80 bytes: conflict-free ldmatrix
+  __shared__ float al[16];                                 // factor the sums so far take on
   __shared__ float2 ml[16];                                // (max, sum) of this slice per head
   __shared__ float fac[16][UGB_LATENT_MAX_SPLITS];         // weight of a slice's sums, gate and 1 / sum included
   if (!p.early) { ugb_pdl_wait(); ugb_pdl_trigger(); }
@@ -158,7 +160,7 @@ latent_attention_mma_kernel(Params p) {
   };
 
   const float scl = p.scale * 1.4426950408889634f;
-  float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+  float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};  // of heads warp and warp + 8; l: this lane's keys
   float o[NT][4];
 #pragma unroll
   for (int d = 0; d < NT; ++d) o[d][0] = o[d][1] = o[d][2] = o[d][3] = 0.f;
@@ -171,36 +173,41 @@ latent_attention_mma_kernel(Params p) {
     issue(j + R::STAGES - 1);
     scores(j);
     __syncthreads();
+    {
+      float f[2], mx[2];
+      const bool seen = j * KT + lane < T;
+#pragma unroll
+      for (int rr = 0; rr < 2; ++rr) {
+        const int row = warp + 8 * rr;
+        f[rr] = seen ? ((sc[0][row][lane] + sc[1][row][lane]) + (sc[2][row][lane] + sc[3][row][lane])) * scl : -INFINITY;
+        mx[rr] = f[rr];
+      }
+#pragma unroll
+      for (int s = 16; s > 0; s >>= 1)
+#pragma unroll
+        for (int rr = 0; rr < 2; ++rr) mx[rr] = fmaxf(mx[rr], __shfl_xor_sync(0xffffffffu, mx[rr], s));
+#pragma unroll
+      for (int rr = 0; rr < 2; ++rr) {
+        const float mn = fmaxf(m[rr], mx[rr]);             // finite: a tile starts below T
+        const float alpha = ex2(m[rr] - mn), pv = ex2(f[rr] - mn);
+        m[rr] = mn;
+        l[rr] = l[rr] * alpha + pv;
+        pr[warp + 8 * rr][lane] = __float2bfloat16_rn(pv);
+        if (lane == 0) al[warp + 8 * rr] = alpha;
+      }
+    }
+    __syncthreads();
+    const float a0 = al[g], a1 = al[g + 8];
+    if (__any_sync(0xffffffffu, a0 != 1.f || a1 != 1.f)) {
+#pragma unroll
+      for (int d = 0; d < NT; ++d) { o[d][0] *= a0; o[d][1] *= a0; o[d][2] *= a1; o[d][3] *= a1; }
+    }
     uint32_t pa[2][4];
 #pragma unroll
-    for (int rr = 0; rr < 2; ++rr) {
-      const int row = g + 8 * rr;
-      float f[8];
-      float mx = -INFINITY;
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {                        // keys 8 e + 2 tq, + 1
-        float2 x[4];
-#pragma unroll
-        for (int q = 0; q < 4; ++q) x[q] = *reinterpret_cast<const float2 *>(&sc[q][row][8 * e + 2 * tq]);
-        const int key = j * KT + 8 * e + 2 * tq;
-        f[2 * e] = key < T ? ((x[0].x + x[1].x) + (x[2].x + x[3].x)) * scl : -INFINITY;
-        f[2 * e + 1] = key + 1 < T ? ((x[0].y + x[1].y) + (x[2].y + x[3].y)) * scl : -INFINITY;
-        mx = fmaxf(mx, fmaxf(f[2 * e], f[2 * e + 1]));
-      }
-      mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
-      mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
-      const float mn = fmaxf(m[rr], mx);                   // finite: a tile starts below T
-      const float alpha = ex2(m[rr] - mn);
-      m[rr] = mn;
-      float sum = 0.f;
-#pragma unroll
-      for (int e = 0; e < 8; ++e) { f[e] = ex2(f[e] - mn); sum += f[e]; }
-      l[rr] = l[rr] * alpha + sum;
-#pragma unroll
-      for (int d = 0; d < NT; ++d) { o[d][2 * rr] *= alpha; o[d][2 * rr + 1] *= alpha; }
-      pa[0][rr] = pack_bf16(f[0], f[1]); pa[0][2 + rr] = pack_bf16(f[2], f[3]);
-      pa[1][rr] = pack_bf16(f[4], f[5]); pa[1][2 + rr] = pack_bf16(f[6], f[7]);
-    }
+    for (int kk = 0; kk < 2; ++kk)                         // rows 0-7, 8-15 of keys 16 kk .. + 7, then of + 8 .. + 15
+      asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+                   : "=r"(pa[kk][0]), "=r"(pa[kk][1]), "=r"(pa[kk][2]), "=r"(pa[kk][3])
+                   : "r"(smem_u32(&pr[ri + 8 * (mi & 1)][16 * kk + 8 * (mi >> 1)])));
     const uint32_t base = ring_u + (uint32_t)((j - tile0) % R::STAGES) * R::TILE;
 #pragma unroll
     for (int kk = 0; kk < 2; ++kk) {
@@ -234,16 +241,18 @@ latent_attention_mma_kernel(Params p) {
   asm volatile("cp.async.wait_group 0;" ::: "memory");
 #pragma unroll
   for (int rr = 0; rr < 2; ++rr) {
-    l[rr] += __shfl_xor_sync(0xffffffffu, l[rr], 1);
-    l[rr] += __shfl_xor_sync(0xffffffffu, l[rr], 2);
+#pragma unroll
+    for (int s = 16; s > 0; s >>= 1) l[rr] += __shfl_xor_sync(0xffffffffu, l[rr], s);
+    if (lane == 0) ml[warp + 8 * rr] = make_float2(m[rr], l[rr]);
   }
   __nv_bfloat16 *out = (__nv_bfloat16 *)p.out + ((size_t)r * p.heads + head0) * LD;
   if (p.splits == 1) {
+    __syncthreads();
 #pragma unroll
     for (int rr = 0; rr < 2; ++rr) {
       const int h = g + 8 * rr;
       if (h >= n_heads) continue;
-      const float f = (p.gate ? p.gate[(size_t)r * p.gate_ld + head0 + h] : 1.f) / l[rr];
+      const float f = (p.gate ? p.gate[(size_t)r * p.gate_ld + head0 + h] : 1.f) / ml[h].y;
 #pragma unroll
       for (int d = 0; d < NT; ++d)
         *reinterpret_cast<uint32_t *>(out + (size_t)h * LD + (chunk0 + d) * 8 + 2 * tq) = pack_bf16(o[d][2 * rr] * f, o[d][2 * rr + 1] * f);
@@ -260,7 +269,6 @@ latent_attention_mma_kernel(Params p) {
     float *po = os + (g + 8 * rr) * LD;
 #pragma unroll
     for (int d = 0; d < NT; ++d) *reinterpret_cast<float2 *>(po + (chunk0 + d) * 8 + 2 * tq) = make_float2(o[d][2 * rr], o[d][2 * rr + 1]);
-    if (warp == 0 && tq == 0) ml[g + 8 * rr] = make_float2(m[rr], l[rr]);
   }
   cluster_sync_all();
   if (threadIdx.x < 16) {
