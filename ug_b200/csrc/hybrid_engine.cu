@@ -296,9 +296,9 @@ int32_t run_layers(ugb_hybrid *m, Work &w, const int *tok, int t_block, int off,
         if ((rc = matmul(m, g))) return rc;
       }
       if (m->on(UGB_HYBRID_K_LATENT_ROWS)) {
-        const int threads = decode ? 512 : 256, per = (n_in / 4 + threads - 1) / threads;
+        const int threads = std::min(512, (n_in / 4 + 31) / 32 * 32), per = (n_in / 4 + threads - 1) / threads;
         auto *k = decode ? (per <= 1 ? latent_inputs_kernel<T, 1, 8> : per <= 2 ? latent_inputs_kernel<T, 2, 8> : latent_inputs_kernel<T, 16, 1>)
-                         : (per <= 2 ? latent_inputs_kernel<T, 2, 1> : per <= 4 ? latent_inputs_kernel<T, 4, 1> : latent_inputs_kernel<T, 16, 1>);
+                         : (per <= 1 ? latent_inputs_kernel<T, 1, 1> : per <= 2 ? latent_inputs_kernel<T, 2, 1> : per <= 4 ? latent_inputs_kernel<T, 4, 1> : latent_inputs_kernel<T, 16, 1>);
         e = ugb_launch(k, dim3(rows), dim3(threads), 0, st, pdl, w.pre, ti.splits, (size_t)rows * n_in,
                        L.q_gain, L.c_gain, (T *)w.cq, (T *)L.cache, w.gate, m->pos, off, t, m->t_max, L.ql, L.cl, L.gl,
                        1.0f / (float)L.d.q_rank, 1.0f / (float)L.d.kv_rank, m->cfg.eps, dev->status_dev);
@@ -590,7 +590,7 @@ int32_t ugb_hybrid_create(ugb_device *dev, const ugb_hybrid_config *cfg, const u
       L.expand = !m->f32 && dp && vp && d.scale > 0.f;
       L.dp = L.expand ? dp : (int)up8(d.dim);
       L.vp = L.expand ? vp : (int)up8(d.vdim);
-      CHECK(L.ql + L.cl + L.gl <= 16 * 4 * 256, UGB_ERR_UNSUPPORTED, "layer %d: latents of %d + %d values", i, d.q_rank, d.kv_rank);
+      CHECK(L.ql + L.cl + L.gl <= 16 * 4 * 512, UGB_ERR_UNSUPPORTED, "layer %d: latents of %d + %d values", i, d.q_rank, d.kv_rank);
       TRY(alloc_bytes(m, &L.w_in, (size_t)(L.ql + L.cl + L.gl) * wl * es, true));
       TRY(alloc_bytes(m, &L.w_uq, (size_t)d.heads * L.dp * L.ql * es, true));
       TRY(alloc_bytes(m, &L.w_uk, (size_t)d.heads * L.dp * L.cl * es, true));

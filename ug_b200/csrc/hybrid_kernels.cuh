@@ -44,8 +44,9 @@ template <bool EXACT> __device__ __forceinline__ float sigmoid_t(float x) {
 }
 __device__ __forceinline__ float sigmoid_f(float x) { return sigmoid_t<true>(x); }
 __device__ __forceinline__ float silu_f(float x) { return x / (1.0f + expf(-x)); }
-// candidate of the minimal gated recurrent unit: u + 1/2 for u >= 0, sigmoid(u) below
-template <bool EXACT> __device__ __forceinline__ float gru_candidate(float u) { return u >= 0.0f ? u + 0.5f : sigmoid_t<EXACT>(u); }
+// candidate of the minimal gated recurrent unit: u + 1/2 for u >= 0, sigmoid(u) below -- the larger of the two on either
+// side, since sigmoid has slope at most 1/4 and equals 1/2 at 0
+template <bool EXACT> __device__ __forceinline__ float gru_candidate(float u) { return fmaxf(u + 0.5f, sigmoid_t<EXACT>(u)); }
 
 __device__ __forceinline__ float block_sum_256(float v, float *sm) {   // sm: 8 floats; all 256 threads
 #pragma unroll
@@ -416,16 +417,16 @@ min_gru_step_kernel(const float *__restrict__ pre, int n_part, size_t part_strid
   Act<T>::st4(out + (size_t)r * ld + 4 * c, make_float4(S.x * silu_f(g.x), S.y * silu_f(g.y), S.z * silu_f(g.z), S.w * silu_f(g.w)));
 }
 
-// A block of t positions per sequence as a scan over time.  A lane is a channel; a warp takes SCAN_STEPS consecutive
+// A block of t positions per sequence as a scan over time.  A lane is a channel; a warp takes STEPS consecutive
 // positions, a CTA SCAN_WARPS warps' worth, a cluster of CTAs (grid.x) consecutive pieces of the sequence.  Each warp
 // composes its positions into one affine map S -> A S + B held in registers, the maps meet in shared memory (warps)
 // and distributed shared memory (CTAs), and every warp then replays its positions from its own incoming state.  The
-// cluster walks the sequence in rounds of SCAN_BLOCK * gridDim.x positions; all CTAs run every round.
+// cluster walks the sequence in rounds of BLOCK * gridDim.x positions; all CTAs run every round.
 // bf16 pre-activations: a lane takes two adjacent channels, so a warp reads 128 bytes of a row either way.
-constexpr int SCAN_WARPS = 16;
+constexpr int SCAN_WARPS = 8;
 template <typename TI> struct Scan {
   static constexpr int V = sizeof(TI) == 2 ? 2 : 1;        // channels per lane
-  static constexpr int STEPS = 4;                          // positions per warp and round
+  static constexpr int STEPS = 8;                          // positions per warp and round
   static constexpr int BLOCK = SCAN_WARPS * STEPS, COLUMNS = 32 * V;
 };
 
@@ -481,9 +482,10 @@ min_gru_scan_kernel(const TI *__restrict__ pre, const float *__restrict__ bz, co
   for (int t0 = 0; t0 < t; t0 += BLOCK * n_cta, ++round) {
     const int i0 = t0 + rank * BLOCK + warp * STEPS;
     const bool whole = i0 + STEPS <= t;
-    float a[STEPS][V], bb[STEPS][V], sg[STEPS][V];
+    float a[STEPS][V], bb[STEPS][V];
+    uint32_t g[STEPS];
 #pragma unroll
-    for (int s = 0; s < STEPS; ++s) { scan_widen<V>(nz[s], a[s]); scan_widen<V>(nu[s], bb[s]); scan_widen<V>(ng[s], sg[s]); }
+    for (int s = 0; s < STEPS; ++s) { scan_widen<V>(nz[s], a[s]); scan_widen<V>(nu[s], bb[s]); g[s] = ng[s]; }
     fetch(i0 + BLOCK * n_cta);
     float A[V], B[V];
 #pragma unroll
@@ -492,10 +494,9 @@ min_gru_scan_kernel(const TI *__restrict__ pre, const float *__restrict__ bz, co
 #pragma unroll
       for (int s = 0; s < STEPS; ++s) {
         const float z = sigmoid_t<EXACT>(a[s][e] + zb[e]);
-        const bool live = whole || i0 + s < t;             // positions behind the block leave the state alone
-        a[s][e] = live ? 1.0f - z : 1.0f;
-        bb[s][e] = live ? z * gru_candidate<EXACT>(bb[s][e] + ub[e]) : 0.0f;
-        sg[s][e] = sg[s][e] * sigmoid_t<EXACT>(sg[s][e]);
+        a[s][e] = 1.0f - z;
+        bb[s][e] = z * gru_candidate<EXACT>(bb[s][e] + ub[e]);
+        if (!whole && i0 + s >= t) { a[s][e] = 1.0f; bb[s][e] = 0.0f; }   // behind the block: leaves the state alone
         A[e] *= a[s][e];
         B[e] = fmaf(a[s][e], B[e], bb[s][e]);
       }
@@ -544,15 +545,19 @@ min_gru_scan_kernel(const TI *__restrict__ pre, const float *__restrict__ bz, co
     for (int s = 0; s < STEPS; ++s) {
 #pragma unroll
       for (int e = 0; e < V; ++e) S[e] = fmaf(a[s][e], S[e], bb[s][e]);
+      float sg[V];
+      scan_widen<V>(g[s], sg);
+#pragma unroll
+      for (int e = 0; e < V; ++e) sg[e] *= sigmoid_t<EXACT>(sg[e]);
       if (on && (whole || i0 + s < t)) {
         T *o = out + (base + i0 + s) * (size_t)ld + c;
         if constexpr (sizeof(T) == 4) {
 #pragma unroll
-          for (int e = 0; e < V; ++e) o[e] = S[e] * sg[s][e];
+          for (int e = 0; e < V; ++e) o[e] = S[e] * sg[e];
         } else if constexpr (V == 2) {
-          *reinterpret_cast<__nv_bfloat162 *>(o) = __floats2bfloat162_rn(S[0] * sg[s][0], S[1] * sg[s][1]);
+          *reinterpret_cast<__nv_bfloat162 *>(o) = __floats2bfloat162_rn(S[0] * sg[0], S[1] * sg[1]);
         } else {
-          *o = __float2bfloat16_rn(S[0] * sg[s][0]);
+          *o = __float2bfloat16_rn(S[0] * sg[0]);
         }
       }
     }
@@ -567,7 +572,7 @@ min_gru_scan_kernel(const TI *__restrict__ pre, const float *__restrict__ bz, co
 // ------------------------------------------------- latent attention inputs ---
 // pre [n_part][rows][q_ld + c_ld + g_ld]: query latent, key/value latent and head gates of one projection.
 //   cq[r] = norm(query latent) * q_gain   cache[b][pos] = norm(kv latent) * c_gain   gate[r] = sigmoid(head gate)
-// row r = (b, i) = (r / t, r % t), pos = *pos_p + pos_off + i.  One CTA of 256 or 512 threads per row, PER groups of 4
+// row r = (b, i) = (r / t, r % t), pos = *pos_p + pos_off + i.  One CTA of up to 512 threads per row, PER groups of 4
 // columns per thread (the segments are multiples of 8 wide), U split-K partials in flight.
 template <typename T, int PER, int U>
 __global__ void __launch_bounds__(512)
