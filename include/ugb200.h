@@ -532,22 +532,39 @@ UGB_API int32_t ugb_llama_time_kernel(ugb_llama *m, int32_t which, int32_t iters
 
 /* --------------------------------------- decoders described by a list of layers */
 /* No counterpart in the reference, which has one fixed layer.  A decoder whose
- * layers are listed one by one: each has a token mixer (a recurrence or latent
+ * layers are listed one by one, in one of two forms.
+ *
+ * UGB_FORM_SANDWICH: each layer has a token mixer (a recurrence or latent
  * attention) and optionally a feed-forward, both between two RMS norms
  * (x += norm_b(f(conv(norm_a(x))))), the sublayer input optionally passed
  * through a causal depthwise convolution, and the stream between layers
  * optionally a learned average of all layer results so far.  With X_0 the
  * normalised embedding and X_{i+1} the result of layer i, what layer i + 1
- * reads is sum_{j <= i+1} dwa_i[j] X_j.  The step functions are those of
+ * reads is sum_{j <= i+1} dwa_i[j] X_j.
+ *
+ * UGB_FORM_PARALLEL: mixer and feed-forward read the same norm,
+ * x += mixer(h) + ff(h) with h = norm1(x), and optionally a per-layer input of
+ * the token follows: x += norm(proj(gelu_tanh(gate x) * table[token, layer])).
+ * The mixer is grouped-query attention with rotary positions and a selective
+ * scan side by side, each with its factor; the feed-forward is gated (silu) or a
+ * mixture of such experts (sigmoid scores, the best `top` of them, the score
+ * multiplies the expert's input) beside an optional shared one.  Layers
+ * loop_start .. loop_stop - 1 may run several times with the same weights and
+ * each time their own state; ahead of pass t, x <- W_in [x; x_0] + step[t] with
+ * x_0 the embedding output.
+ *
+ * The step functions are those of
  * ugb_llama: batch rows are independent sequences that share one position; a
  * decode step is one captured CUDA graph; a prompt runs in chunks of positions
  * and may be continued by further prompts or steps at any position.  Per
- * sequence the engine keeps, by layer: the last taps - 1 convolution inputs of
- * both sublayers, a f32 recurrent state, or one latent row per position. */
+ * sequence the engine keeps, by layer run: the last taps - 1 convolution inputs,
+ * a f32 recurrent state, one latent row per position, or keys and values. */
 typedef struct ugb_hybrid ugb_hybrid;
 
-enum { UGB_MIXER_MINGRU = 0, UGB_MIXER_LATENT_ATTENTION = 1 };
-enum { UGB_FF_NONE = 0, UGB_FF_RELU2 = 1 /* down(max(up h, 0)^2) */ };
+enum { UGB_FORM_SANDWICH = 0, UGB_FORM_PARALLEL = 1 };
+enum { UGB_MIXER_MINGRU = 0, UGB_MIXER_LATENT_ATTENTION = 1, UGB_MIXER_ATTENTION_SCAN = 2 /* parallel form */ };
+enum { UGB_FF_NONE = 0, UGB_FF_RELU2 = 1 /* down(max(up h, 0)^2), sandwich form */,
+       UGB_FF_GATED = 2 /* down(silu(gate h) * up h), parallel form */, UGB_FF_EXPERTS = 3 /* parallel form */ };
 
 typedef struct {
   int32_t width;           /* of the residual stream                                     */
@@ -560,6 +577,10 @@ typedef struct {
                               FP32 pipe                                                   */
   float eps;               /* of every norm, inside the root                              */
   float gain_offset;       /* gain of a stream norm = gain_offset + stored weight         */
+  int32_t form;            /* UGB_FORM_*                                                  */
+  int32_t loop_start, loop_stop, loop_times;   /* parallel form; loop_times 0 = no loop   */
+  int32_t side_dim;        /* parallel form: columns of a layer's token input, 0 = none   */
+  float logit_softcap;     /* logits <- cap tanh(logits / cap); 0 = none                  */
 } ugb_hybrid_config;
 
 typedef struct {
@@ -568,7 +589,14 @@ typedef struct {
   int32_t heads, dim, vdim, q_rank, kv_rank;   /* latent attention                        */
   float scale;             /* latent attention: factor of the scores                      */
   int32_t feed_forward;    /* UGB_FF_*                                                    */
-  int32_t ff;              /* feed-forward columns                                        */
+  int32_t ff;              /* feed-forward columns; experts: of the shared one, 0 = none  */
+  /* attention beside a scan: heads, dim, vdim and scale above, and */
+  int32_t kv_heads, rot_dims, rot_interleaved;   /* rotated dimensions of a head; pairs (2i, 2i + 1) or (i, i + rot_dims / 2) */
+  int32_t qk_norm;         /* 1: rotated queries and keys are divided by their root mean square */
+  float rot_base, attention_scale;               /* factor of the attention's output       */
+  int32_t inner, state, conv, dt_rank;           /* scan: channels, states, taps, rank of the step size */
+  float scan_scale;        /* factor of the scan's output                                 */
+  int32_t experts, top, expert_ff;
 } ugb_hybrid_layer;
 
 enum { UGB_HYBRID_LOGITS = 0, UGB_HYBRID_NEXT_TOKENS = 1, UGB_HYBRID_HIDDEN = 2, UGB_HYBRID_PREFILL_LOGITS = 3,
@@ -585,12 +613,25 @@ UGB_API int32_t ugb_hybrid_destroy(ugb_hybrid *m);
  * [width, channels]; latent attention: "mix.dq" [q_rank, width], "mix.dq.norm",
  * "mix.uq" [heads * dim, q_rank], "mix.dkv" [kv_rank, width], "mix.dkv.norm",
  * "mix.uk" [heads * dim, kv_rank], "mix.uv" [heads * vdim, kv_rank], "mix.g"
- * [heads, width], "mix.o" [width, heads * vdim].  BF16 or F32; f32 matrices are
- * rounded to nearest even when the model is bf16. */
+ * [heads, width], "mix.o" [width, heads * vdim].
+ * Parallel form: "embed", "final.norm", "head"; "loop.in" [width, 2 width] (x
+ * first), "loop.step" [times, width], "side.embed" [vocab, layers * side_dim]; of
+ * layer i "norm1" [width], "mix.left.q" [heads * dim, width], "mix.left.k",
+ * "mix.left.v" [kv_heads * dim / vdim, width], "mix.left.o" [width, heads * vdim],
+ * "mix.right.in" [2 inner, width] (x, then z), "mix.right.conv" [inner, taps],
+ * "mix.right.conv.b" [inner], "mix.right.x" [dt_rank + 2 state, inner],
+ * "mix.right.dt" [inner, dt_rank], "mix.right.dt.b" [inner], "mix.right.A_log"
+ * [inner, state], "mix.right.D" [inner], "mix.right.o" [width, inner];
+ * "mlp.gate", "mlp.up" [ff, width], "mlp.down" [width, ff], or "mlp.router"
+ * [experts, width], "mlp.e<j>.gate" / ".up" / ".down" and "mlp.shared.gate" /
+ * ".up" / ".down"; "side.gate" [side_dim, width], "side.proj" [width, side_dim],
+ * "side.norm" [width].
+ * BF16 or F32; f32 matrices are rounded to nearest even when the model is bf16. */
 UGB_API int32_t ugb_hybrid_load_weight(ugb_hybrid *m, const char *name, const ugb_slice *w);
 /* "pdl" (0 / 1), "prefill_rows" (16..65536, before the first prompt),
- * "absorb_max" (blocks of at most this many positions run attention in the
- * latent space instead of expanding keys and values, default 16), "att_splits"
+ * "absorb_max" (blocks of at most this many positions run attention position by
+ * position -- latent attention in the latent space -- instead of on the tcgen05
+ * kernel, default 16), "att_splits"
  * (slices of the cache per row in a decode step, 0 = chosen from the batch),
  * "keep_layers" (0 / 1: keep the stream after every layer of a prompt). */
 UGB_API int32_t ugb_hybrid_set_option(ugb_hybrid *m, const char *key, int32_t value);
@@ -611,7 +652,12 @@ enum { UGB_HYBRID_K_ROWS = 0 /* residual, norms, average, fused convolution */, 
        UGB_HYBRID_K_GRU_IN = 2, UGB_HYBRID_K_GRU = 3, UGB_HYBRID_K_LATENT_IN = 4, UGB_HYBRID_K_LATENT_ROWS = 5,
        UGB_HYBRID_K_UQ = 6, UGB_HYBRID_K_ABSORB = 7 /* q W_uk, W_uv o, or the expansion of keys and values */,
        UGB_HYBRID_K_ATTENTION = 8, UGB_HYBRID_K_OUT = 9, UGB_HYBRID_K_UP = 10, UGB_HYBRID_K_DOWN = 11,
-       UGB_HYBRID_K_HEAD = 12, UGB_HYBRID_K_ALL = 13 };
+       UGB_HYBRID_K_HEAD = 12,
+       /* parallel form, beside ROWS, CONV, ATTENTION, OUT, UP (gated, shared) and HEAD */
+       UGB_HYBRID_K_MIX_IN = 13 /* q | k | v | x | z | router */, UGB_HYBRID_K_MIX_ROWS = 14 /* rotation, cache, a step's convolution and choice */,
+       UGB_HYBRID_K_SCAN_IN = 15 /* step size, B, C */, UGB_HYBRID_K_SCAN = 16, UGB_HYBRID_K_ROUTE = 17 /* choice, rows by expert */,
+       UGB_HYBRID_K_EXPERT_UP = 18, UGB_HYBRID_K_EXPERT_DOWN = 19, UGB_HYBRID_K_SIDE = 20 /* products of the token input */,
+       UGB_HYBRID_K_SIDE_GATE = 21, UGB_HYBRID_K_LOOP = 22, UGB_HYBRID_K_ALL = 23 };
 UGB_API int32_t ugb_hybrid_time_kernel(ugb_hybrid *m, int32_t which, int32_t t, int32_t iters, float *ms_per_pass);
 
 /* The engine's mechanisms as operators on plain buffers (all F32 or, where
@@ -643,6 +689,38 @@ UGB_API int32_t ugb_causal_attention_wide(ugb_device *dev, const ugb_slice *q, c
 UGB_API int32_t ugb_residual_update(ugb_device *dev, ugb_slice *x, const ugb_slice *y, const ugb_slice *post_gain,
                                     ugb_slice *bank, const ugb_slice *dwa, size_t n, const ugb_slice *gain, ugb_slice *h,
                                     size_t rows, size_t width, float eps);
+/* out = silu(bias + the causal convolution of ugb_causal_conv without h itself); bias F32 [width], the rest as there. */
+UGB_API int32_t ugb_gated_conv(ugb_device *dev, const ugb_slice *h, const ugb_slice *w, const ugb_slice *bias, ugb_slice *tail,
+                               ugb_slice *out, size_t b, size_t t, size_t width, size_t taps);
+/* Queries, keys and values of a block: pre T [b, t, (heads + kv_heads) * dim + kv_heads * vdim] (q | k | v heads), cos / sin
+ * F32 [t_max, rot_dims / 2], positions pos[0] + i.  q T [b, t, heads, dim] and the key cache T [b, kv_heads, t_max, dim] get
+ * the rotated heads, with qk_norm divided by their root mean square over dim; values go to vcache T [b, kv_heads, t_max, vdim]. */
+UGB_API int32_t ugb_head_inputs(ugb_device *dev, const ugb_slice *pre, const ugb_slice *cos_, const ugb_slice *sin_,
+                                const ugb_slice *pos, ugb_slice *q, ugb_slice *kcache, ugb_slice *vcache, size_t b, size_t t,
+                                size_t heads, size_t kv_heads, size_t dim, size_t vdim, size_t rot_dims, int32_t interleaved,
+                                int32_t qk_norm, float eps, size_t t_max);
+/* Attention of single positions over caches of keys and values: q T [b, t, heads, dq], k / v T [b, kv_heads, t_max, dq / dv],
+ * out T [b, t, heads, dv] times out_scale; query i attends positions 0 .. pos[0] + i, query head h reads head
+ * h / (heads / kv_heads).  n_slices: as in ugb_latent_attend, where the bf16 kernel takes the heads (64 or 128 wide). */
+UGB_API int32_t ugb_grouped_attend(ugb_device *dev, const ugb_slice *q, const ugb_slice *k, const ugb_slice *v, const ugb_slice *pos,
+                                   ugb_slice *out, size_t b, size_t t, size_t heads, size_t kv_heads, size_t dq, size_t dv,
+                                   size_t t_max, float scale, float out_scale, int32_t n_slices);
+/* The same for a block at positions pos0 .. pos0 + t - 1 on the tcgen05 kernel: BF16, dq and dv 64 or 128. */
+UGB_API int32_t ugb_grouped_attend_block(ugb_device *dev, const ugb_slice *q, const ugb_slice *k, const ugb_slice *v, ugb_slice *out,
+                                         size_t b, size_t t, size_t pos0, size_t heads, size_t kv_heads, size_t dq, size_t dv,
+                                         size_t t_max, float scale, float out_scale);
+/* Selective scan of a block: x, dt, z, out T [b, t, channels] (dt before bias and softplus), bc T [b, t, 2 states] (B | C), a_log
+ * F32 [channels, states], skip, dt_bias F32 [channels], state F32 [b, channels, states] in and out; out = (C S + skip x) silu(z)
+ * times scale.  states: 8, 16, 24, 32, 48, 64, 128 or 256. */
+UGB_API int32_t ugb_selective_scan(ugb_device *dev, const ugb_slice *x, const ugb_slice *dt, const ugb_slice *bc, const ugb_slice *z,
+                                   const ugb_slice *a_log, const ugb_slice *skip, const ugb_slice *dt_bias, ugb_slice *state,
+                                   ugb_slice *out, size_t b, size_t t, size_t channels, size_t states, float scale);
+/* One position of every sequence: low_bc F32 [rows, rank + 2 states], w_dt T [rank, channels], z F32 [rows, channels]; dt =
+ * softplus(w_dt^T low + dt_bias); the rest as above with t = 1. */
+UGB_API int32_t ugb_selective_step(ugb_device *dev, const ugb_slice *x, const ugb_slice *low_bc, const ugb_slice *w_dt,
+                                   const ugb_slice *z, const ugb_slice *a_log, const ugb_slice *skip, const ugb_slice *dt_bias,
+                                   ugb_slice *state, ugb_slice *out, size_t rows, size_t channels, size_t rank, size_t states,
+                                   float scale);
 
 #ifdef __cplusplus
 }

@@ -49,6 +49,8 @@ struct Params {
   float scale;
   const float *gate;   // f32 [batch * t][gate_ld]: factor per query row and head, or null
   int gate_ld;
+  long long out_ld;    // output elements between positions
+  float out_scale;
   __nv_bfloat16 *out;
   ugb_status_word *status;
   int *sched;   // {next item, CTAs done}: both zero between launches; null = items dealt round-robin
@@ -330,9 +332,9 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __gri
       }
       if (alive && it.n_tiles > 0) fold(g0 + it.n_tiles - 1, alpha_prev);
       if (alive && qi < p.t) {
-        float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+        float inv = l_run > 0.f ? p.out_scale / l_run : 0.f;
         if (p.gate) inv *= p.gate[((size_t)it.b * p.t + qi) * p.gate_ld + it.head];
-        __nv_bfloat16 *dst = p.out + ((size_t)it.b * p.t + qi) * ((size_t)p.n_heads * DV) + (size_t)it.head * DV;
+        __nv_bfloat16 *dst = p.out + ((size_t)it.b * p.t + qi) * (size_t)p.out_ld + (size_t)it.head * DV;
 #pragma unroll
         for (int c = 0; c < DV / 8; ++c) {
           uint4 v;
@@ -383,6 +385,7 @@ int32_t launch(ugb_device *dev, const ugb_prefill_attention_args &a) {
   Params p;
   p.t = a.t; p.pos0 = a.pos0; p.n_heads = a.n_heads; p.n_kv = a.n_kv; p.batch = a.batch; p.scale = a.scale; p.out = a.out;
   p.gate = a.gate; p.gate_ld = a.gate_ld;
+  p.out_ld = a.out_ld ? a.out_ld : (long long)a.n_heads * DV; p.out_scale = a.out_scale;
   p.status = dev->status_dev;
   p.sched = a.dynamic ? dev->sched_dev : nullptr;
   const long long n_items = (long long)((a.t + BQ - 1) / BQ) * a.n_heads * a.batch;

@@ -4,7 +4,7 @@
 
 #include "ugb_internal.h"
 
-// out[b, i, head, :] = gate softmax_j(scale * q[b, i, head, :] . k[b, kvh, j, :]) v[b, kvh, j, :] over the cached
+// out[b, i, head, :] = out_scale gate softmax_j(scale * q[b, i, head, :] . k[b, kvh, j, :]) v[b, kvh, j, :] over the cached
 // positions j <= pos0 + i, for i in [0, t).  All base pointers 16-byte aligned.
 struct ugb_prefill_attention_args {
   const __nv_bfloat16 *q;          // [batch, t, n_heads, dq]
@@ -17,6 +17,8 @@ struct ugb_prefill_attention_args {
   float scale;
   const float *gate = nullptr;     // f32 [batch * t][gate_ld]: factor per query and head
   int gate_ld = 0;
+  long long out_ld = 0;            // output elements between positions (a multiple of 8), 0 = n_heads * dv
+  float out_scale = 1.0f;          // factor of every output
   int dynamic = 1;                 // the persistent CTAs draw their work items from the device's counter (longest
                                    // first); 0: the items are dealt round-robin
 };

@@ -83,6 +83,7 @@ struct Params {
   unsigned long long *prof;   // measurement aid (or null): %globaltimer stamps of CTA 0, see UGB_TC_PROF_* in the header
   int pair_k;             // 1: CTAs 2c and 2c + 1 are a cluster and take the two k halves of tile c (BM = 64,
                           // UGB_EPI_SILU_MUL_BF16): rank 1 hands its sums to rank 0 through shared memory
+  const int *groups;      // grouped rows: m tile i multiplies the N rows of B from groups[i] * N on (< 0: no tile); or null
   long long c_batch;      // output elements between batch steps
   long long c_ld;         // output elements between rows
   long long c_split;      // output elements between split-K partials
@@ -132,7 +133,14 @@ tc_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
   if (threadIdx.x == 0) UGB_TC_STAMP(UGB_TC_PROF_START);
   bool pair_ready = false;           // pair_k: this epilogue thread saw its accumulator complete
   int pair_m0 = 0, pair_n0 = 0;
+  if (p.groups) ugb_pdl_wait();      // the map of tiles is written by a preceding kernel
   const int tiles_per_batch = p.tiles_m * p.tiles_n;
+  // m tile of tile r of a batch step, and the first row of B its group has (-1: nothing to compute)
+  auto group_row = [&](int r) {
+    if (!p.groups) return 0;
+    const int g = __ldcg(p.groups + (p.n_fast ? r / p.tiles_n : r % p.tiles_m));
+    return g < 0 ? -1 : g * p.N;
+  };
   const int tiles_per_split = tiles_per_batch * p.batch;
   const int n_tiles = tiles_per_split * p.splits;
   // tile number -> (k split, tile inside the split); with pair_k the two k halves of a tile are neighbours
@@ -250,7 +258,9 @@ tc_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
         const int bi = ts / tiles_per_batch;
         const int r = ts - bi * tiles_per_batch;
         const int m0 = (p.n_fast ? r / p.tiles_n : r % p.tiles_m) * TILE_M + (int)rank * BM;
-        const int n0 = (p.n_fast ? r % p.tiles_n : r / p.tiles_m) * BN;
+        const int b_row = group_row(r);
+        if (b_row < 0) continue;
+        const int n0 = b_row + (p.n_fast ? r % p.tiles_n : r / p.tiles_m) * BN;
         const int bz = p.b_batched ? bi : 0;
         const int kb0 = sp * p.kb_per_split;
         const int kb1 = min(p.k_blocks, kb0 + p.kb_per_split);
@@ -283,8 +293,9 @@ tc_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
       uint32_t phase = 0, acc_phase = 0;
       bool alive = true;
       for (int tile = cta0; tile < n_tiles && alive; tile += n_ctas) {
-        int sp, ts_unused;
-        split_of(tile, sp, ts_unused);
+        int sp, ts;
+        split_of(tile, sp, ts);
+        if (group_row(ts % tiles_per_batch) < 0) continue;
         const int kb0 = sp * p.kb_per_split;
         const int kb1 = min(p.k_blocks, kb0 + p.kb_per_split);
         if (!mbar_wait(smem_u32(&acc_empty[acc]), acc_phase ^ 1u, abort_flag, p.status, 2)) break;
@@ -330,6 +341,7 @@ tc_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
       split_of(tile, sp, ts);
       const int bi = ts / tiles_per_batch;
       const int r = ts - bi * tiles_per_batch;
+      if (group_row(r) < 0) continue;
       const int m0 = (p.n_fast ? r / p.tiles_n : r % p.tiles_m) * TILE_M + (int)rank * BM;
       const int n0 = (p.n_fast ? r % p.tiles_n : r / p.tiles_m) * BN;
       if (!mbar_wait(smem_u32(&acc_full[acc]), acc_phase, abort_flag, p.status, 4)) break;
@@ -690,6 +702,7 @@ int32_t launch_tc(ugb_device *dev, TcState *st, const ugb_tc_gemm_args &g, size_
   p.f16 = g.f16 ? 1 : 0;
   p.late_trigger = g.late_trigger ? 1 : 0;
   p.prof = g.prof;
+  p.groups = g.groups;
   p.pair_k = 0;
   if (g.pair_k) {
     // two CTAs (a cluster) per tile, each over half of k
@@ -718,7 +731,7 @@ int32_t launch_tc(ugb_device *dev, TcState *st, const ugb_tc_gemm_args &g, size_
   if (rc) return rc;
   const uint64_t nb = p.b_batched ? batch : 1;
   const uint64_t bs = p.b_batched ? (uint64_t)g.b_batch : n * k;
-  if (g.b_is_nk) rc = encode_map(dev, st, &tmB, g.b, k, n, nb, k, bs, BK, C_::BN_CTA, g.f16);
+  if (g.b_is_nk) rc = encode_map(dev, st, &tmB, g.b, k, g.groups ? n * (uint64_t)g.n_groups : n, nb, k, bs, BK, C_::BN_CTA, g.f16);
   else rc = encode_map(dev, st, &tmB, g.b, n, k, nb, n, bs, 64, BK, g.f16);
   if (rc) return rc;
 
@@ -790,6 +803,9 @@ int32_t ugb_tc_gemm(ugb_device *dev, const ugb_tc_gemm_args &g) {
   if (g.f16 && g.epi != UGB_EPI_BF16 && g.epi != UGB_EPI_F32) return UGB_ERR_UNSUPPORTED;   // the fused epilogues write bf16
   if (g.epi == UGB_EPI_ROPE_QKV && (m <= 64 || batch != 1 || !g.b_is_nk || n % 64 != 0 || g.rope.t < 1)) return UGB_ERR_UNSUPPORTED;
   if (m == 0 || n == 0) return UGB_ERR_UNSUPPORTED;
+  if (g.groups && (batch != 1 || !g.b_is_nk || g.splits > 1 || g.pair_k || g.b_static || g.n_groups < 1 || (g.tile_m != 64 && g.tile_m != 128) ||
+                   m % g.tile_m != 0))
+    return UGB_ERR_UNSUPPORTED;
 
   TcState *st = state_of(dev);
   if (int32_t rc = ensure_encode(dev, st)) return rc;
@@ -802,7 +818,7 @@ int32_t ugb_tc_gemm(ugb_device *dev, const ugb_tc_gemm_args &g) {
   int bn = g.bn;
   if (bn == 0) bn = (m <= 128) ? 64 : 256;
   if (!g.b_is_nk && (bn == 80 || bn == 96)) bn = 128;                  // n-major B is boxed in 64-column pieces
-  if (m <= 64) {
+  if (g.groups ? g.tile_m == 64 : m <= 64) {
     if (bn == 64) return launch_tc<64, 64>(dev, st, g, batch, m);
     if (bn == 80) return launch_tc<64, 80>(dev, st, g, batch, m);      // widths that split n into close to one
     if (bn == 96) return launch_tc<64, 96>(dev, st, g, batch, m);      // tile per SM where 64 / 128 do not
@@ -812,7 +828,7 @@ int32_t ugb_tc_gemm(ugb_device *dev, const ugb_tc_gemm_args &g) {
   }
   if (bn == 80 || bn == 96) bn = 128;                                  // BM = 128 needs n % 16 == 0 tiles: keep the three sizes
   // CTA pairs: 256 x 256 tiles over two SMs; every SM fetches half as much of B per flop
-  const bool pair = g.pair < 0 ? dev->gemm_pair != 0 : g.pair != 0;
+  const bool pair = g.groups ? false : g.pair < 0 ? dev->gemm_pair != 0 : g.pair != 0;
   if (pair && bn == 256 && m > 128 && g.splits <= 1 && dev->sm_count >= 2) return launch_tc<128, 256, true>(dev, st, g, batch, m);
   if (bn == 64) return launch_tc<128, 64>(dev, st, g, batch, m);
   if (bn == 128) return launch_tc<128, 128>(dev, st, g, batch, m);

@@ -54,6 +54,11 @@ struct ugb_tc_gemm_args {
   bool pair_k = false;  // m <= 64, an epilogue that writes bf16 columns: two CTAs (a thread-block cluster) per tile, each over half of k; the
                         // second hands its sums to the first through distributed shared memory.  UGB_ERR_UNSUPPORTED when
                         // twice the tiles exceed the SMs
+  // Rows grouped by the weights they multiply: rows [i tile_m, (i + 1) tile_m) of A and of the output belong to group
+  // groups[i] (device memory, written by a preceding kernel; < 0: rows without work), whose weights are rows
+  // [groups[i] n, (groups[i] + 1) n) of b [n_groups * n, k].  tile_m 64 or 128, m a multiple of it, b_is_nk, batch 1, no splits.
+  const int *groups = nullptr;
+  int n_groups = 0, tile_m = 0;
   unsigned long long *prof = nullptr;   // measurement aid, see UGB_TC_PROF_*
   int pair = -1;        // 256 x 256 tiles on pairs of CTAs (cta_group::2) where the shape allows: 1 / 0, -1 = the device's setting
   ugb_tc_rope_epilogue rope = {};   // UGB_EPI_ROPE_QKV only

@@ -1,8 +1,9 @@
-// Decoders described by a list of layers (ugb_hybrid_*): token mixers of several kinds behind one chain of sandwich
-// norms, input convolutions and a depth average.  The step loop, its CUDA graph, the prompt loop and weight upload are
-// those of engine_core.cuh; the products run on the tcgen05 GEMM (bf16) or the FP32-pipe kernels (f32).
+// Decoders described by a list of layers (ugb_hybrid_*).  The step loop, its CUDA graph, the prompt loop and weight upload
+// are those of engine_core.cuh; the products run on the tcgen05 GEMM (bf16) or the FP32-pipe kernels (f32).  This file holds
+// the model's life cycle and the sandwich form of a layer -- token mixers of several kinds behind one chain of sandwich
+// norms, input convolutions and a depth average; the parallel form is in hybrid_parallel.cu.
 //
-// Launches of a layer (T = activation type):
+// Launches of a sandwich layer (T = activation type):
 //   row_update     stream += norm(previous product); layer bank, depth average; norm -> T   [decode: + convolution]
 //   causal_conv    prompts only: the input convolution over the block
 //   mingru:        GEMM z|u|g -> f32;  min_gru_step (decode) / min_gru_scan (prompt) -> T;  GEMM out -> f32
@@ -25,105 +26,43 @@
 
 #include "attention_tc.cuh"
 #include "decode_kernels.cuh"
-#include "engine_core.cuh"
 #include "gemm_tcgen05.cuh"
-#include "hybrid_kernels.cuh"
+#include "grouped_attention.cuh"
+#include "hybrid_engine.cuh"
 #include "latent_attention.cuh"
 
 using namespace ugb_hybrid_k;
 
-namespace {
-
-size_t up8(size_t n) { return (n + 7) / 8 * 8; }
-
-struct Layer {
-  ugb_hybrid_layer d{};
-  int ul = 0, fl = 0;                         // padded recurrent channels, feed-forward columns
-  int ql = 0, cl = 0, gl = 0, dp = 0, vp = 0; // latent attention: query latent, cache row, gates, head widths
-  bool expand = false;                        // long blocks may run on expanded keys and values
-  float *norm1 = nullptr, *norm1b = nullptr, *norm2 = nullptr, *norm2b = nullptr, *conv1 = nullptr, *conv2 = nullptr, *dwa = nullptr;
-  void *w_in = nullptr, *w_out = nullptr;     // mixer input projections side by side, output projection
-  float *bz = nullptr, *bu = nullptr;
-  float *q_gain = nullptr, *c_gain = nullptr;
-  void *w_uq = nullptr, *w_uk = nullptr, *w_uv = nullptr;
-  void *w_up = nullptr, *w_down = nullptr;
-  // state of the sequences
-  void *tail1 = nullptr, *tail2 = nullptr;    // inside ugb_hybrid::tails
-  float *state = nullptr;                     // mingru: [batch][ul]
-  void *cache = nullptr;                      // latent attention: [batch][t_max][cl]
-};
-
-// Activations of up to `rows` rows.
-struct Work {
-  int rows = 0;
-  float *x = nullptr, *bank = nullptr, *pre = nullptr, *gate = nullptr;
-  void *h = nullptr, *hc = nullptr, *mid = nullptr;       // norm output, convolved, mixer / feed-forward inner
-  void *cq = nullptr, *q = nullptr, *ql = nullptr, *ol = nullptr, *o = nullptr;
-};
-
-struct Mat {                       // out[b, m, n] = a . w
-  void *out; const void *a, *w;
-  size_t m, n, k, batch = 1, a_ld = 0, a_batch = 0, w_batch = 0, c_ld = 0, c_batch = 0;
-  bool nk = true;
-  bool f32_out = true;             // f32 result (split over k when splits > 1), else T
-  bool relu2 = false;
-  int splits = 1, bn = 0;
-};
-
-}  // namespace
-
-struct ugb_hybrid : ugb_engine {
-  ugb_hybrid_config cfg{};
-  std::vector<Layer> layers;
-  bool f32 = false;
-  int wl = 0;                      // padded width
-  void *embed = nullptr, *head = nullptr;
-  float *embed_gain = nullptr, *final_gain = nullptr;
-  unsigned char *tails = nullptr, *tails_next = nullptr;   // [layer][2][batch][taps - 1][wl], a block writes the second
-  size_t tail_bytes = 0;
-  Work dec, pf;
-  void *kx = nullptr, *vx = nullptr;                       // expanded keys / values of one layer
-  int att_splits_opt = 0, absorb_max = 16, keep_layers = 0;
-  float *layer_out = nullptr;
-  size_t layer_cap = 0;
-  int layer_rows = 0;
-  int only = UGB_HYBRID_K_ALL;     // measurement aid: the kernel kind that is launched
-
-  size_t es() const { return f32 ? 4 : 2; }
-  bool on(int kind) const { return only == UGB_HYBRID_K_ALL || only == kind; }
-  int att_splits() const;
-  int32_t enqueue_step(const int *tok) override;
-  int32_t ensure_prefill_workspace() override;
-  int32_t enqueue_prefill_chunk(const int *tok, int t, int c0, int tc, bool all_logits) override;
-  int32_t enqueue_prefill_tail(int tc) override;
-  int32_t enqueue_head(bool after_step) override;
-};
+using Mat = ugb_hybrid_mat;
+using Tiling = ugb_hybrid_tiling;
+static size_t up8(size_t n) { return ugb_up8(n); }
 
 int ugb_hybrid::att_splits() const {
   if (att_splits_opt > 0) return std::min(att_splits_opt, (int)UGB_LATENT_MAX_SPLITS);
   // two CTAs per SM over the (row, group of 16 heads) pairs
   int heads = 1;
-  for (const Layer &L : layers) heads = std::max(heads, L.d.heads);
+  for (const ugb_hybrid_weights &L : layers) heads = std::max(heads, L.d.heads);
   const int pairs = batch * ((heads + 15) / 16);
   return std::max(1, std::min((int)UGB_LATENT_MAX_SPLITS, 2 * dev->sm_count / pairs));
 }
 
-namespace {
-
-int32_t alloc_bytes(ugb_hybrid *m, void **p, size_t bytes, bool zero) {
+int32_t ugb_hybrid_alloc(ugb_hybrid *m, void **p, size_t bytes, bool zero) {
   unsigned char *b = nullptr;
   if (int32_t rc = dmalloc(m, &b, bytes, zero)) return rc;
   *p = b;
   return UGB_OK;
 }
 
-int32_t matmul(ugb_hybrid *m, const Mat &x) {
+int32_t ugb_hybrid_matmul(ugb_hybrid *m, const Mat &x) {
   ugb_device *dev = m->dev;
   if (m->f32) {
+    if (x.groups)
+      return ugb_f32_grouped_gemm(dev, (float *)x.out, (const float *)x.a, (const float *)x.w, x.groups, x.m, x.tile, (int)x.n, (int)x.k);
     int32_t rc = ugb_f32_gemm(dev, (float *)x.out, (const float *)x.a, (const float *)x.w, x.batch, x.m, x.n, x.k,
                               x.a_ld ? x.a_ld : x.k, x.a_batch, x.nk, x.w_batch, x.c_ld ? x.c_ld : x.n,
                               x.c_batch ? x.c_batch : x.m * (x.c_ld ? x.c_ld : x.n));
-    if (rc || !x.relu2) return rc;
+    if (rc || !(x.relu2 || x.silu_mul)) return rc;
+    if (x.silu_mul) return ugb_fail(dev, UGB_ERR_UNSUPPORTED, "f32 product with a fused gate");
     relu2_kernel<<<dev->sm_count * 4, 256, 0, dev->stream>>>((float *)x.out, x.m * x.n / 4);
     return ugb_after_launch(dev, "relu2_kernel");
   }
@@ -133,10 +72,12 @@ int32_t matmul(ugb_hybrid *m, const Mat &x) {
   g.a_batch = (long long)x.a_batch; g.b_batch = (long long)x.w_batch; g.c_batch = (long long)x.c_batch;
   g.a_ld = x.a_ld == x.k ? 0 : (long long)x.a_ld; g.c_ld = x.c_ld == x.n ? 0 : (long long)x.c_ld;
   g.b_is_nk = x.nk;
-  g.epi = x.relu2 ? UGB_EPI_RELU2_BF16 : (x.f32_out ? UGB_EPI_F32 : UGB_EPI_BF16);
-  g.splits = x.splits; g.bn = x.bn; g.b_static = true; g.pdl = m->pdl != 0; g.late_trigger = true;
-  g.smem_kib = x.m <= 64 ? 144 : 0;
-  if (!x.f32_out && x.batch == 1 && x.nk && x.m <= 64 && x.k >= 256) {
+  g.epi = x.relu2 ? UGB_EPI_RELU2_BF16 : x.silu_mul ? UGB_EPI_SILU_MUL_BF16 : (x.f32_out ? UGB_EPI_F32 : UGB_EPI_BF16);
+  if (x.silu_mul) g.c_ld = x.c_ld == x.n / 2 ? 0 : (long long)x.c_ld;
+  g.splits = x.splits; g.bn = x.bn; g.b_static = x.groups == nullptr; g.pdl = m->pdl != 0; g.late_trigger = true;
+  g.groups = x.groups; g.n_groups = x.n_groups; g.tile_m = x.tile;
+  g.smem_kib = x.m <= 64 || (x.groups && x.tile == 64) ? 144 : 0;
+  if (!x.f32_out && !x.groups && x.batch == 1 && x.nk && x.m <= 64 && x.k >= 256) {
     // a T result cannot be split into partials: the two k halves of a tile on a pair of CTAs, with the narrowest tile that fits the SMs
     for (int bn : {64, 96, 128, 160})
       if ((x.n + bn - 1) / bn * 2 <= (size_t)dev->sm_count) {
@@ -155,9 +96,8 @@ int32_t matmul(ugb_hybrid *m, const Mat &x) {
   return rc;
 }
 
-// k splits of a decode product with a f32 result: as many CTAs as SMs, no fewer than two k blocks each
-struct Tiling { int bn, splits; };
-Tiling tiling(const ugb_hybrid *m, size_t n, size_t k) {
+// As many CTAs as SMs, no fewer than two k blocks each
+Tiling ugb_hybrid_tile(const ugb_hybrid *m, size_t n, size_t k) {
   if (m->f32 || m->batch > 64) return {0, 1};
   // A CTA's time goes with its k blocks and hardly with its tile width (an MMA of 64 rows costs the same up to 160
   // columns), so: the fewest k blocks per CTA over widths and splits that fit one wave, then the fewest partials,
@@ -165,7 +105,7 @@ Tiling tiling(const ugb_hybrid *m, size_t n, size_t k) {
   const int sms = m->dev->sm_count, kb = (int)((k + 63) / 64);
   Tiling best{128, 1};
   int best_kb = kb + 1;
-  for (int s = 1; s <= std::min(8, kb); ++s)
+  for (int s = 1; s <= std::min(UGB_HYBRID_MAX_SPLITS, kb); ++s)
     for (int bn : {64, 80, 96, 128, 160}) {
       const int tiles = (int)((n + bn - 1) / bn), per = (kb + s - 1) / s;
       if (tiles * s > sms || per >= best_kb) continue;
@@ -175,9 +115,8 @@ Tiling tiling(const ugb_hybrid *m, size_t n, size_t k) {
   if (best_kb > kb) return {256, 1};           // more tiles than SMs whatever the width
   return {best.bn, ugb_tc_gemm_effective_splits(k, best.splits)};
 }
-constexpr int MAX_SPLITS = 8;
 
-template <typename T> int32_t launch_rows(ugb_hybrid *m, RowArgs<T> &a, int rows, bool early) {
+template <typename T> int32_t ugb_hybrid_rows(ugb_hybrid *m, RowArgs<T> &a, int rows, bool early) {
   if (!m->on(UGB_HYBRID_K_ROWS)) return UGB_OK;
   a.early = early ? 1 : 0;
   a.ld = m->wl; a.inv_width = 1.0f / (float)m->cfg.width; a.eps = m->cfg.eps; a.status = m->dev->status_dev;
@@ -194,6 +133,20 @@ template <typename T> int32_t launch_rows(ugb_hybrid *m, RowArgs<T> &a, int rows
   return ugb_after_launch(m->dev, "row_update_kernel");
 }
 
+template int32_t ugb_hybrid_rows<float>(ugb_hybrid *, RowArgs<float> &, int, bool);
+template int32_t ugb_hybrid_rows<__nv_bfloat16>(ugb_hybrid *, RowArgs<__nv_bfloat16> &, int, bool);
+
+int32_t ugb_hybrid_keep(ugb_hybrid *m, const ugb_hybrid_work &w, int run, int t_block, int off, int t) {
+  if (!m->keep_layers || !m->layer_out) return UGB_OK;     // rows (b, off + i) of [run][batch * t_block][wl]
+  const size_t wl = m->wl;
+  for (int b = 0; b < m->batch; ++b)
+    UGB_CUDA(m->dev, cudaMemcpyAsync(m->layer_out + ((size_t)run * m->batch * t_block + (size_t)b * t_block + off) * wl,
+                                     w.x + (size_t)b * t * wl, (size_t)t * wl * 4, cudaMemcpyDeviceToDevice, m->dev->stream));
+  return UGB_OK;
+}
+
+namespace {
+
 template <typename T>
 int32_t launch_conv(ugb_device *dev, const T *h, const float *w, const T *tail_in, T *tail_out, T *out, int b, int t, int taps, int ld) {
   const dim3 grid((unsigned)((t + CONV_STRIP - 1) / CONV_STRIP), (unsigned)((ld / 8 + 127) / 128), (unsigned)b);
@@ -201,7 +154,7 @@ int32_t launch_conv(ugb_device *dev, const T *h, const float *w, const T *tail_i
   if (taps == 2) k = causal_conv_kernel<T, 2>;
   else if (taps == 3) k = causal_conv_kernel<T, 3>;
   else if (taps == 4) k = causal_conv_kernel<T, 4>;
-  k<<<grid, 128, 0, dev->stream>>>(h, w, tail_in, tail_out, out, t, taps, ld);
+  k<<<grid, 128, 0, dev->stream>>>(h, (size_t)ld, w, nullptr, tail_in, tail_out, out, t, taps, ld);
   return ugb_after_launch(dev, "causal_conv_kernel");
 }
 
@@ -220,7 +173,7 @@ int32_t launch_scan(ugb_device *dev, const TI *pre, const float *bz, const float
 // One pass over all layers for rows (b, i), i < t, positions *pos + off + i.  decode: t == 1 and the convolutions and
 // recurrent states advance inside the row kernels.  Leaves the final norm's output in w.h.
 template <typename T>
-int32_t run_layers(ugb_hybrid *m, Work &w, const int *tok, int t_block, int off, int t, bool decode) {
+int32_t run_layers(ugb_hybrid *m, ugb_hybrid_work &w, const int *tok, int t_block, int off, int t, bool decode) {
   ugb_device *dev = m->dev;
   cudaStream_t st = dev->stream;
   const bool pdl = m->pdl != 0;
@@ -228,7 +181,7 @@ int32_t run_layers(ugb_hybrid *m, Work &w, const int *tok, int t_block, int off,
   // between one row kernel and the next: what earlier row kernels wrote is complete when a row kernel starts.
   const bool early = decode && pdl && !m->f32;
   const int B = m->batch, rows = B * t, wl = m->wl, taps = m->cfg.conv_taps;
-  const size_t bank_stride = (size_t)w.rows * wl, n_tail = taps > 1 ? (size_t)B * (taps - 1) * wl : 0;
+  const size_t bank_stride = (size_t)w.rows * wl;
   int32_t rc;
   cudaError_t e;
 
@@ -236,15 +189,15 @@ int32_t run_layers(ugb_hybrid *m, Work &w, const int *tok, int t_block, int off,
   auto input_of = [&](const float *conv, int layer, int which, const T **in) -> int32_t {
     *in = (const T *)w.h;
     if (decode || !conv) return UGB_OK;
-    const T *ti = (const T *)m->tails + ((size_t)layer * 2 + which) * n_tail;
-    T *to = (T *)m->tails_next + ((size_t)layer * 2 + which) * n_tail;
+    const T *ti = (const T *)(m->tails + m->runs[layer].tail[which]);
+    T *to = (T *)(m->tails_next + m->runs[layer].tail[which]);
     *in = (const T *)w.hc;
     return m->on(UGB_HYBRID_K_CONV) ? launch_conv<T>(dev, (const T *)w.h, conv, ti, to, (T *)w.hc, B, t, taps, wl) : UGB_OK;
   };
   auto fuse_conv = [&](RowArgs<T> &a, const float *conv, int layer, int which) {
     if (!decode || !conv) return;
     a.conv = conv; a.taps = taps;
-    a.tail = (T *)m->tails + ((size_t)layer * 2 + which) * n_tail;
+    a.tail = (T *)(m->tails + m->runs[layer].tail[which]);
   };
 
   {
@@ -255,52 +208,53 @@ int32_t run_layers(ugb_hybrid *m, Work &w, const int *tok, int t_block, int off,
     a.gain = m->layers.empty() ? m->final_gain : m->layers[0].norm1;
     a.h = (T *)w.h;
     if (!m->layers.empty()) fuse_conv(a, m->layers[0].conv1, 0, 0);
-    if ((rc = launch_rows<T>(m, a, rows, early))) return rc;
+    if ((rc = ugb_hybrid_rows<T>(m, a, rows, early))) return rc;
   }
   const int n_layers = (int)m->layers.size();
   for (int i = 0; i < n_layers; ++i) {
-    Layer &L = m->layers[i];
+    const ugb_hybrid_weights &L = m->layers[i];
+    const ugb_hybrid_run &R = m->runs[i];
     const T *in = nullptr;
     if ((rc = input_of(L.conv1, i, 0, &in))) return rc;
     Tiling out_t{0, 1};
     if (L.d.mixer == UGB_MIXER_MINGRU) {
-      const Tiling ti = decode ? tiling(m, 3 * (size_t)L.ul, wl) : Tiling{0, 1};
+      const Tiling ti = decode ? ugb_hybrid_tile(m, 3 * (size_t)L.ul, wl) : Tiling{0, 1};
       if (m->on(UGB_HYBRID_K_GRU_IN)) {
         Mat g{w.pre, in, L.w_in, (size_t)rows, 3 * (size_t)L.ul, (size_t)wl};
         g.splits = ti.splits; g.bn = ti.bn;
         g.f32_out = decode || m->f32;            // a block's projection is rounded to T, a step's partials are summed in f32
-        if ((rc = matmul(m, g))) return rc;
+        if ((rc = ugb_hybrid_matmul(m, g))) return rc;
       }
       if (m->on(UGB_HYBRID_K_GRU)) {
         if (decode) {
           e = ugb_launch(min_gru_step_kernel<T>, dim3(rows, (L.ul / 4 + 127) / 128), dim3(128), 0, st, pdl, w.pre, ti.splits,
-                         (size_t)rows * 3 * L.ul, L.bz, L.bu, L.state, (T *)w.mid, L.ul);
+                         (size_t)rows * 3 * L.ul, L.bz, L.bu, R.state, (T *)w.mid, L.ul);
           if (e != cudaSuccess) return ugb_fail(dev, UGB_ERR_CUDA, "launch of min_gru_step_kernel failed: %s", cudaGetErrorString(e));
           if ((rc = ugb_after_launch(dev, "min_gru_step_kernel"))) return rc;
-        } else if ((rc = launch_scan<T, T>(dev, (const T *)w.pre, L.bz, L.bu, L.state, (T *)w.mid, B, t, L.ul))) {
+        } else if ((rc = launch_scan<T, T>(dev, (const T *)w.pre, L.bz, L.bu, R.state, (T *)w.mid, B, t, L.ul))) {
           return rc;
         }
       }
-      if (decode) out_t = tiling(m, wl, L.ul);
+      if (decode) out_t = ugb_hybrid_tile(m, wl, L.ul);
       if (m->on(UGB_HYBRID_K_OUT)) {
         Mat g{w.pre, w.mid, L.w_out, (size_t)rows, (size_t)wl, (size_t)L.ul};
         g.splits = out_t.splits; g.bn = out_t.bn;
-        if ((rc = matmul(m, g))) return rc;
+        if ((rc = ugb_hybrid_matmul(m, g))) return rc;
       }
     } else {
       const int H = L.d.heads, n_in = L.ql + L.cl + L.gl;
-      const Tiling ti = decode ? tiling(m, n_in, wl) : Tiling{0, 1};
+      const Tiling ti = decode ? ugb_hybrid_tile(m, n_in, wl) : Tiling{0, 1};
       if (m->on(UGB_HYBRID_K_LATENT_IN)) {
         Mat g{w.pre, in, L.w_in, (size_t)rows, (size_t)n_in, (size_t)wl};
         g.splits = ti.splits; g.bn = ti.bn;
-        if ((rc = matmul(m, g))) return rc;
+        if ((rc = ugb_hybrid_matmul(m, g))) return rc;
       }
       if (m->on(UGB_HYBRID_K_LATENT_ROWS)) {
         const int threads = std::min(512, (n_in / 4 + 31) / 32 * 32), per = (n_in / 4 + threads - 1) / threads;
         auto *k = decode ? (per <= 1 ? latent_inputs_kernel<T, 1, 8> : per <= 2 ? latent_inputs_kernel<T, 2, 8> : latent_inputs_kernel<T, 16, 1>)
                          : (per <= 1 ? latent_inputs_kernel<T, 1, 1> : per <= 2 ? latent_inputs_kernel<T, 2, 1> : per <= 4 ? latent_inputs_kernel<T, 4, 1> : latent_inputs_kernel<T, 16, 1>);
         e = ugb_launch(k, dim3(rows), dim3(threads), 0, st, pdl, w.pre, ti.splits, (size_t)rows * n_in,
-                       L.q_gain, L.c_gain, (T *)w.cq, (T *)L.cache, w.gate, m->pos, off, t, m->t_max, L.ql, L.cl, L.gl,
+                       L.q_gain, L.c_gain, (T *)w.cq, (T *)R.cache, w.gate, m->pos, off, t, m->t_max, L.ql, L.cl, L.gl,
                        1.0f / (float)L.d.q_rank, 1.0f / (float)L.d.kv_rank, m->cfg.eps, dev->status_dev);
         if (e != cudaSuccess) return ugb_fail(dev, UGB_ERR_CUDA, "launch of latent_inputs_kernel failed: %s", cudaGetErrorString(e));
         if ((rc = ugb_after_launch(dev, "latent_inputs_kernel"))) return rc;
@@ -309,17 +263,17 @@ int32_t run_layers(ugb_hybrid *m, Work &w, const int *tok, int t_block, int off,
       if (m->on(UGB_HYBRID_K_UQ)) {
         Mat g{w.q, w.cq, L.w_uq, (size_t)rows, qw, (size_t)L.ql};
         g.f32_out = false;
-        if ((rc = matmul(m, g))) return rc;
+        if ((rc = ugb_hybrid_matmul(m, g))) return rc;
       }
       if (!decode && L.expand && t > m->absorb_max) {
         const size_t ctx = (size_t)m->host_pos + off + t;        // positions cached once this block is in
         if (m->on(UGB_HYBRID_K_ABSORB)) {
-          Mat g{m->kx, L.cache, L.w_uk, ctx, qw, (size_t)L.cl};
+          Mat g{m->kx, R.cache, L.w_uk, ctx, qw, (size_t)L.cl};
           g.f32_out = false;
           g.batch = B; g.a_batch = (size_t)m->t_max * L.cl; g.c_batch = ctx * qw;
-          if ((rc = matmul(m, g))) return rc;
+          if ((rc = ugb_hybrid_matmul(m, g))) return rc;
           g.out = m->vx; g.w = L.w_uv; g.n = ow; g.c_batch = ctx * ow;
-          if ((rc = matmul(m, g))) return rc;
+          if ((rc = ugb_hybrid_matmul(m, g))) return rc;
         }
         if (m->on(UGB_HYBRID_K_ATTENTION)) {
           ugb_prefill_attention_args a;
@@ -334,11 +288,11 @@ int32_t run_layers(ugb_hybrid *m, Work &w, const int *tok, int t_block, int off,
           g.f32_out = false; g.nk = false;
           g.batch = H; g.a_ld = qw; g.a_batch = L.dp; g.w_batch = (size_t)L.dp * L.cl; g.c_ld = lw; g.c_batch = L.cl;
           if (rows <= 64) g.bn = 64;
-          if ((rc = matmul(m, g))) return rc;
+          if ((rc = ugb_hybrid_matmul(m, g))) return rc;
         }
         if (m->on(UGB_HYBRID_K_ATTENTION)) {
           ugb_latent_attention_args a{};
-          a.q = w.ql; a.cache = L.cache; a.out = w.ol; a.gate = w.gate; a.f32 = m->f32; a.rows = rows; a.t = t;
+          a.q = w.ql; a.cache = R.cache; a.out = w.ol; a.gate = w.gate; a.f32 = m->f32; a.rows = rows; a.t = t;
           a.pos_p = m->pos; a.pos_off = off; a.heads = H; a.ld = L.cl; a.t_max = m->t_max; a.gate_ld = L.gl; a.scale = L.d.scale;
           a.splits = decode ? m->att_splits() : 1;
           a.pdl = pdl; a.early = early;
@@ -349,14 +303,14 @@ int32_t run_layers(ugb_hybrid *m, Work &w, const int *tok, int t_block, int off,
           g.f32_out = false;
           g.batch = H; g.a_ld = lw; g.a_batch = L.cl; g.w_batch = (size_t)L.vp * L.cl; g.c_ld = ow; g.c_batch = L.vp;
           if (rows <= 64) g.bn = 64;
-          if ((rc = matmul(m, g))) return rc;
+          if ((rc = ugb_hybrid_matmul(m, g))) return rc;
         }
       }
-      if (decode) out_t = tiling(m, wl, ow);
+      if (decode) out_t = ugb_hybrid_tile(m, wl, ow);
       if (m->on(UGB_HYBRID_K_OUT)) {
         Mat g{w.pre, w.o, L.w_out, (size_t)rows, (size_t)wl, ow};
         g.splits = out_t.splits; g.bn = out_t.bn;
-        if ((rc = matmul(m, g))) return rc;
+        if ((rc = ugb_hybrid_matmul(m, g))) return rc;
       }
     }
     // stream += norm(mixer output); with a feed-forward its input follows, else the layer ends here
@@ -373,43 +327,41 @@ int32_t run_layers(ugb_hybrid *m, Work &w, const int *tok, int t_block, int off,
     a.post_gain = L.norm1b; a.x = w.x; a.h = (T *)w.h;
     if (L.d.feed_forward == UGB_FF_NONE) layer_end(a);
     else { a.gain = L.norm2; fuse_conv(a, L.conv2, i, 1); }
-    if ((rc = launch_rows<T>(m, a, rows, early))) return rc;
+    if ((rc = ugb_hybrid_rows<T>(m, a, rows, early))) return rc;
     if (L.d.feed_forward != UGB_FF_NONE) {
       if ((rc = input_of(L.conv2, i, 1, &in))) return rc;
       if (m->on(UGB_HYBRID_K_UP)) {
         Mat g{w.mid, in, L.w_up, (size_t)rows, (size_t)L.fl, (size_t)wl};
         g.f32_out = false; g.relu2 = true;
-        if ((rc = matmul(m, g))) return rc;
+        if ((rc = ugb_hybrid_matmul(m, g))) return rc;
       }
-      const Tiling td = decode ? tiling(m, wl, L.fl) : Tiling{0, 1};
+      const Tiling td = decode ? ugb_hybrid_tile(m, wl, L.fl) : Tiling{0, 1};
       if (m->on(UGB_HYBRID_K_DOWN)) {
         Mat g{w.pre, w.mid, L.w_down, (size_t)rows, (size_t)wl, (size_t)L.fl};
         g.splits = td.splits; g.bn = td.bn;
-        if ((rc = matmul(m, g))) return rc;
+        if ((rc = ugb_hybrid_matmul(m, g))) return rc;
       }
       RowArgs<T> f;
       f.part = w.pre; f.n_part = td.splits; f.part_stride = (size_t)rows * wl;
       f.post_gain = L.norm2b; f.x = w.x; f.h = (T *)w.h;
       layer_end(f);
-      if ((rc = launch_rows<T>(m, f, rows, early))) return rc;
+      if ((rc = ugb_hybrid_rows<T>(m, f, rows, early))) return rc;
     }
-    if (!decode && m->keep_layers && m->layer_out) {     // rows (b, off + i) of [layer][batch * t_block][wl]
-      for (int b = 0; b < B; ++b)
-        UGB_CUDA(dev, cudaMemcpyAsync(m->layer_out + ((size_t)i * B * t_block + (size_t)b * t_block + off) * wl,
-                                      w.x + (size_t)b * t * wl, (size_t)t * wl * 4, cudaMemcpyDeviceToDevice, st));
-    }
+    if (!decode && (rc = ugb_hybrid_keep(m, w, i, t_block, off, t))) return rc;
   }
   return UGB_OK;
 }
 
-int32_t run_layers_any(ugb_hybrid *m, Work &w, const int *tok, int t_block, int off, int t, bool decode) {
+int32_t run_layers_any(ugb_hybrid *m, ugb_hybrid_work &w, const int *tok, int t_block, int off, int t, bool decode) {
+  if (m->parallel()) return ugb_parallel_run(m, w, tok, t_block, off, t, decode);
   return m->f32 ? run_layers<float>(m, w, tok, t_block, off, t, decode) : run_layers<__nv_bfloat16>(m, w, tok, t_block, off, t, decode);
 }
 
-int32_t alloc_work(ugb_hybrid *m, Work &w, int rows, bool decode) {
-  const size_t R = rows, es = m->es(), wl = m->wl, splits = decode ? MAX_SPLITS : 1;
+int32_t alloc_work(ugb_hybrid *m, ugb_hybrid_work &w, int rows, bool decode) {
+  if (m->parallel()) return ugb_parallel_work(m, w, rows, decode);
+  const size_t R = rows, es = m->es(), wl = m->wl, splits = decode ? UGB_HYBRID_MAX_SPLITS : 1;
   size_t pre = wl, mid = 8, ql = 8, gl = 8, q = 8, lat = 8, o = 8;
-  for (const Layer &L : m->layers) {
+  for (const ugb_hybrid_weights &L : m->layers) {
     pre = std::max({pre, (size_t)3 * L.ul, (size_t)(L.ql + L.cl + L.gl)});
     mid = std::max({mid, (size_t)L.ul, (size_t)L.fl});
     ql = std::max(ql, (size_t)L.ql); gl = std::max(gl, (size_t)L.gl);
@@ -422,43 +374,14 @@ int32_t alloc_work(ugb_hybrid *m, Work &w, int rows, bool decode) {
   int32_t rc;
   const size_t banks = m->cfg.depth_average ? std::max<size_t>(1, m->layers.size()) : 0;
   if ((rc = dmalloc(m, &w.x, R * wl)) || (rc = dmalloc(m, &w.pre, splits * R * pre)) || (rc = dmalloc(m, &w.gate, R * gl)) ||
-      (rc = dmalloc(m, &w.bank, banks * R * wl)) || (rc = alloc_bytes(m, &w.h, R * wl * es, true)) ||
-      (rc = alloc_bytes(m, &w.hc, decode ? 16 : R * wl * es, false)) || (rc = alloc_bytes(m, &w.mid, R * mid * es, false)) ||
-      (rc = alloc_bytes(m, &w.cq, R * ql * es, false)) || (rc = alloc_bytes(m, &w.q, R * q * es, false)) ||
-      (rc = alloc_bytes(m, &w.ql, R * lat * es, false)) || (rc = alloc_bytes(m, &w.ol, R * lat * es, false)) ||
-      (rc = alloc_bytes(m, &w.o, R * o * es, false)))
+      (rc = dmalloc(m, &w.bank, banks * R * wl)) || (rc = ugb_hybrid_alloc(m, &w.h, R * wl * es, true)) ||
+      (rc = ugb_hybrid_alloc(m, &w.hc, decode ? 16 : R * wl * es, false)) || (rc = ugb_hybrid_alloc(m, &w.mid, R * mid * es, false)) ||
+      (rc = ugb_hybrid_alloc(m, &w.cq, R * ql * es, false)) || (rc = ugb_hybrid_alloc(m, &w.q, R * q * es, false)) ||
+      (rc = ugb_hybrid_alloc(m, &w.ql, R * lat * es, false)) || (rc = ugb_hybrid_alloc(m, &w.ol, R * lat * es, false)) ||
+      (rc = ugb_hybrid_alloc(m, &w.o, R * o * es, false)))
     return rc;
   w.rows = rows;
   return UGB_OK;
-}
-
-// gain[i] = offset + w[i], zero behind n
-__global__ void gain_kernel(const float *__restrict__ w, float *__restrict__ gain, int n, float offset) {
-  const int i = blockIdx.x * blockDim.x + threadIdx.x;
-  if (i < n) gain[i] = offset + w[i];
-}
-// conv weights [width][taps] -> [taps][ld]
-__global__ void taps_kernel(const float *__restrict__ w, float *__restrict__ out, int width, int taps, int ld) {
-  const int i = blockIdx.x * blockDim.x + threadIdx.x;
-  if (i < width * taps) out[(size_t)(i % taps) * ld + i / taps] = w[i];
-}
-
-// The tensor as f32 in stream-ordered scratch, handed to `use`.
-template <typename F>
-int32_t with_f32(ugb_hybrid *m, const ugb_slice *w, size_t n, const char *name, F use) {
-  ugb_device *dev = m->dev;
-  void *tmp = nullptr;
-  UGB_CUDA(dev, ugb_malloc_async(dev, &tmp, n * 4));
-  int32_t rc = engine_put_matrix(m, w, tmp, UGB_F32, 1, n, 0, 1, 0, n, n, name);
-  if (!rc) rc = use((const float *)tmp);
-  cudaFreeAsync(tmp, dev->stream);
-  return rc;
-}
-int32_t put_gain(ugb_hybrid *m, const ugb_slice *w, float *dst, int n, float offset, const char *name) {
-  return with_f32(m, w, n, name, [&](const float *s) {
-    gain_kernel<<<(n + 255) / 256, 256, 0, m->dev->stream>>>(s, dst, n, offset);
-    return ugb_after_launch(m->dev, "gain_kernel");
-  });
 }
 
 }  // namespace
@@ -474,9 +397,9 @@ int32_t ugb_hybrid::ensure_prefill_workspace() {
   int32_t rc;
   if ((rc = alloc_work(this, pf, batch * chunk, false))) return rc;
   size_t k = 0, v = 0;
-  for (const Layer &L : layers)
-    if (L.expand) { k = std::max(k, (size_t)L.d.heads * L.dp); v = std::max(v, (size_t)L.d.heads * L.vp); }
-  if ((rc = alloc_bytes(this, &kx, (size_t)batch * t_max * k * es(), false)) || (rc = alloc_bytes(this, &vx, (size_t)batch * t_max * v * es(), false)))
+  for (const ugb_hybrid_weights &L : layers)
+    if (L.expand && !parallel()) { k = std::max(k, (size_t)L.d.heads * L.dp); v = std::max(v, (size_t)L.d.heads * L.vp); }
+  if ((rc = ugb_hybrid_alloc(this, &kx, (size_t)batch * t_max * k * es(), false)) || (rc = ugb_hybrid_alloc(this, &vx, (size_t)batch * t_max * v * es(), false)))
     return rc;
   pf_chunk = chunk;
   pf_rows = batch * chunk;
@@ -485,7 +408,7 @@ int32_t ugb_hybrid::ensure_prefill_workspace() {
 
 int32_t ugb_hybrid::enqueue_prefill_chunk(const int *tok, int t, int c0, int tc, bool all_logits) {
   if (keep_layers && c0 == 0) {
-    const size_t need = layers.size() * (size_t)batch * t * wl;
+    const size_t need = runs.size() * (size_t)batch * t * wl;
     if (need > layer_cap) {
       float *p = nullptr;
       if (int32_t rc = dmalloc(this, &p, need)) return rc;    // freed with the model
@@ -501,7 +424,10 @@ int32_t ugb_hybrid::enqueue_prefill_chunk(const int *tok, int t, int c0, int tc,
   if (all_logits) {
     Mat g{pf_logits + (size_t)c0 * logits_ld, pf.h, head, (size_t)tc, (size_t)logits_ld, (size_t)wl};
     g.batch = batch; g.a_batch = (size_t)tc * wl; g.c_batch = (size_t)t * logits_ld;
-    if ((rc = matmul(this, g))) return rc;
+    if ((rc = ugb_hybrid_matmul(this, g))) return rc;
+    if (cfg.logit_softcap > 0.f)
+      for (int b = 0; b < batch; ++b)
+        if ((rc = ugb_parallel_softcap(this, pf_logits + ((size_t)b * t + c0) * logits_ld, (size_t)tc * logits_ld))) return rc;
   }
   return UGB_OK;
 }
@@ -520,8 +446,9 @@ int32_t ugb_hybrid::enqueue_head(bool) {
   Mat g{logits, dec.h, head, (size_t)batch, (size_t)logits_ld, (size_t)wl};
   if (!f32 && batch <= 64) g.bn = logits_ld > 128 * dev->sm_count ? 256 : 128;
   int32_t rc;
-  if ((rc = matmul(this, g))) return rc;
+  if ((rc = ugb_hybrid_matmul(this, g))) return rc;
   if (only != UGB_HYBRID_K_ALL) return UGB_OK;
+  if (cfg.logit_softcap > 0.f && (rc = ugb_parallel_softcap(this, logits, (size_t)batch * logits_ld))) return rc;
   cudaError_t e = ugb_launch(ugb_decode::argmax_rows_kernel, dim3(batch), dim3(1024), 0, dev->stream, pdl != 0, logits, vl, logits_ld, next, pos);
   if (e != cudaSuccess) return ugb_fail(dev, UGB_ERR_CUDA, "launch of argmax_rows_kernel failed: %s", cudaGetErrorString(e));
   return ugb_after_launch(dev, "argmax_rows_kernel");
@@ -552,10 +479,19 @@ int32_t ugb_hybrid_create(ugb_device *dev, const ugb_hybrid_config *cfg, const u
 #define TRY(e) do { if ((rc = (e)) != UGB_OK) { engine_free(m); delete m; return rc; } } while (0)
 #define CHECK(cond, code, ...) do { if (!(cond)) { rc = ugb_fail(dev, code, __VA_ARGS__); engine_free(m); delete m; return rc; } } while (0)
   m->layers.resize(cfg->layers);
-  for (int i = 0; i < cfg->layers; ++i) {
-    Layer &L = m->layers[i];
-    L.d = layers[i];
+  CHECK(cfg->form == UGB_FORM_SANDWICH || cfg->form == UGB_FORM_PARALLEL, UGB_ERR_UNSUPPORTED, "form %d of the layers", cfg->form);
+  for (int i = 0; i < cfg->layers; ++i) m->layers[i].d = layers[i];
+  if (m->parallel()) TRY(ugb_parallel_model(m));
+  else m->runs.resize(cfg->layers);
+  for (int i = 0; i < cfg->layers && !m->parallel(); ++i) {
+    ugb_hybrid_weights &L = m->layers[i];
+    ugb_hybrid_run &R = m->runs[i];
+    R.layer = i;
     const ugb_hybrid_layer &d = L.d;
+    for (int k = 0; k < 2 && cfg->conv_taps > 1; ++k) {
+      R.tail[k] = m->tail_bytes;
+      m->tail_bytes += (size_t)batch * (cfg->conv_taps - 1) * wl * es;
+    }
     TRY(dmalloc(m, &L.norm1, wl, true));
     TRY(dmalloc(m, &L.norm1b, wl, true));
     if (cfg->conv_taps) TRY(dmalloc(m, &L.conv1, cfg->conv_taps * wl, true));
@@ -567,18 +503,19 @@ int32_t ugb_hybrid_create(ugb_device *dev, const ugb_hybrid_config *cfg, const u
       TRY(dmalloc(m, &L.norm2, wl, true));
       TRY(dmalloc(m, &L.norm2b, wl, true));
       if (cfg->conv_taps) TRY(dmalloc(m, &L.conv2, cfg->conv_taps * wl, true));
-      TRY(alloc_bytes(m, &L.w_up, L.fl * wl * es, true));
-      TRY(alloc_bytes(m, &L.w_down, wl * L.fl * es, true));
+      TRY(ugb_hybrid_alloc(m, &L.w_up, L.fl * wl * es, true));
+      TRY(ugb_hybrid_alloc(m, &L.w_down, wl * L.fl * es, true));
     }
     if (d.mixer == UGB_MIXER_MINGRU) {
       CHECK(d.width > 0, UGB_ERR_INVALID, "layer %d: %d recurrent channels", i, d.width);
       L.d.heads = 0;
       L.ul = (int)up8(d.width);
-      TRY(alloc_bytes(m, &L.w_in, 3 * (size_t)L.ul * wl * es, true));
-      TRY(alloc_bytes(m, &L.w_out, wl * L.ul * es, true));
+      TRY(ugb_hybrid_alloc(m, &L.w_in, 3 * (size_t)L.ul * wl * es, true));
+      TRY(ugb_hybrid_alloc(m, &L.w_out, wl * L.ul * es, true));
       TRY(dmalloc(m, &L.bz, L.ul, true));
       TRY(dmalloc(m, &L.bu, L.ul, true));
-      TRY(dmalloc(m, &L.state, (size_t)batch * L.ul, true));
+      R.state_len = (size_t)batch * L.ul;
+      TRY(dmalloc(m, &R.state, R.state_len, true));
     } else {
       CHECK(d.mixer == UGB_MIXER_LATENT_ATTENTION, UGB_ERR_UNSUPPORTED, "layer %d: mixer kind %d", i, d.mixer);
       CHECK(d.heads > 0 && d.dim > 0 && d.vdim > 0 && d.q_rank > 0 && d.kv_rank > 0, UGB_ERR_INVALID, "layer %d: non-positive attention dimension", i);
@@ -591,21 +528,20 @@ int32_t ugb_hybrid_create(ugb_device *dev, const ugb_hybrid_config *cfg, const u
       L.dp = L.expand ? dp : (int)up8(d.dim);
       L.vp = L.expand ? vp : (int)up8(d.vdim);
       CHECK(L.ql + L.cl + L.gl <= 16 * 4 * 512, UGB_ERR_UNSUPPORTED, "layer %d: latents of %d + %d values", i, d.q_rank, d.kv_rank);
-      TRY(alloc_bytes(m, &L.w_in, (size_t)(L.ql + L.cl + L.gl) * wl * es, true));
-      TRY(alloc_bytes(m, &L.w_uq, (size_t)d.heads * L.dp * L.ql * es, true));
-      TRY(alloc_bytes(m, &L.w_uk, (size_t)d.heads * L.dp * L.cl * es, true));
-      TRY(alloc_bytes(m, &L.w_uv, (size_t)d.heads * L.vp * L.cl * es, true));
-      TRY(alloc_bytes(m, &L.w_out, wl * d.heads * L.vp * es, true));
+      TRY(ugb_hybrid_alloc(m, &L.w_in, (size_t)(L.ql + L.cl + L.gl) * wl * es, true));
+      TRY(ugb_hybrid_alloc(m, &L.w_uq, (size_t)d.heads * L.dp * L.ql * es, true));
+      TRY(ugb_hybrid_alloc(m, &L.w_uk, (size_t)d.heads * L.dp * L.cl * es, true));
+      TRY(ugb_hybrid_alloc(m, &L.w_uv, (size_t)d.heads * L.vp * L.cl * es, true));
+      TRY(ugb_hybrid_alloc(m, &L.w_out, wl * d.heads * L.vp * es, true));
       TRY(dmalloc(m, &L.q_gain, L.ql, true));
       TRY(dmalloc(m, &L.c_gain, L.cl, true));
-      TRY(alloc_bytes(m, &L.cache, (size_t)batch * m->t_max * L.cl * es, true));
+      TRY(ugb_hybrid_alloc(m, &R.cache, (size_t)batch * m->t_max * L.cl * es, true));
     }
   }
-  TRY(alloc_bytes(m, &m->embed, (size_t)cfg->vocab * wl * es, true));
-  TRY(alloc_bytes(m, &m->head, (size_t)m->logits_ld * wl * es, true));
+  TRY(ugb_hybrid_alloc(m, &m->embed, (size_t)cfg->vocab * wl * es, true));
+  TRY(ugb_hybrid_alloc(m, &m->head, (size_t)m->logits_ld * wl * es, true));
   TRY(dmalloc(m, &m->embed_gain, wl, true));
   TRY(dmalloc(m, &m->final_gain, wl, true));
-  m->tail_bytes = cfg->conv_taps > 1 ? (size_t)cfg->layers * 2 * batch * (cfg->conv_taps - 1) * wl * es : 0;
   TRY(dmalloc(m, &m->tails, m->tail_bytes, true));
   TRY(dmalloc(m, &m->tails_next, m->tail_bytes, true));
   TRY(dmalloc(m, &m->logits, (size_t)batch * m->logits_ld, true));
@@ -613,6 +549,7 @@ int32_t ugb_hybrid_create(ugb_device *dev, const ugb_hybrid_config *cfg, const u
   TRY(dmalloc(m, &m->pos, 1, true));
   TRY(alloc_work(m, m->dec, batch, true));
   TRY(ugb_latent_attention_prepare(dev));
+  TRY(ugb_grouped_attention_prepare(dev));
 #undef TRY
 #undef CHECK
   *out = m;
@@ -649,26 +586,33 @@ int32_t ugb_hybrid_load_weight(ugb_hybrid *m, const char *name, const ugb_slice 
   auto vec = [&](float *dst, size_t n) { return engine_put_matrix(m, w, dst, UGB_F32, 1, n, 0, 1, 0, n, n, name); };
   auto conv = [&](float *dst) {
     UGB_REQUIRE(dev, dst != nullptr, UGB_ERR_INVALID, "%s: the model has no input convolution there", name);
-    return with_f32(m, w, W * c.conv_taps, name, [&](const float *src) {
+    return ugb_hybrid_f32(m, w, W * c.conv_taps, name, [&](const float *src) {
       taps_kernel<<<((int)W * c.conv_taps + 255) / 256, 256, 0, dev->stream>>>(src, dst, (int)W, c.conv_taps, (int)wl);
       return ugb_after_launch(dev, "taps_kernel");
     });
   };
   auto gain = [&](float *dst) {
     UGB_REQUIRE(dev, dst != nullptr, UGB_ERR_INVALID, "%s: the layer has no such norm", name);
-    return put_gain(m, w, dst, (int)W, c.gain_offset, name);
+    return ugb_hybrid_gain(m, w, dst, (int)W, c.gain_offset, name);
   };
   m->loaded++;
   if (s == "embed") return put(m->embed, c.vocab, W, wl);
   if (s == "head") return put(m->head, c.vocab, W, wl);
-  if (s == "embed.norm") return gain(m->embed_gain);
+  if (s == "embed.norm" && !m->parallel()) return gain(m->embed_gain);
   if (s == "final.norm") return gain(m->final_gain);
+  if (m->parallel()) {
+    bool known = true;
+    const int32_t rc = ugb_parallel_load(m, name, w, &known);
+    if (known) return rc;
+    m->loaded--;
+    return ugb_fail(dev, UGB_ERR_INVALID, "unknown weight name %s", name);
+  }
   const size_t dot = s.find('.');
   if (s.size() > 1 && s[0] == 'l' && dot != std::string::npos && dot > 1 &&
       s.find_first_not_of("0123456789", 1) == dot && dot < 10) {
     const int i = atoi(s.c_str() + 1);
     UGB_REQUIRE(dev, i < c.layers, UGB_ERR_INVALID, "%s: layer index out of range", name);
-    Layer &L = m->layers[i];
+    ugb_hybrid_weights &L = m->layers[i];
     const ugb_hybrid_layer &d = L.d;
     const std::string k = s.substr(dot + 1);
     if (k == "norm1") return gain(L.norm1);
@@ -742,8 +686,8 @@ int32_t ugb_hybrid_reset(ugb_hybrid *m, int32_t pos) {
   if (pos == 0) {
     UGB_CUDA(dev, cudaSetDevice(dev->ordinal));
     if (m->tail_bytes) UGB_CUDA(dev, cudaMemsetAsync(m->tails, 0, m->tail_bytes, dev->stream));
-    for (const Layer &L : m->layers)
-      if (L.state) UGB_CUDA(dev, cudaMemsetAsync(L.state, 0, (size_t)m->batch * L.ul * 4, dev->stream));
+    for (const ugb_hybrid_run &R : m->runs)
+      if (R.state) UGB_CUDA(dev, cudaMemsetAsync(R.state, 0, R.state_len * 4, dev->stream));
   }
   return engine_reset(m, pos);
 }
@@ -771,7 +715,7 @@ int32_t ugb_hybrid_read(ugb_hybrid *m, int32_t what, void *host_dst, size_t len)
       return engine_read_rows(m, m->pf_logits, (size_t)m->batch * m->pf_logits_t, m->vl, m->logits_ld, host_dst, len);
     case UGB_HYBRID_LAYERS:
       UGB_REQUIRE(dev, m->layer_out, UGB_ERR_INVALID, "no layer outputs: set option keep_layers and run ugb_hybrid_prefill first");
-      return engine_read_rows(m, m->layer_out, m->layers.size() * (size_t)m->layer_rows, m->cfg.width, m->wl, host_dst, len);
+      return engine_read_rows(m, m->layer_out, m->runs.size() * (size_t)m->layer_rows, m->cfg.width, m->wl, host_dst, len);
     default: return ugb_fail(dev, UGB_ERR_INVALID, "ugb_hybrid_read: unknown selector %d", what);
   }
 }
@@ -779,9 +723,11 @@ int32_t ugb_hybrid_read(ugb_hybrid *m, int32_t what, void *host_dst, size_t len)
 uint64_t ugb_hybrid_state_bytes(const ugb_hybrid *m, int32_t positions) {
   if (!m) return 0;
   uint64_t n = m->tail_bytes / m->batch;
-  for (const Layer &L : m->layers) {
-    if (L.state) n += (uint64_t)L.ul * 4;
-    if (L.cache) n += (uint64_t)positions * L.cl * m->es();
+  for (const ugb_hybrid_run &R : m->runs) {
+    const ugb_hybrid_weights &L = m->layers[R.layer];
+    if (R.state) n += R.state_len / m->batch * 4;
+    if (R.vcache) n += (uint64_t)positions * L.d.kv_heads * (L.dp + L.vp) * m->es();
+    else if (R.cache) n += (uint64_t)positions * L.cl * m->es();
   }
   return n;
 }
@@ -966,12 +912,12 @@ int32_t ugb_residual_update(ugb_device *dev, ugb_slice *x, const ugb_slice *y, c
     RowArgs<float> a;
     fill(a);
     a.h = (float *)h->ptr;
-    return launch_rows<float>(&m, a, (int)rows, false);
+    return ugb_hybrid_rows<float>(&m, a, (int)rows, false);
   }
   RowArgs<__nv_bfloat16> a;
   fill(a);
   a.h = (__nv_bfloat16 *)h->ptr;
-  return launch_rows<__nv_bfloat16>(&m, a, (int)rows, false);
+  return ugb_hybrid_rows<__nv_bfloat16>(&m, a, (int)rows, false);
 }
 
 }  // extern "C"

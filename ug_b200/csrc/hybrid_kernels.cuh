@@ -1,5 +1,6 @@
 // Row kernels of the layer-list engine (hybrid_engine.cu): everything between the matrix products of a decoder whose
-// layers are recurrent or latent-attention mixers with sandwich norms, input convolutions and a depth average.
+// layers are recurrent or latent-attention mixers with sandwich norms, input convolutions and a depth average; the residual
+// update and the convolution also serve layers in the parallel form (parallel_kernels.cuh).
 //
 // T is the activation type (bf16, or f32 when the model runs in 32 bits).  Norms, the residual stream, the layer
 // bank, gates and the recurrence are f32 whatever T is.  Every row buffer is `ld` elements wide (a multiple of 8, the
@@ -63,10 +64,11 @@ __device__ __forceinline__ float sq4(float4 v) { return (v.x * v.x + v.y * v.y) 
 
 // ------------------------------------------------------------- row update ---
 // One CTA per row r, in this order:
-//   y   = sum of the projection partials, or the embedding row of token id(r)
+//   y   = sum of the projection partials, or the embedding row of token id(r);  + sum_k routed[slot[r][k]];  + bias
 //   x   = x + norm(y) * post_gain          (post_gain null: y itself; add_x 0: the stream starts here)
 //   bank_out = x;  x = sum_j dwa[j] bank[j] + dwa[n_avg] x        (with a depth average)
-//   h   = norm(x) * gain, rounded to T
+//   copy = x rounded to T (twice, where a second place is given)
+//   h   = norm(x) * gain, rounded to T     (gain null: none)
 //   h   = h + sum_j conv[j] h_(-taps+1+j)  (conv set: one new position per sequence; the tail of earlier h's is the
 //                                           sequence's state and moves on by one)
 template <typename T> struct RowArgs {
@@ -76,6 +78,10 @@ template <typename T> struct RowArgs {
   const float *part = nullptr;         // or projection partials [n_part][rows][ld]
   int n_part = 0;
   size_t part_stride = 0;
+  const float *routed = nullptr;       // rows of other products that belong to this one: slot[r][k] < 0 = none
+  const int *slot = nullptr;
+  int top = 0;
+  const float *bias = nullptr;         // [ld], joins y
   const float *post_gain = nullptr;
   float *x = nullptr;
   int add_x = 1;
@@ -86,6 +92,10 @@ template <typename T> struct RowArgs {
   int n_avg = 0;
   const float *gain = nullptr;
   T *h = nullptr;
+  T *copy = nullptr, *copy2 = nullptr; // rows copy_ld apart
+  size_t copy_ld = 0;
+  int *zero = nullptr;                 // n_zero counters that the kernels behind this one want at zero
+  int n_zero = 0;
   const float *conv = nullptr;         // [taps][ld]
   int taps = 0;
   T *tail = nullptr;                   // [rows][taps - 1][ld]
@@ -156,6 +166,8 @@ row_update_kernel(RowArgs<T> a) {
     }
   }
   if (a.early) { ugb_pdl_wait(); ugb_pdl_trigger(); }
+  if (a.zero && r == 0)
+    for (int i = threadIdx.x; i < a.n_zero; i += 256) a.zero[i] = 0;
   float4 y[VPT];
   if (a.tok) {
     const int id = a.tok[(size_t)(r / a.t) * a.tok_stride + a.tok_off + r % a.t];
@@ -195,11 +207,32 @@ row_update_kernel(RowArgs<T> a) {
         for (int i = 0; i < VPT; ++i) { y[i].x += q[u][i].x; y[i].y += q[u][i].y; y[i].z += q[u][i].z; y[i].w += q[u][i].w; }
     }
   }
+  for (int k = 0; k < a.top; ++k) {
+    const int to = __ldcg(a.slot + (size_t)r * a.top + k);
+    if (to < 0) continue;
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = threadIdx.x + i * 256;
+      if (c >= nvec) continue;
+      const float4 q = __ldcs(reinterpret_cast<const float4 *>(a.routed + (size_t)to * a.ld) + c);
+      y[i].x += q.x; y[i].y += q.y; y[i].z += q.z; y[i].w += q.w;
+    }
+  }
+  if (a.bias) {
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = threadIdx.x + i * 256;
+      if (c >= nvec) continue;
+      const float4 q = __ldg(reinterpret_cast<const float4 *>(a.bias) + c);
+      y[i].x += q.x; y[i].y += q.y; y[i].z += q.z; y[i].w += q.w;
+    }
+  }
   float4 g2[VPT];
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
     const int c = threadIdx.x + i * 256;
-    g2[i] = c < nvec ? __ldg(reinterpret_cast<const float4 *>(a.gain) + c) : zero;
+    g2[i] = zero;
+    if (a.gain && c < nvec) g2[i] = __ldg(reinterpret_cast<const float4 *>(a.gain) + c);
   }
   float inv = 1.f;
   if (a.post_gain) {
@@ -234,8 +267,11 @@ row_update_kernel(RowArgs<T> a) {
   for (int i = 0; i < VPT; ++i) {
     const int c = threadIdx.x + i * 256;
     if (c < nvec) xr[c] = v[i];
+    if (a.copy && c < nvec) Act<T>::st4(a.copy + (size_t)r * a.copy_ld + 4 * c, v[i]);
+    if (a.copy2 && c < nvec) Act<T>::st4(a.copy2 + (size_t)r * a.copy_ld + 4 * c, v[i]);
     ss += sq4(v[i]);
   }
+  if (!a.gain) return;
   const float inv2 = 1.0f / sqrtf(block_sum_256(ss, sm) * a.inv_width + a.eps);
   auto fma4 = [](float4 w, float4 q, float4 &s) {
     s.x = fmaf(w.x, q.x, s.x); s.y = fmaf(w.y, q.y, s.y); s.z = fmaf(w.z, q.z, s.z); s.w = fmaf(w.w, q.w, s.w);
@@ -279,9 +315,10 @@ row_update_kernel(RowArgs<T> a) {
   }
 }
 
-// ------------------------------------------------- causal input convolution ---
-// out[b, i] = h[b, i] + sum_j w[j] h[b, i - (taps - 1) + j] over a block of t positions per sequence, rows before the
+// ------------------------------------------------------- causal convolution ---
+// c[b, i] = sum_j w[j] h[b, i - (taps - 1) + j] over a block of t positions per sequence (rows h_ld apart), rows before the
 // block from tail_in [b][taps - 1][ld]; the block's own last taps - 1 rows go to tail_out (a different buffer).
+// out[b, i] = h[b, i] + c[b, i], or with ACT silu(c[b, i] + bias).
 // One thread per 8 channels and CONV_STRIP positions; with TAPS > 0 (the tap count, when it is small) the rows of the
 // strip slide through registers, all of them requested before the first is used; TAPS = 0 takes any tap count.
 constexpr int CONV_STRIP = 8;
@@ -317,18 +354,27 @@ template <typename T> __device__ __forceinline__ void st8(T *p, const Row8<T> &r
   }
 }
 
-template <typename T, int TAPS>
+template <typename T, int TAPS, bool ACT = false>
 __global__ void __launch_bounds__(128)
-causal_conv_kernel(const T *__restrict__ h, const float *__restrict__ w, const T *__restrict__ tail_in, T *__restrict__ tail_out,
-                   T *__restrict__ out, int t, int taps_any, int ld) {
+causal_conv_kernel(const T *__restrict__ h, size_t h_ld, const float *__restrict__ w, const float *__restrict__ bias,
+                   const T *__restrict__ tail_in, T *__restrict__ tail_out, T *__restrict__ out, int t, int taps_any, int ld) {
   const int taps = TAPS > 0 ? TAPS : taps_any;
   const int c = blockIdx.y * blockDim.x + threadIdx.x, b = blockIdx.z;
   if (c >= ld >> 3) return;
-  const T *hb = h + (size_t)b * t * ld + 8 * c;
+  const T *hb = h + (size_t)b * t * h_ld + 8 * c;
   const T *ti = tail_in + (size_t)b * (taps - 1) * ld + 8 * c;
   T *to = tail_out + (size_t)b * (taps - 1) * ld + 8 * c;
   T *ob = out + (size_t)b * t * ld + 8 * c;
-  auto row = [&](int i) { return i >= 0 ? ld8<T>(hb + (size_t)i * ld) : ld8<T>(ti + (size_t)(i + taps - 1) * ld); };
+  auto row = [&](int i) { return i >= 0 ? ld8<T>(hb + (size_t)i * h_ld) : ld8<T>(ti + (size_t)(i + taps - 1) * ld); };
+  Row8<float> bv{};
+  if constexpr (ACT) bv = ld8<float>(bias + 8 * c);
+  auto finish = [&](Row8<T> &o, const Row8<T> &x) {        // x: the position itself, the convolution's last input
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      if constexpr (ACT) { const float s = o.v[e] + bv.v[e]; o.v[e] = s * sigmoid_t<sizeof(T) == 4>(s); }
+      else o.v[e] += x.v[e];
+    }
+  };
   const int i0 = blockIdx.x * CONV_STRIP, i1 = min(i0 + CONV_STRIP, t);
   if constexpr (TAPS > 0) {
     using Raw = typename RawRow8<T>::type;                 // rows wait as they are stored and are widened when used
@@ -336,7 +382,7 @@ causal_conv_kernel(const T *__restrict__ h, const float *__restrict__ w, const T
 #pragma unroll
     for (int k = 0; k < CONV_STRIP + TAPS - 1; ++k) {
       const int i = i0 - (TAPS - 1) + k;
-      if (i < i1) q[k] = *reinterpret_cast<const Raw *>(i >= 0 ? hb + (size_t)i * ld : ti + (size_t)(i + TAPS - 1) * ld);
+      if (i < i1) q[k] = *reinterpret_cast<const Raw *>(i >= 0 ? hb + (size_t)i * h_ld : ti + (size_t)(i + TAPS - 1) * ld);
     }
     Row8<float> wv[TAPS];
 #pragma unroll
@@ -351,8 +397,7 @@ causal_conv_kernel(const T *__restrict__ h, const float *__restrict__ w, const T
 #pragma unroll
         for (int e = 0; e < 8; ++e) o.v[e] = fmaf(wv[j].v[e], x.v[e], o.v[e]);
       }
-#pragma unroll
-      for (int e = 0; e < 8; ++e) o.v[e] += x.v[e];        // the last tap is the position itself
+      finish(o, x);
       st8<T>(ob + (size_t)(i0 + k) * ld, o);
     }
   } else {
@@ -364,8 +409,7 @@ causal_conv_kernel(const T *__restrict__ h, const float *__restrict__ w, const T
 #pragma unroll
         for (int e = 0; e < 8; ++e) o.v[e] = fmaf(wv.v[e], own.v[e], o.v[e]);
       }
-#pragma unroll
-      for (int e = 0; e < 8; ++e) o.v[e] += own.v[e];
+      finish(o, own);
       st8<T>(ob + (size_t)i * ld, o);
     }
   }
@@ -652,6 +696,18 @@ static __global__ void relu2_kernel(float *__restrict__ x, size_t n4) {
     v.x = fmaxf(v.x, 0.f); v.y = fmaxf(v.y, 0.f); v.z = fmaxf(v.z, 0.f); v.w = fmaxf(v.w, 0.f);
     reinterpret_cast<float4 *>(x)[i] = make_float4(v.x * v.x, v.y * v.y, v.z * v.z, v.w * v.w);
   }
+}
+
+// ---------------------------------------------------------------- loading ----
+// gain[i] = offset + w[i], zero behind n
+static __global__ void gain_kernel(const float *__restrict__ w, float *__restrict__ gain, int n, float offset) {
+  const int i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i < n) gain[i] = offset + w[i];
+}
+// conv weights [width][taps] -> [taps][ld]
+static __global__ void taps_kernel(const float *__restrict__ w, float *__restrict__ out, int width, int taps, int ld) {
+  const int i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i < width * taps) out[(size_t)(i % taps) * ld + i / taps] = w[i];
 }
 
 }  // namespace ugb_hybrid_k

@@ -360,6 +360,51 @@ int32_t launch_simt(ugb_device *dev, void *dst, const void *lhs, const void *rhs
 
 }  // namespace
 
+namespace {
+// 64 x 64 tiles of grouped rows: rows [i tile_m, (i + 1) tile_m) multiply weights groups[i] (< 0: nothing to do).
+__global__ void __launch_bounds__(256)
+f32_grouped_kernel(float *__restrict__ c, const float *__restrict__ a, const float *__restrict__ b, const int *__restrict__ groups, int tile_m, int n, int k) {
+  __shared__ float as[16][64 + 4], bs[16][64 + 4];
+  const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64, g = groups[m0 / tile_m];
+  if (g < 0) return;
+  const float *ga = a + (size_t)m0 * k, *gb = b + (size_t)g * n * k;
+  const int lr = threadIdx.x >> 2, lk = (threadIdx.x & 3) * 4, tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  float acc[4][4] = {};
+  for (int k0 = 0; k0 < k; k0 += 16) {
+    float4 va = make_float4(0.f, 0.f, 0.f, 0.f), vb = va;
+    if (k0 + lk < k) {                                       // k % 4 == 0
+      va = *reinterpret_cast<const float4 *>(ga + (size_t)lr * k + k0 + lk);
+      if (n0 + lr < n) vb = *reinterpret_cast<const float4 *>(gb + (size_t)(n0 + lr) * k + k0 + lk);
+    }
+    __syncthreads();
+    as[lk][lr] = va.x; as[lk + 1][lr] = va.y; as[lk + 2][lr] = va.z; as[lk + 3][lr] = va.w;
+    bs[lk][lr] = vb.x; bs[lk + 1][lr] = vb.y; bs[lk + 2][lr] = vb.z; bs[lk + 3][lr] = vb.w;
+    __syncthreads();
+#pragma unroll
+    for (int kk = 0; kk < 16; ++kk) {
+      const float4 x = *reinterpret_cast<const float4 *>(&as[kk][4 * ty]), y = *reinterpret_cast<const float4 *>(&bs[kk][4 * tx]);
+      const float xv[4] = {x.x, x.y, x.z, x.w}, yv[4] = {y.x, y.y, y.z, y.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(xv[i], yv[j], acc[i][j]);
+    }
+  }
+  if (n0 + 4 * tx >= n) return;                              // n % 4 == 0
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+    *reinterpret_cast<float4 *>(c + (size_t)(m0 + 4 * ty + i) * n + n0 + 4 * tx) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+}
+}  // namespace
+
+int32_t ugb_f32_grouped_gemm(ugb_device *dev, float *c, const float *a, const float *b, const int *groups, size_t m, int tile_m, int n, int k) {
+  if (m == 0 || n == 0) return UGB_OK;
+  UGB_REQUIRE(dev, tile_m % 64 == 0 && m % tile_m == 0 && m / 64 <= 65535 && n % 4 == 0 && k % 4 == 0, UGB_ERR_UNSUPPORTED,
+              "f32 grouped product: %zu rows in tiles of %d, n %d, k %d", m, tile_m, n, k);
+  f32_grouped_kernel<<<dim3((unsigned)((n + 63) / 64), (unsigned)(m / 64)), 256, 0, dev->stream>>>(c, a, b, groups, tile_m, n, k);
+  return ugb_after_launch(dev, "f32_grouped_kernel");
+}
+
 int32_t ugb_f32_gemm(ugb_device *dev, float *c, const float *a, const float *b, size_t batch, size_t m, size_t n, size_t k,
                      size_t a_ld, size_t a_batch, bool b_is_nk, size_t b_batch, size_t c_ld, size_t c_batch) {
   if (batch == 0 || m == 0 || n == 0) return UGB_OK;

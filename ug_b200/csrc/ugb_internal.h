@@ -79,6 +79,10 @@ static inline cudaError_t ugb_malloc_async(ugb_device *dev, void **p, size_t byt
 int32_t ugb_f32_gemm(ugb_device *dev, float *c, const float *a, const float *b, size_t batch, size_t m, size_t n, size_t k,
                      size_t a_ld, size_t a_batch, bool b_is_nk, size_t b_batch, size_t c_ld, size_t c_batch);
 
+// c[m, n] = a[m, k] . w with rows grouped by the weights they multiply: rows of tile i (tile_m of them, a multiple of 64) take
+// the n rows of w [.., k] from groups[i] * n on; groups (device memory) < 0: rows without work.
+int32_t ugb_f32_grouped_gemm(ugb_device *dev, float *c, const float *a, const float *w, const int *groups, size_t m, int tile_m, int n, int k);
+
 // Records a formatted message on the device handle and returns `code`.
 int32_t ugb_fail(ugb_device *dev, int32_t code, const char *fmt, ...);
 // Checks the launch error of the kernel just enqueued and counts it.

@@ -19,9 +19,14 @@ def _kabidra(config, st, dev, batch, t_max, dtype):
     return kabidra.Model.from_safetensors(kabidra.Config.from_dict(config), st, dev, batch, t_max, dtype)
 
 
+def _zidevik(config, st, dev, batch, t_max, dtype):
+    from . import zidevik
+    return zidevik.Model.from_safetensors(zidevik.Config.from_dict(config), st, dev, batch, t_max, dtype)
+
+
 # architecture name -> loader; precisions each can run in
-ARCHITECTURES = {"Llama": _llama, "Kabidra": _kabidra}
-DTYPES = {"Llama": (DType.BF16,), "Kabidra": (DType.BF16, DType.F32)}
+ARCHITECTURES = {"Llama": _llama, "Kabidra": _kabidra, "Zidevik": _zidevik}
+DTYPES = {"Llama": (DType.BF16,), "Kabidra": (DType.BF16, DType.F32), "Zidevik": (DType.BF16, DType.F32)}
 
 
 def architecture(config):
