@@ -1,10 +1,7 @@
 """Small Kabidra configurations, random weights and comparisons shared by the Kabidra tests."""
 import functools
-import json
-import struct
 
-import numpy as np
-
+from hybrid_cases import agree, logit_err, position_err, write_model  # noqa: F401 (used by the tests)
 from oracle import kabidra_ref as K
 from ug_b200 import synth
 from ug_b200.kabidra_config import LATENT, MINGRU, Config, Layer
@@ -54,40 +51,3 @@ def oracle_logits(name, tokens, seed=300):
 
 def tokens(name, seed, n, batch=1):
     return synth.tokens(seed, (batch, n), CONFIGS[name].vocab)
-
-
-def position_err(got, want):
-    """Per position: rms(difference without its mean) / rms(all oracle logits without their mean)."""
-    d = np.asarray(got, np.float64) - want
-    d -= d.mean(axis=-1, keepdims=True)
-    w = want - want.mean(axis=-1, keepdims=True)
-    return np.sqrt(np.mean(d * d, axis=-1)) / np.sqrt(np.mean(w * w))
-
-
-def logit_err(got, want):
-    return float(np.max(position_err(got, want)))
-
-
-# Largest error of a position, and of the average over the positions compared.  bf16 rounding is amplified most where
-# two keys or the two sides of a branch are close, hence the distance between the two limits.
-LIMITS = {"f32": (2e-5, 1e-5), "bf16": (6e-2, 2.5e-2)}
-
-
-def agree(got, want, f32, slack=1.0):
-    e = position_err(got, want)
-    most, mean = LIMITS["f32" if f32 else "bf16"]
-    assert np.max(e) < slack * most and np.mean(e) < slack * mean, (float(np.max(e)), float(np.mean(e)), int(np.argmax(e)))
-    return True
-
-
-def write_model(folder, cfg, w):
-    """config.json and model.safetensors (uint16 arrays as BF16)."""
-    (folder / "config.json").write_text(json.dumps(cfg.to_dict()))
-    header, blobs, at = {}, [], 0
-    for name, a in w.items():
-        raw = np.ascontiguousarray(a).tobytes()
-        header[name] = {"dtype": "BF16", "shape": list(a.shape), "data_offsets": [at, at + len(raw)]}
-        blobs.append(raw)
-        at += len(raw)
-    h = json.dumps(header).encode()
-    (folder / "model.safetensors").write_bytes(struct.pack("<Q", len(h)) + h + b"".join(blobs))

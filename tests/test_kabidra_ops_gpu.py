@@ -2,43 +2,11 @@
 import numpy as np
 import pytest
 
+from hybrid_cases import Buf, close
 from oracle import kabidra_ref as K
-from ug_b200 import DType, UgError, synth
+from ug_b200 import UgError, synth
 
 pytestmark = pytest.mark.gpu
-
-
-class Buf:
-    """Host arrays in the activation type of a test: f32, or f32 values that bf16 holds exactly."""
-
-    def __init__(self, dev, bf16):
-        self.dev, self.bf16 = dev, bf16
-
-    def act(self, x):
-        """(device slice, the values it holds as float64)"""
-        x = np.ascontiguousarray(x, np.float32)
-        if not self.bf16:
-            return self.dev.slice_from_values(x.ravel()), x.astype(np.float64)
-        bits = synth.to_bf16_bits(x)
-        return self.dev.slice_from_values(bits.ravel(), bf16=True), synth.bf16_bits_to_f32(bits).astype(np.float64)
-
-    def f32(self, x):
-        return self.dev.slice_from_values(np.ascontiguousarray(x, np.float32).ravel())
-
-    def out(self, n):
-        return self.dev.allocate_uninit(DType.BF16 if self.bf16 else DType.F32, n)
-
-    def read(self, s, shape):
-        v = s.to_vec()
-        return (synth.bf16_bits_to_f32(v) if v.dtype == np.uint16 else v).reshape(shape).astype(np.float64)
-
-    @property
-    def tol(self):
-        return 8e-3 if self.bf16 else 2e-5
-
-
-def close(got, want, tol):
-    return float(np.max(np.abs(got - want)) / max(np.max(np.abs(want)), 1e-30)) < tol
 
 
 @pytest.mark.parametrize("bf16", [False, True])

@@ -300,3 +300,32 @@ class Device:
         """x += norm(y) post_gain; with a bank of n earlier results, x becomes their weighted sum; h = norm(x) gain."""
         self._check(lib.ugb_residual_update(self._h, x._h, y._h, post_gain._h, bank._h if bank else None,
                                             dwa._h if dwa else None, n, gain._h, h._h, rows, width, eps))
+
+    def gated_conv(self, h, w, bias, tail, out, b, t, width, taps):
+        """silu(bias + depthwise causal convolution over time); ``tail`` (the rows before the block) is moved on."""
+        self._check(lib.ugb_gated_conv(self._h, h._h, w._h, bias._h, tail._h, out._h, b, t, width, taps))
+
+    def head_inputs(self, pre, cos, sin, pos, q, kcache, vcache, b, t, heads, kv_heads, dim, vdim, rot_dims, interleaved, qk_norm, eps, t_max):
+        """Rotary positions and norm of query and key heads, append of keys and values to their caches."""
+        self._check(lib.ugb_head_inputs(self._h, pre._h, cos._h, sin._h, pos._h, q._h, kcache._h, vcache._h, b, t, heads, kv_heads, dim,
+                                        vdim, rot_dims, int(interleaved), int(qk_norm), eps, t_max))
+
+    def grouped_attend(self, q, k, v, pos, out, b, t, heads, kv_heads, dq, dv, t_max, scale, out_scale=1.0, n_slices=1):
+        """Grouped-query attention of single positions over caches of keys and values."""
+        self._check(lib.ugb_grouped_attend(self._h, q._h, k._h, v._h, pos._h, out._h, b, t, heads, kv_heads, dq, dv, t_max, scale,
+                                           out_scale, n_slices))
+
+    def grouped_attend_block(self, q, k, v, out, b, t, pos0, heads, kv_heads, dq, dv, t_max, scale, out_scale=1.0):
+        """The same for a block of positions on the tcgen05 kernel (bf16, heads of 64 or 128)."""
+        self._check(lib.ugb_grouped_attend_block(self._h, q._h, k._h, v._h, out._h, b, t, pos0, heads, kv_heads, dq, dv, t_max, scale,
+                                                 out_scale))
+
+    def selective_scan(self, x, dt, bc, z, a_log, skip, dt_bias, state, out, b, t, channels, states, scale=1.0):
+        """Selective scan over a block; ``state`` is moved on."""
+        self._check(lib.ugb_selective_scan(self._h, x._h, dt._h, bc._h, z._h, a_log._h, skip._h, dt_bias._h, state._h, out._h, b, t,
+                                           channels, states, scale))
+
+    def selective_step(self, x, low_bc, w_dt, z, a_log, skip, dt_bias, state, out, rows, channels, rank, states, scale=1.0):
+        """One position of the selective scan for every row, step-size projection included."""
+        self._check(lib.ugb_selective_step(self._h, x._h, low_bc._h, w_dt._h, z._h, a_log._h, skip._h, dt_bias._h, state._h, out._h,
+                                           rows, channels, rank, states, scale))

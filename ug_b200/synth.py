@@ -110,6 +110,38 @@ def kabidra_weights(cfg, seed_base=300):
         return dict(ex.map(one, enumerate(weight_shapes(cfg).items())))
 
 
+def zidevik_tensor(seed, name, shape):
+    """One random tensor of a Zidevik model as bf16 bit patterns.  Matrices ~ N(0, 1 / columns); gains, biases and
+    convolution taps are spread widely enough that a model without them computes something else; the channels of the scan
+    forget over a few to some hundreds of positions."""
+    tail = name.split(".", 1)[-1]
+    x = normal(seed, shape)
+    if tail in ("norm1", "norm", "side.norm", "mix.right.D"):
+        x = np.float32(1.0) + np.float32(0.2) * x
+    elif tail == "mix.right.conv":
+        x = np.float32(0.5) * x
+    elif tail in ("mix.right.conv.b", "step"):
+        x = np.float32(0.3) * x
+    elif tail == "mix.right.dt.b":
+        x = np.float32(0.5) * x - np.float32(1.5)
+    elif tail == "mix.right.A_log":
+        x = np.float32(1.5) * x - np.float32(2.0)
+    elif tail == "mlp.router":
+        x = x * np.float32(2 * shape[1] ** -0.5)
+    elif name == "loop.in":                # most of the stream goes on into the next pass
+        x = x * np.float32(0.6 * shape[1] ** -0.5)
+        x[:, :shape[0]] += np.float32(0.8) * np.eye(shape[0], dtype=np.float32)
+    elif len(shape) == 2 and tail != "embed" and name != "embed":
+        x = x * np.float32(shape[1] ** -0.5)
+    return to_bf16_bits(x)
+
+
+def zidevik_weights(cfg, seed_base=500):
+    """All tensors of a Zidevik model, name -> uint16 array; seed = seed_base + index of the tensor in load order."""
+    from .zidevik_config import weight_shapes
+    return {name: zidevik_tensor(seed_base + i, name, shape) for i, (name, shape) in enumerate(weight_shapes(cfg).items())}
+
+
 def llama_weights_f32(weights):
     """The f32 view of bf16 weights that load_with_cast BF16 -> F32 produces (any model's)."""
     return {k: (bf16_bits_to_f32(v) if v.dtype == np.uint16 else v) for k, v in weights.items()}
