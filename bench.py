@@ -1202,12 +1202,173 @@ class KabidraWorkload:
         return {"workload": self.name}
 
 
+class ZidevikWorkload(KabidraWorkload):
+    """The Zidevik decoder at the layer sizes of the 1.1B Llama benchmark model, beside Kabidra and Llama at those sizes: the
+    decode steps, prompts and single kernels of KabidraWorkload for all three in one process."""
+    metric = "tokens/s, Zidevik decode (64 sequences, 2048 cached positions)"
+    name = ("Zidevik, width 2048, 22 layers of which 6 run twice (attention with 32 heads of 64 on 4 beside a scan of 4096 channels "
+            "with 16 states; feed-forwards alternately dense with 5632 columns and 2 of 16 experts of 1408 beside a shared one of "
+            "2816; token input of 256), vocab 32000, bf16; beside Kabidra and the Llama-1.1B shape")
+    SFU_PER_CLOCK = 16           # special functions per clock and SM
+
+    def __init__(self, rank=0):
+        from ug_b200.zidevik_config import Config
+        self.cfg = Config.like_llama_1b()
+
+    def setup(self, dev):
+        import re
+        from concurrent.futures import ThreadPoolExecutor
+
+        from ug_b200 import synth
+        from ug_b200.zidevik_config import weight_shapes
+        shapes = weight_shapes(self.cfg)
+        kind = lambda n: (re.sub(r"\.e\d+\.", ".e.", re.sub(r"^l\d+\.", "l.", n)), shapes[n])   # one set per kind of tensor and shape
+        first = {}
+        for n in shapes:
+            first.setdefault(kind(n), n)
+        with ThreadPoolExecutor(max_workers=min(16, os.cpu_count() or 1)) as ex:
+            made = dict(zip(first, ex.map(lambda n: synth.zidevik_tensor(500, n, shapes[n]), first.values())))
+        self.weights = {n: made[kind(n)] for n in shapes}
+        self.other = KabidraWorkload()
+        self.other.setup(dev)
+        self.sms = 148
+
+    def splits(self, n, k, decode, batch):
+        """k splits of a step's product, as the engine chooses them."""
+        if not decode or batch > 64:
+            return 1
+        kb = (k + 63) // 64
+        best, fewest = 1, kb + 1
+        for s in range(1, min(8, kb) + 1):
+            for bn in (64, 80, 96, 128, 160):
+                per = (kb + s - 1) // s
+                if (n + bn - 1) // bn * s <= self.sms and per < fewest:
+                    best, fewest = s, per
+        per = (kb + best - 1) // best
+        return (kb + per - 1) // per
+
+    def work(self, rows, batch, t, depth):
+        """Per kind of kernel: (launches, bytes moved at least once, flops) of one pass over all layer runs."""
+        from ug_b200.zidevik_config import Experts
+        c, decode, w, s = self.cfg, t == 1, self.cfg.width, self.cfg.side_dim
+        runs = list(range(c.loop.start)) + list(range(c.loop.start, c.loop.stop)) * c.loop.times + list(range(c.loop.stop, len(c.layers)))
+        out = {}
+
+        def add(name, launches, nbytes, flops=0):
+            o = out.get(name, (0, 0, 0))
+            out[name] = (o[0] + launches, o[1] + nbytes, o[2] + flops)
+        pn = lambda n, k: self.splits(n, k, decode, batch)
+        act = lambda n, k: 4 * pn(n, k) if decode else 2                  # bytes per value of a projection that feeds row kernels
+        mm = lambda name, n, k, per: add(name, 1, 2 * n * k + rows * (2 * k + per * n), 2 * rows * n * k)
+        res = lambda n, k: 4 * pn(n, k)                                    # f32 products of the residual stream
+        for i in runs:
+            l = c.layers[i]
+            a, r, x = l.left, l.right, isinstance(l.mlp, Experts)
+            heads, E, N = a.heads * a.dim + a.kv_heads * (a.dim + a.vdim), l.mlp.count if x else 0, r.state
+            ff, low, cat = (l.mlp.shared if x else l.mlp) or 0, r.dt_rank + 2 * r.state, 0
+            cat = a.heads * a.vdim + r.inner + ff
+            n_in = heads + 2 * r.inner + (E if decode else 0)
+            mm("mix_in", n_in, w, act(n_in, w))
+            if decode:
+                add("mix_rows", 1, rows * (act(n_in, w) * (heads + r.inner + E) + 2 * heads + r.inner * (2 + 4 * (r.conv - 1))))
+                mm("scan_in", low, r.inner, act(low, r.inner))
+                add("scan", 1, rows * r.inner * (8 * N + act(n_in, w) + 4) + rows * low * act(low, r.inner) + 2 * r.dt_rank * r.inner)
+                add("attention", 1, batch * depth * a.kv_heads * (a.dim + a.vdim) * 2, batch * depth * a.heads * 2 * (a.dim + a.vdim))
+            else:
+                add("mix_rows", 1, rows * 4 * heads)
+                add("conv", 1, rows * r.inner * 4)
+                mm("scan_in", low, r.inner, 2)
+                mm("scan_in", r.inner, r.dt_rank, 2)
+                add("scan", 1, rows * (8 * r.inner + 4 * N))
+                pairs = batch * (depth * t + t * (t + 1) // 2)
+                add("attention", 1, rows * (a.heads + a.kv_heads) * (a.dim + a.vdim) * 2, pairs * a.heads * 2 * (a.dim + a.vdim))
+            if ff:
+                add("up", 1, 4 * ff * w + rows * (2 * w + 2 * ff), 4 * rows * ff * w)
+            if x:
+                n = rows * l.mlp.top
+                used = min(E, n)
+                add("route", 1 if decode else 3, rows * 2 * w + n * 2 * w + (0 if decode else 2 * E * w + rows * (2 * w + 8 * E)), 0 if decode else 2 * rows * E * w)
+                add("expert_up", 1, used * 4 * l.mlp.ff * w + n * (2 * w + 2 * l.mlp.ff), 4 * n * l.mlp.ff * w)
+                add("expert_down", 1, used * 2 * l.mlp.ff * w + n * (2 * l.mlp.ff + 4 * w), 2 * n * l.mlp.ff * w)
+            mm("out", w, cat, res(w, cat))
+            add("rows", 1, rows * w * (res(w, cat) + 8 + 2 + (4 * l.mlp.top if x else 0)))
+            mm("side", s, w, res(s, w))
+            mm("side", w, s, res(w, s))
+            add("side_gate", 1, rows * s * (res(s, w) + 4))
+            add("rows", 1, rows * w * (res(w, s) + 8 + 2))
+        for _ in range(c.loop.times):
+            mm("loop", w, 2 * w, res(w, 2 * w))
+            add("rows", 1, rows * w * (res(w, 2 * w) + 4 + 2))
+        add("rows", 1, rows * w * (2 + 4 + 2 + 2))
+        return out
+
+    def kernels(self, model, rows, batch, t, depth, peaks):
+        out = super().kernels(model, rows, batch, t, depth, peaks)
+        if t > 1:                                                           # the scan's other limit: one power per state and position
+            c = self.cfg
+            n = sum(c.layers[i].right.inner * c.layers[i].right.state for i in range(len(c.layers))) * rows
+            n += (c.loop.times - 1) * sum(c.layers[i].right.inner * c.layers[i].right.state for i in range(c.loop.start, c.loop.stop)) * rows
+            out["scan"]["frac_of_special_functions"] = round(1e3 * n / (self.SFU_PER_CLOCK * self.sms * 1.965e9) / out["scan"]["ms"], 3)
+        return out
+
+    def record(self, dev, warmup, steps, peaks):
+        from ug_b200 import kabidra, llama, synth, zidevik
+        from ug_b200.llama_config import Config as LlamaConfig
+        lc = LlamaConfig.llama_1b()
+        lw = _weights(lc)
+        made = {"zidevik": (self, lambda b, t: zidevik.Model.new(self.cfg, self.weights, dev, b, t)),
+                "kabidra": (self.other, lambda b, t: kabidra.Model.new(self.other.cfg, self.other.weights, dev, b, t)),
+                "llama": (None, lambda b, t: llama.Model.new(lc, lw, dev, b, t))}
+        sampler = ClockSampler(0)
+        sampler.start()
+        rec = {"workload": self.name, "metric": self.metric, "unit": self.unit, "dtype": self.dtype, "steps": steps,
+               "data": "synthetic (random weights and tokens)", "peak_source": peaks["source"], "decode": {}, "prefill": {}}
+        for batch, depth in self.DECODE:
+            prompts, r = synth.tokens(8, (batch, depth), self.cfg.vocab), {}
+            for key, (wl, make) in made.items():
+                m = make(batch, depth + warmup + steps + 64)
+                m.prefill(prompts)
+                ms = self.timed(dev, lambda: m.decode(1), max(warmup, 3), steps)
+                r[key] = {"tokens_per_s": round(1e3 * batch / ms, 1), "ms_per_step": round(ms, 4)}
+                at = m.position
+                if wl:
+                    r[key]["state_bytes_per_sequence"] = m.state_bytes(at)
+                    r[key]["kernels"] = wl.kernels(m, batch, batch, 1, at, peaks)
+                    r[key]["kernels"]["head"] = {"ms": round(m.time_kernel("head"), 4), "launches": 1}
+                else:
+                    kv = 2 * lc.num_hidden_layers * 2 * lc.num_key_value_heads * lc.head_dim() * at * batch
+                    r[key]["attention_frac"] = round(kv / peaks["hbm"] / 1e6 / m.time_kernel("decode_attention", 20), 3)
+                m.close()
+            rec["decode"]["%d x %d" % (batch, depth)] = r
+        for batch, t in self.PREFILL:
+            prompts, r = dev.slice_from_values(synth.tokens(9, (batch, t), self.cfg.vocab).reshape(-1)), {}
+            for key, (wl, make) in made.items():
+                m = make(batch, t + (32 if wl else 0))
+
+                def step():
+                    m.reset()
+                    m.prefill(prompts)
+                ms = self.timed(dev, step, max(warmup, 3), max(3, steps // 5))
+                r[key] = {"tokens_per_s": round(1e3 * batch * t / ms, 1), "ms_per_step": round(ms, 4)}
+                if wl:
+                    m.reset()
+                    m.decode(1)
+                    step()                       # the kernels timed alone find a prompt's routing and activations
+                    m.reset()
+                    r[key]["kernels"] = wl.kernels(m, batch * t, batch, t, 0, peaks)
+                m.close()
+            rec["prefill"]["%d x %d" % (batch, t)] = r
+        rec["clocks"] = sampler.stop()
+        rec["value"] = rec["decode"]["64 x 2048"]["zidevik"]["tokens_per_s"]
+        return rec
+
+
 WORKLOADS = {"rms_silu": RmsSiluWorkload, "softmax": SoftmaxWorkload, "softmax_c1": SoftmaxC1Workload,
              "gemm": GemmWorkload, "decode": DecodeWorkload, "prefill": PrefillWorkload,
              "graph_softmax": lambda r: GraphRowWorkload("softmax"), "graph_rms_norm": lambda r: GraphRowWorkload("rms_norm"),
              "gemm_f32": lambda r: F32MatmulWorkload("gemm_f32"), "gemv_f32": lambda r: F32MatmulWorkload("gemv_f32"),
              "graph_decode": GraphDecodeWorkload, "llama_ops": LlamaOpsWorkload,
-             "kabidra": KabidraWorkload}
+             "kabidra": KabidraWorkload, "zidevik": ZidevikWorkload}
 DEFAULT_WORKLOAD = "decode"
 
 # DRAM traffic of the decode step's kernels, from ncu captures of single launches (dram__bytes_read.sum +

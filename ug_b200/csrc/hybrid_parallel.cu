@@ -57,9 +57,10 @@ int32_t launch_gated_conv(ugb_device *dev, const T *h, size_t h_ld, const float 
 
 template <typename TI, typename T, bool STEP>
 int32_t launch_mixer_inputs(ugb_device *dev, const MixerIn<TI, T> &a, int rows, bool pdl) {
-  int units = a.heads + a.kv_heads + (a.kv_heads * a.vp + 127) / 128;
-  if (STEP) units += (a.ci + 127) / 128 + (a.experts > 0 ? 1 : 0);
-  const cudaError_t e = ugb_launch(mixer_inputs_kernel<TI, T, STEP>, dim3(rows, (units + 7) / 8), dim3(256), 0, dev->stream, pdl, a);
+  const MixerUnits n = mixer_units<STEP>(a.heads + a.kv_heads, a.dp, a.kv_heads * a.vp, a.ci, a.experts);
+  const long long warps = (long long)rows * n.all;
+  UGB_REQUIRE(dev, warps < (1ll << 31), UGB_ERR_UNSUPPORTED, "mixer inputs: %d rows of %d units", rows, n.all);
+  const cudaError_t e = ugb_launch(mixer_inputs_kernel<TI, T, STEP>, dim3((unsigned)((warps + 7) / 8)), dim3(256), 0, dev->stream, pdl, a, rows);
   if (e != cudaSuccess) return ugb_fail(dev, UGB_ERR_CUDA, "launch of mixer_inputs_kernel failed: %s", cudaGetErrorString(e));
   return ugb_after_launch(dev, "mixer_inputs_kernel");
 }
@@ -86,6 +87,7 @@ int32_t run(ugb_hybrid *m, ugb_hybrid_work &w, const int *tok, int t_block, int 
   // to its predecessor's predecessor is complete (see row_update_kernel).
   const bool early = decode && pdl && !m->f32;
   const int B = m->batch, rows = B * t, wl = m->wl, n_runs = (int)m->runs.size();
+  const bool whole = m->only == UGB_HYBRID_K_ALL;            // kernels timed alone leave the counts of the last whole pass as they are
   const bool looped = m->cfg.loop_times > 0, side = m->cfg.side_dim > 0;
   int32_t rc;
   cudaError_t e;
@@ -99,7 +101,7 @@ int32_t run(ugb_hybrid *m, ugb_hybrid_work &w, const int *tok, int t_block, int 
     }
     a.h = (T *)w.h;
     a.gain = i < n_runs ? m->layers[m->runs[i].layer].norm1 : m->final_gain;
-    if (i < n_runs && m->layers[m->runs[i].layer].d.feed_forward == UGB_FF_EXPERTS) { a.zero = w.count; a.n_zero = m->layers[m->runs[i].layer].d.experts; }
+    if (whole && i < n_runs && m->layers[m->runs[i].layer].d.feed_forward == UGB_FF_EXPERTS) { a.zero = w.count; a.n_zero = m->layers[m->runs[i].layer].d.experts; }
   };
   {
     RowArgs<T> a;
@@ -125,7 +127,7 @@ int32_t run(ugb_hybrid *m, ugb_hybrid_work &w, const int *tok, int t_block, int 
       a.part = w.prod; a.n_part = ti.splits; a.part_stride = (size_t)rows * wl;
       a.bias = m->loop_step + (size_t)R.enter * wl;
       a.x = w.x; a.add_x = 0; a.h = (T *)w.h; a.gain = L.norm1;
-      if (experts) { a.zero = w.count; a.n_zero = d.experts; }
+      if (experts && whole) { a.zero = w.count; a.n_zero = d.experts; }
       if ((rc = ugb_hybrid_rows<T>(m, a, rows, early))) return rc;
     }
 
@@ -152,7 +154,7 @@ int32_t run(ugb_hybrid *m, ugb_hybrid_work &w, const int *tok, int t_block, int 
         heads(a);
         a.pre = w.pre; a.n_part = in_t.splits; a.part_stride = pre_part;
         a.conv_w = L.conv_w; a.conv_b = L.conv_b; a.taps = d.conv; a.ci = L.ci; a.tail = tail; a.u = (T *)w.hc;
-        if (experts) { a.experts = d.experts; a.top = d.top; a.choice = w.choice; a.count = w.count; }
+        if (experts && whole) { a.experts = d.experts; a.top = d.top; a.choice = w.choice; a.count = w.count; }
         if ((rc = launch_mixer_inputs<float, T, true>(dev, a, rows, pdl))) return rc;
       }
     } else {
@@ -225,6 +227,7 @@ int32_t run(ugb_hybrid *m, ugb_hybrid_work &w, const int *tok, int t_block, int 
           const size_t es = m->es();
           Mat g{w.router, w.h, (const char *)L.w_in + n_in * wl * es, (size_t)rows, (size_t)L.ep, (size_t)wl};
           if ((rc = ugb_hybrid_matmul(m, g))) return rc;
+          if (!whole) UGB_CUDA(dev, cudaMemsetAsync(w.count, 0, d.experts * sizeof(int), dev->stream));
           route_kernel<<<(rows + ROUTE_ROWS - 1) / ROUTE_ROWS, 256, 0, dev->stream>>>(w.router, L.ep, rows, d.experts, d.top, w.choice, w.count);
           if ((rc = ugb_after_launch(dev, "route_kernel"))) return rc;
         }
@@ -264,8 +267,8 @@ int32_t run(ugb_hybrid *m, ugb_hybrid_work &w, const int *tok, int t_block, int 
         if ((rc = ugb_hybrid_matmul(m, g))) return rc;
       }
       if (m->on(UGB_HYBRID_K_SIDE_GATE)) {
-        e = ugb_launch(token_gate_kernel<T>, dim3(rows, (m->sl + 127) / 128), dim3(128), 0, dev->stream, pdl, w.side, g_t.splits, (size_t)rows * m->sl, m->sl,
-                       m->cfg.side_dim, tok, t, t_block, off, (const T *)m->side_embed, (size_t)m->cfg.layers * m->cfg.side_dim,
+        e = ugb_launch(token_gate_kernel<T>, dim3((unsigned)(((size_t)rows * m->sl / 4 + 255) / 256)), dim3(256), 0, dev->stream, pdl, w.side, g_t.splits,
+                       (size_t)rows * m->sl, (size_t)rows * m->sl / 4, m->sl, m->cfg.side_dim, tok, t, t_block, off, (const T *)m->side_embed, (size_t)m->cfg.layers * m->cfg.side_dim,
                        R.layer * m->cfg.side_dim, m->cfg.vocab, (T *)w.side_h);
         if (e != cudaSuccess) return ugb_fail(dev, UGB_ERR_CUDA, "launch of token_gate_kernel failed: %s", cudaGetErrorString(e));
         if ((rc = ugb_after_launch(dev, "token_gate_kernel"))) return rc;
@@ -308,7 +311,7 @@ int32_t ugb_parallel_layer(ugb_hybrid *m, int i) {
   UGB_REQUIRE(dev, d.mixer == UGB_MIXER_ATTENTION_SCAN, UGB_ERR_UNSUPPORTED, "layer %d: mixer kind %d in the parallel form", i, d.mixer);
   UGB_REQUIRE(dev, d.heads > 0 && d.kv_heads > 0 && d.heads % d.kv_heads == 0 && d.dim > 0 && d.vdim > 0, UGB_ERR_INVALID,
               "layer %d: %d heads on %d, %d- and %d-wide", i, d.heads, d.kv_heads, d.dim, d.vdim);
-  UGB_REQUIRE(dev, d.dim <= 64 * HEAD_PAIRS && d.vdim <= 512, UGB_ERR_UNSUPPORTED, "layer %d: heads of %d and %d values", i, d.dim, d.vdim);
+  UGB_REQUIRE(dev, d.dim <= HEAD_DIM_MAX && d.vdim <= 512, UGB_ERR_UNSUPPORTED, "layer %d: heads of %d and %d values", i, d.dim, d.vdim);
   UGB_REQUIRE(dev, d.rot_dims >= 0 && d.rot_dims <= d.dim && d.rot_dims % 2 == 0, UGB_ERR_INVALID, "layer %d: %d rotated dimensions of %d", i, d.rot_dims, d.dim);
   UGB_REQUIRE(dev, d.inner > 0 && d.state > 0 && d.conv > 0 && d.conv <= 64 && d.dt_rank > 0, UGB_ERR_INVALID,
               "layer %d: scan of %d channels, %d states, %d taps, rank %d", i, d.inner, d.state, d.conv, d.dt_rank);
@@ -575,7 +578,7 @@ int32_t ugb_head_inputs(ugb_device *dev, const ugb_slice *pre, const ugb_slice *
                         int32_t interleaved, int32_t qk_norm, float eps, size_t t_max) {
   if (!dev) return UGB_ERR_INVALID;
   if (int32_t rc = act_dtype(dev, pre, q, "head_inputs")) return rc;
-  UGB_REQUIRE(dev, dim % 8 == 0 && vdim % 8 == 0 && dim > 0 && vdim > 0 && dim <= 64 * HEAD_PAIRS && rot_dims <= dim && rot_dims % 2 == 0 && heads > 0 &&
+  UGB_REQUIRE(dev, dim % 8 == 0 && vdim % 8 == 0 && dim > 0 && vdim > 0 && dim <= HEAD_DIM_MAX && rot_dims <= dim && rot_dims % 2 == 0 && heads > 0 &&
                        kv_heads > 0 && b * t <= (1u << 30) && t_max <= (1u << 30) && heads + kv_heads * (1 + vdim) <= 65535, UGB_ERR_SHAPE, "head_inputs: unsupported shape");
   const size_t ld = (heads + kv_heads) * dim + kv_heads * vdim;
   UGB_SLICE(dev, pre, q->dtype, b * t * ld);

@@ -15,7 +15,7 @@ namespace ugb_hybrid_k {
 //   router -> choice of experts
 // Row r = (b, i) = (r / t, r % t) at position *pos_p + pos_off + i.  The projection is a sum of f32 partials in a step,
 // one T row in a block.
-constexpr int HEAD_PAIRS = 4;          // pairs of dimensions per lane: heads of up to 256
+constexpr int HEAD_DIM_MAX = 256;      // a lane takes 8 dimensions of a head
 constexpr int ROUTER_PER_LANE = 8;     // up to 256 experts
 
 template <typename TI, typename T> struct MixerIn {
@@ -63,34 +63,36 @@ __device__ __forceinline__ void top_experts(float (&z)[ROUTER_PER_LANE], int exp
   }
 }
 
+// Lanes of a warp that share a head: 8 dimensions each, rounded up to a power of two.
+__host__ __device__ __forceinline__ int head_lanes(int dp) {
+  int n = 1;
+  while (8 * n < dp) n *= 2;
+  return n;
+}
+// Warps' worth of work in a row: groups of heads, pieces of 256 values, in a step pieces of 128 scan inputs and the router.
+struct MixerUnits { int heads, v, x, all; };
+template <bool STEP> __host__ __device__ __forceinline__ MixerUnits mixer_units(int heads, int dp, int v, int ci, int experts) {
+  MixerUnits n;
+  const int per = 32 / head_lanes(dp);
+  n.heads = (heads + per - 1) / per;
+  n.v = (v + 255) / 256;
+  n.x = STEP ? (ci + 127) / 128 : 0;
+  n.all = n.heads + n.v + n.x + (STEP && experts > 0 ? 1 : 0);
+  return n;
+}
+
 template <typename TI, typename T, bool STEP>
 __global__ void __launch_bounds__(256)
-mixer_inputs_kernel(MixerIn<TI, T> a) {
-  const int r = blockIdx.x, unit = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  const int n_head = a.heads + a.kv_heads, n_v = (a.kv_heads * a.vp + 127) / 128, n_x = STEP ? (a.ci + 127) / 128 : 0;
-  const int b = r / a.t;
+mixer_inputs_kernel(MixerIn<TI, T> a, int rows) {
+  const int n_head = a.heads + a.kv_heads;
+  const MixerUnits n = mixer_units<STEP>(n_head, a.dp, a.kv_heads * a.vp, a.ci, a.experts);
+  const int id = blockIdx.x * 8 + (threadIdx.x >> 5), r = id / n.all, unit = id - r * n.all, lane = threadIdx.x & 31;
   ugb_pdl_wait();
   ugb_pdl_trigger();
+  if (r >= rows) return;
+  const int b = r / a.t;
   const TI *row = a.pre + (size_t)r * a.ld;
-  auto sum2 = [&](int c0, int c1, bool on) {               // the partials are added in order
-    float2 s = make_float2(0.f, 0.f);
-    if (!on) return s;
-    for (int p = 0; p < a.n_part; p += 4) {
-      float2 v[4];
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        v[e] = make_float2(0.f, 0.f);
-        if (p + e < a.n_part) {
-          const TI *q = row + (size_t)(p + e) * a.part_stride;
-          v[e] = make_float2((float)q[c0], (float)q[c1]);
-        }
-      }
-#pragma unroll
-      for (int e = 0; e < 4; ++e) { s.x += v[e].x; s.y += v[e].y; }
-    }
-    return s;
-  };
-  auto sum4 = [&](int c) {
+  auto sum4 = [&](int c) {                                 // the partials are added in order
     float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
     for (int p = 0; p < a.n_part; p += 4) {
       float4 v[4];
@@ -101,56 +103,90 @@ mixer_inputs_kernel(MixerIn<TI, T> a) {
     }
     return s;
   };
-  if (unit < n_head + n_v) {
+  auto sum8 = [&](int c) {
+    if constexpr (!STEP) return ld8<TI>(row + c);
+    Row8<TI> s;
+    const float4 x = sum4(c), y = sum4(c + 4);
+    s.v[0] = x.x; s.v[1] = x.y; s.v[2] = x.z; s.v[3] = x.w; s.v[4] = y.x; s.v[5] = y.y; s.v[6] = y.z; s.v[7] = y.w;
+    return s;
+  };
+  if (unit < n.heads + n.v) {
     const int pos = *a.pos_p + a.pos_off + r % a.t;
     if (pos < 0 || pos >= a.t_max) {
       if (lane == 0 && atomicCAS(&a.status->code, 0u, (unsigned)UGB_ERR_INVALID) == 0u) a.status->detail = (unsigned)pos;
       return;
     }
-    if (unit < n_head) {
-      const int half = a.rot_dims >> 1, col = unit * a.dp, pairs = a.dp >> 1;
-      float2 v[HEAD_PAIRS];
-      float ss = 0.f;
+    if (unit < n.heads) {
+      const int share = head_lanes(a.dp), head = unit * (32 / share) + lane / share, i0 = 8 * (lane % share), half = a.rot_dims >> 1;
+      const bool on = head < n_head && i0 < a.dp;          // dp is a multiple of 8
+      Row8<TI> x{};
+      if (on) x = sum8(head * a.dp + i0);
+      if (on && i0 < a.rot_dims) {
+        const float *cs = a.cos_ + (size_t)pos * half, *sn = a.sin_ + (size_t)pos * half;
+        if (a.interleaved) {
+          const int p0 = i0 >> 1;
+          float c[4], s[4];
+          if ((half & 3) == 0) {                           // four angles at once: all inside, the table's rows aligned
+            *reinterpret_cast<float4 *>(c) = __ldg(reinterpret_cast<const float4 *>(cs + p0));
+            *reinterpret_cast<float4 *>(s) = __ldg(reinterpret_cast<const float4 *>(sn + p0));
+          } else {
 #pragma unroll
-      for (int j = 0; j < HEAD_PAIRS; ++j) {
-        const int p = lane + 32 * j;
-        const bool rot = p < half;
-        const int c0 = rot && !a.interleaved ? p : 2 * p, c1 = rot && !a.interleaved ? p + half : 2 * p + 1;
-        v[j] = sum2(col + c0, col + c1, p < pairs);
-        if (rot) {
-          const float c = __ldg(a.cos_ + (size_t)pos * half + p), s = __ldg(a.sin_ + (size_t)pos * half + p);
-          v[j] = make_float2(v[j].x * c - v[j].y * s, v[j].y * c + v[j].x * s);
+            for (int e = 0; e < 4; ++e) {
+              c[e] = p0 + e < half ? __ldg(cs + p0 + e) : 1.f;
+              s[e] = p0 + e < half ? __ldg(sn + p0 + e) : 0.f;
+            }
+          }
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const float u = x.v[2 * e], v = x.v[2 * e + 1];
+            x.v[2 * e] = u * c[e] - v * s[e];
+            x.v[2 * e + 1] = v * c[e] + u * s[e];
+          }
+        } else {                                           // the partner of a dimension lies half the rotated part away
+#pragma unroll
+          for (int e = 0; e < 8; ++e) {
+            const int i = i0 + e;
+            if (i >= a.rot_dims) break;
+            const int p = i < half ? i : i - half, other = i < half ? i + half : i - half;
+            float y = 0.f;
+            for (int q = 0; q < a.n_part; ++q) y += (float)row[(size_t)q * a.part_stride + head * a.dp + other];
+            const float c = __ldg(cs + p), s = __ldg(sn + p);
+            x.v[e] = i < half ? x.v[e] * c - y * s : x.v[e] * c + y * s;
+          }
         }
-        ss += v[j].x * v[j].x + v[j].y * v[j].y;
       }
-      float inv = 1.f;
       if (a.qk_norm) {
+        float ss = 0.f;
 #pragma unroll
-        for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-        inv = 1.0f / sqrtf(ss / (float)a.dim + a.eps);
-      }
-      T *dst = unit < a.heads ? a.q + ((size_t)r * a.heads + unit) * a.dp
-                              : a.kcache + (((size_t)b * a.kv_heads + unit - a.heads) * a.t_max + pos) * a.dp;
+        for (int e = 0; e < 8; ++e) ss = fmaf(x.v[e], x.v[e], ss);
+        for (int o = share >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+        const float inv = 1.0f / sqrtf(ss / (float)a.dim + a.eps);
 #pragma unroll
-      for (int j = 0; j < HEAD_PAIRS; ++j) {
-        const int p = lane + 32 * j;
-        if (p >= pairs) continue;
-        const bool split = p < half && !a.interleaved;
-        dst[split ? p : 2 * p] = (T)(v[j].x * inv);
-        dst[split ? p + half : 2 * p + 1] = (T)(v[j].y * inv);
+        for (int e = 0; e < 8; ++e) x.v[e] *= inv;
       }
+      if (!on) return;
+      T *dst = head < a.heads ? a.q + ((size_t)r * a.heads + head) * a.dp
+                              : a.kcache + (((size_t)b * a.kv_heads + head - a.heads) * a.t_max + pos) * a.dp;
+      Row8<T> y;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) y.v[e] = x.v[e];
+      st8<T>(dst + i0, y);
     } else {
-      const int c = (unit - n_head) * 128 + 4 * lane;
+      const int c = (unit - n.heads) * 256 + 8 * lane;
       if (c >= a.kv_heads * a.vp) return;
-      const int h = c / a.vp;                              // vp is a multiple of 8: the 4 values belong to one head
-      Act<T>::st4(a.vcache + (((size_t)b * a.kv_heads + h) * a.t_max + pos) * a.vp + c - h * a.vp, sum4(n_head * a.dp + c));
+      const int h = c / a.vp;                              // vp is a multiple of 8: the 8 values belong to one head
+      const Row8<TI> x = sum8(n_head * a.dp + c);
+      Row8<T> y;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) y.v[e] = x.v[e];
+      st8<T>(a.vcache + (((size_t)b * a.kv_heads + h) * a.t_max + pos) * a.vp + c - h * a.vp, y);
     }
     return;
   }
   if constexpr (STEP) {
     const int x0 = n_head * a.dp + a.kv_heads * a.vp;
-    if (unit < n_head + n_v + n_x) {
-      const int c = (unit - n_head - n_v) * 128 + 4 * lane;
+    if (unit < n.heads + n.v + n.x) {
+      const int c = (unit - n.heads - n.v) * 128 + 4 * lane;
       if (c >= a.ci) return;
       float4 x = sum4(x0 + c), s = __ldg(reinterpret_cast<const float4 *>(a.conv_b + c));
       // what the convolution sees, now and later, is the rounded input
@@ -165,12 +201,14 @@ mixer_inputs_kernel(MixerIn<TI, T> a) {
       constexpr bool EXACT = sizeof(T) == 4;
       Act<T>::st4(a.u + (size_t)r * a.ci + c, make_float4(s.x * sigmoid_t<EXACT>(s.x), s.y * sigmoid_t<EXACT>(s.y),
                                                          s.z * sigmoid_t<EXACT>(s.z), s.w * sigmoid_t<EXACT>(s.w)));
-    } else if (unit == n_head + n_v + n_x && a.experts > 0) {
+    } else if (a.experts > 0) {
       float z[ROUTER_PER_LANE];
 #pragma unroll
       for (int j = 0; j < ROUTER_PER_LANE; ++j) {
         const int e = lane + 32 * j;
-        z[j] = e < a.experts ? sum2(x0 + 2 * a.ci + e, x0 + 2 * a.ci + e, true).x : -INFINITY;
+        z[j] = e < a.experts ? 0.f : -INFINITY;
+        if (e < a.experts)
+          for (int p = 0; p < a.n_part; ++p) z[j] += (float)row[(size_t)p * a.part_stride + x0 + 2 * a.ci + e];
       }
       top_experts(z, a.experts, a.top, [&](int k, int e, float zk) {
         if (lane == 0) a.choice[(size_t)r * a.top + k] = make_float4(__int_as_float(e), __int_as_float(atomicAdd(a.count + e, 1)), sigmoid_f(zk), 0.f);
@@ -270,28 +308,43 @@ static __global__ void silu_mul_kernel(const float *__restrict__ gu, float *__re
 
 // ------------------------------------------------------------- token input ---
 // out[r][j] = gelu_tanh(sum of the partials of row r, column j) * table[token(r)][off + j], zero behind n.
+// A thread takes 4 columns of a row; n4 = rows * ld / 4.
 template <typename T>
-__global__ void __launch_bounds__(128)
-token_gate_kernel(const float *__restrict__ part, int n_part, size_t part_stride, int ld, int n, const int *__restrict__ tok, int t,
+__global__ void __launch_bounds__(256)
+token_gate_kernel(const float *__restrict__ part, int n_part, size_t part_stride, size_t n4, int ld, int n, const int *__restrict__ tok, int t,
                   int tok_stride, int tok_off, const T *__restrict__ table, size_t table_ld, int off, int vocab, T *__restrict__ out) {
   ugb_pdl_wait();
   ugb_pdl_trigger();
-  const int r = blockIdx.x, j = blockIdx.y * blockDim.x + threadIdx.x;
-  if (j >= ld) return;
+  const size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (idx >= n4) return;
+  const int r = (int)(idx / (ld >> 2)), j = 4 * (int)(idx - (size_t)r * (ld >> 2));
   const int id = tok[(size_t)(r / t) * tok_stride + tok_off + r % t];
-  float s = 0.f, e = 0.f;
-  if (j < n && id >= 0 && id < vocab) e = (float)table[(size_t)id * table_ld + off + j];
-  for (int p = 0; p < n_part; p += 4) {
-    float v[4];
+  float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int p = 0; p < n_part; p += 4) {                    // the partials are added in order
+    float4 v[4];
 #pragma unroll
-    for (int k = 0; k < 4; ++k) v[k] = p + k < n_part ? part[(size_t)(p + k) * part_stride + (size_t)r * ld + j] : 0.f;
-    s += v[0]; s += v[1]; s += v[2]; s += v[3];
+    for (int k = 0; k < 4; ++k)
+      v[k] = p + k < n_part ? *reinterpret_cast<const float4 *>(part + (size_t)(p + k) * part_stride + (size_t)r * ld + j) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int k = 0; k < 4; ++k) { s.x += v[k].x; s.y += v[k].y; s.z += v[k].z; s.w += v[k].w; }
   }
-  const float g = 0.5f * s * (1.0f + tanhf(0.7978845608028654f * (s + 0.044715f * s * s * s)));
-  out[(size_t)r * ld + j] = (T)(g * e);
+  float e[4] = {0.f, 0.f, 0.f, 0.f};
+  if (id >= 0 && id < vocab) {
+    const T *src = table + (size_t)id * table_ld + off + j;
+    if (j + 4 <= n && ((off | n | (int)(table_ld & 3)) & 3) == 0) {
+      const float4 q = Act<T>::ld4(src);
+      e[0] = q.x; e[1] = q.y; e[2] = q.z; e[3] = q.w;
+    } else {
+#pragma unroll
+      for (int k = 0; k < 4; ++k)
+        if (j + k < n) e[k] = (float)src[k];
+    }
+  }
+  auto gelu = [](float x) { return 0.5f * x * (1.0f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x))); };
+  Act<T>::st4(out + (size_t)r * ld + j, make_float4(gelu(s.x) * e[0], gelu(s.y) * e[1], gelu(s.z) * e[2], gelu(s.w) * e[3]));
 }
 
-// ---------------------------------------------------------------- loading ----
+// ------------------------------------------------------- logits, loading ----
 static __global__ void softcap_kernel(float *__restrict__ x, size_t n4, float cap) {
   ugb_pdl_wait();
   ugb_pdl_trigger();

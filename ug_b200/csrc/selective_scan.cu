@@ -1,20 +1,21 @@
 // Selective scan (see selective_scan.cuh).
 //
-//   selective_scan_kernel  a block of positions.  A CTA owns 256 / LP channels of one sequence and walks the block in
-//                          pieces of TT positions: step sizes (softplus), dt x, B and C go to shared memory, LP lanes per
-//                          channel advance NS states each in registers, and the sums over a channel's lanes are exchanged
-//                          eight positions at a time.  The next piece is on its way while a piece is worked on.
+//   selective_scan_kernel  a block of positions.  A CTA owns 128 / LP channels of one sequence and walks the block in
+//                          pieces of TT positions: four warps prepare step sizes (softplus), gates, B and C in shared memory,
+//                          four warps advance the states, LP lanes per channel with NS states each in registers, and
+//                          exchange the sums over a channel's lanes several positions at a time.
 //   selective_step_kernel  one position of several sequences: the step-size projection, the state update and the gate in one
 //                          kernel; everything that does not come from the preceding product is fetched ahead of the wait.
 #include "selective_scan.cuh"
+
+#include <algorithm>
+#include <type_traits>
 
 #include "hybrid_kernels.cuh"
 
 namespace {
 
 using namespace ugb_hybrid_k;
-
-constexpr int THREADS = 256;
 
 // softplus(x) = log(1 + e^x); fast form: hardware exp2 / log2, a short series where e^x is small
 template <bool EXACT> __device__ __forceinline__ float softplus_t(float x) {
@@ -79,6 +80,7 @@ template <int NS> __device__ __forceinline__ void st_states(float *p, const floa
   }
 }
 
+// ---------------------------------------------------------------- a block ----
 template <typename T> struct Block {
   const T *u, *dt, *xdb, *z;
   const float *a, *skip, *dt_bias;
@@ -88,118 +90,184 @@ template <typename T> struct Block {
   float scale;
   int channels, xr, rp, t;
 };
+constexpr int SCANNERS = 128, HELPERS = 128;
 
+// two floats at a time (one instruction each on this architecture)
+__device__ __forceinline__ uint64_t pack2(float a, float b) {
+  uint64_t r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+  return r;
+}
+__device__ __forceinline__ void unpack2(uint64_t v, float &a, float &b) { asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v)); }
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+  uint64_t r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+
+// The two halves of the CTA meet here from different places of the code: a barrier that is named, not __syncthreads.
+__device__ __forceinline__ void piece_barrier() { asm volatile("bar.sync 1, %0;" ::"n"(SCANNERS + HELPERS) : "memory"); }
+
+// grid (groups of 128 / LP channels, sequences).  128 scanning threads, 128 helping ones, pieces of TT positions in two shared
+// buffers: while the scanners advance the states over piece i, the helpers turn piece i + 1 -- fetched two pieces ahead -- into
+// step sizes, step size times input, output gate and skip term.
 template <typename T, int LP, int NS>
-__global__ void __launch_bounds__(THREADS)
+__global__ void __launch_bounds__(SCANNERS + HELPERS)
 selective_scan_kernel(Block<T> p) {
   constexpr bool EXACT = sizeof(T) == 4;
-  constexpr int CC = THREADS / LP, TT = LP == 8 ? 32 : 8, NP = LP * NS;
-  constexpr int PAIRS = (TT * CC / 2 + THREADS - 1) / THREADS;       // channel pairs a thread stages per piece
+  constexpr int CC = SCANNERS / LP, TT = LP <= 8 ? 16 : 8, NP = LP * NS, G = LP < 8 ? LP : 8;
+  constexpr int ROWS = HELPERS / (CC / 2);                           // positions between a helper's channel pairs
+  constexpr int PAIRS = (TT + ROWS - 1) / ROWS, BCS = TT * NP / HELPERS;
+  static_assert(NS % 2 == 0 && TT % G == 0 && BCS * HELPERS == TT * NP, "shape");
   using Raw = typename Pair<T>::Raw;
-  __shared__ float2 sdt[TT][CC];                                     // dt, dt x
-  __shared__ __align__(16) float sbc[TT][2 * NP];                    // B | C
-  __shared__ float sy[TT][CC + 4];                                   // the pitch keeps the exchange conflict-free
-  const int tid = threadIdx.x, ch = tid / LP, l = tid % LP;
-  const int c0 = blockIdx.x * CC, b = blockIdx.y, c = c0 + ch;
-  const bool on = c < p.channels;
+  __shared__ __align__(16) float4 sd[2][TT][CC];                     // dt, dt, dt x, dt x
+  __shared__ __align__(16) float sbc[2][TT][2 * NP];                 // B | C
+  __shared__ float2 sg[2][TT][CC + 4];                               // gate, skip x; the pitch keeps the scanners' reads conflict-free
+  const int tid = threadIdx.x, c0 = blockIdx.x * CC, b = blockIdx.y;
   const size_t row0 = (size_t)b * p.t;
+  const int pieces = (p.t + TT - 1) / TT;
+
+  if (tid >= SCANNERS) {
+    const int h = tid - SCANNERS, cp = (h % (CC / 2)) * 2, rs = h / (CC / 2);
+    const bool on = c0 + cp < p.channels;
+    float2 bias = make_float2(0.f, 0.f), skip = bias;
+    if (on) {
+      bias = *reinterpret_cast<const float2 *>(p.dt_bias + c0 + cp);
+      skip = *reinterpret_cast<const float2 *>(p.skip + c0 + cp);
+    }
+    const Raw zero = Pair<T>::pack(0.f, 0.f);
+    const T *pd = p.dt + row0 * p.channels + c0 + cp, *pu = p.u + row0 * p.channels + c0 + cp, *pz = p.z + row0 * p.z_ld + c0 + cp;
+    const T *pb = p.xdb + row0 * p.xr + p.rp;
+    struct Fetched { Raw d[PAIRS], u[PAIRS], z[PAIRS], bc[BCS]; } next, after;
+    auto fetch = [&](Fetched &f, int piece) {
+      const int t0 = piece * TT;
+#pragma unroll
+      for (int i = 0; i < PAIRS; ++i) {
+        const int s = rs + i * ROWS, t = t0 + s;
+        f.d[i] = f.u[i] = f.z[i] = zero;
+        if (s < TT && t < p.t && on) {
+          f.d[i] = ld_pair(pd + (size_t)t * p.channels);
+          f.u[i] = ld_pair(pu + (size_t)t * p.channels);
+          f.z[i] = ld_pair(pz + (size_t)t * p.z_ld);
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < BCS; ++i) {
+        const int idx = h + i * HELPERS, t = t0 + idx / NP;
+        f.bc[i] = t < p.t ? ld_pair(pb + (size_t)t * p.xr + 2 * (idx % NP)) : zero;
+      }
+    };
+    auto stage = [&](const Fetched &f, int piece) {
+      const int q = piece & 1, t0 = piece * TT;
+#pragma unroll
+      for (int i = 0; i < PAIRS; ++i) {
+        const int s = rs + i * ROWS;
+        if (s >= TT) continue;
+        const bool live = t0 + s < p.t;                              // behind the block: leaves the state alone
+        const float2 d = Pair<T>::wide(f.d[i]), u = Pair<T>::wide(f.u[i]), z = Pair<T>::wide(f.z[i]);
+        const float dx = live ? softplus_t<EXACT>(d.x + bias.x) : 0.f, dy = live ? softplus_t<EXACT>(d.y + bias.y) : 0.f;
+        sd[q][s][cp] = make_float4(dx, dx, dx * u.x, dx * u.x);
+        sd[q][s][cp + 1] = make_float4(dy, dy, dy * u.y, dy * u.y);
+        sg[q][s][cp] = make_float2(z.x * sigmoid_t<EXACT>(z.x) * p.scale, skip.x * u.x);
+        sg[q][s][cp + 1] = make_float2(z.y * sigmoid_t<EXACT>(z.y) * p.scale, skip.y * u.y);
+      }
+#pragma unroll
+      for (int i = 0; i < BCS; ++i) {
+        const int idx = h + i * HELPERS;
+        *reinterpret_cast<float2 *>(&sbc[q][idx / NP][2 * (idx % NP)]) = Pair<T>::wide(f.bc[i]);
+      }
+    };
+    fetch(next, 0);
+    fetch(after, 1);
+    stage(next, 0);
+    next = after;
+    fetch(after, 2);
+    piece_barrier();
+    for (int i = 0; i < pieces; ++i) {
+      if (i + 1 < pieces) {
+        stage(next, i + 1);
+        next = after;
+        fetch(after, i + 3);
+      }
+      piece_barrier();
+    }
+    return;
+  }
+
+  const int ch = tid / LP, l = tid % LP, c = c0 + ch;
+  const bool on = c < p.channels;
   float S[NS], A[NS];
 #pragma unroll
   for (int n = 0; n < NS; ++n) S[n] = A[n] = 0.f;
   float *state = p.state + ((size_t)b * p.channels + c) * NP + l * NS;
   if (on) { ld_states<NS>(state, S); ld_states<NS>(p.a + (size_t)c * NP + l * NS, A); }
-  // staging: this thread's channel pair is the same in every row
-  const int cp = (tid % (CC / 2)) * 2, rs = tid / (CC / 2);
-  constexpr int ROWS = THREADS / (CC / 2);                           // rows between a thread's pairs
-  const bool pair_on = c0 + cp < p.channels;
-  float2 bias = make_float2(0.f, 0.f), skip = bias;
-  if (pair_on) {
-    bias = *reinterpret_cast<const float2 *>(p.dt_bias + c0 + cp);
-    skip = *reinterpret_cast<const float2 *>(p.skip + c0 + cp);
-  }
-  const Raw zero = Pair<T>::pack(0.f, 0.f);
-  Raw rd[PAIRS], ru[PAIRS], rz[PAIRS], rb[NS];
-  auto fetch = [&](int t0) {
+  uint64_t S2[NS / 2], A2[NS / 2];
 #pragma unroll
-    for (int i = 0; i < PAIRS; ++i) {
-      const int s = rs + i * ROWS;
-      rd[i] = ru[i] = rz[i] = zero;
-      if (s < TT && t0 + s < p.t && pair_on) {
-        const size_t r = row0 + t0 + s;
-        rd[i] = ld_pair(p.dt + r * p.channels + c0 + cp);
-        ru[i] = ld_pair(p.u + r * p.channels + c0 + cp);
-        rz[i] = ld_pair(p.z + r * p.z_ld + c0 + cp);
-      }
-    }
+  for (int n = 0; n < NS / 2; ++n) { S2[n] = pack2(S[2 * n], S[2 * n + 1]); A2[n] = pack2(A[2 * n], A[2 * n + 1]); }
+  T *out = p.out + (row0 + l % G) * p.out_ld + c;
+  piece_barrier();
+  for (int i = 0; i < pieces; ++i) {
+    const int q = i & 1, t0 = i * TT;
+#pragma unroll(G < 8 ? 2 : 1)
+    for (int s0 = 0; s0 < TT; s0 += G) {
+      float v[G];
 #pragma unroll
-    for (int i = 0; i < NS; ++i) {                                   // TT * NP pairs of B and C
-      const int idx = tid + i * THREADS, s = idx / NP;
-      rb[i] = t0 + s < p.t ? ld_pair(p.xdb + (row0 + t0 + s) * p.xr + p.rp + 2 * (idx % NP)) : zero;
-    }
-  };
-  fetch(0);
-  for (int t0 = 0; t0 < p.t; t0 += TT) {
-    float2 u[PAIRS], z[PAIRS];
-#pragma unroll
-    for (int i = 0; i < PAIRS; ++i) {
-      const int s = rs + i * ROWS;
-      const float2 d = Pair<T>::wide(rd[i]);
-      u[i] = Pair<T>::wide(ru[i]);
-      z[i] = Pair<T>::wide(rz[i]);
-      if (s < TT) {
-        const bool live = t0 + s < p.t;                              // behind the block: leaves the state alone
-        const float dx = live ? softplus_t<EXACT>(d.x + bias.x) : 0.f, dy = live ? softplus_t<EXACT>(d.y + bias.y) : 0.f;
-        sdt[s][cp] = make_float2(dx, dx * u[i].x);
-        sdt[s][cp + 1] = make_float2(dy, dy * u[i].y);
-      }
-    }
-#pragma unroll
-    for (int i = 0; i < NS; ++i) {
-      const int idx = tid + i * THREADS;
-      *reinterpret_cast<float2 *>(&sbc[idx / NP][2 * (idx % NP)]) = Pair<T>::wide(rb[i]);
-    }
-    fetch(t0 + TT);
-    __syncthreads();
-#pragma unroll 1
-    for (int s0 = 0; s0 < TT; s0 += 8) {
-      float v[8];
-#pragma unroll
-      for (int k = 0; k < 8; ++k) {
-        const float2 d = sdt[s0 + k][ch];
+      for (int k = 0; k < G; ++k) {
+        const float4 d = sd[q][s0 + k][ch];
         float B[NS], C[NS];
-        ld_states<NS>(&sbc[s0 + k][l * NS], B);
-        ld_states<NS>(&sbc[s0 + k][NP + l * NS], C);
-        v[k] = 0.f;
+        ld_states<NS>(&sbc[q][s0 + k][l * NS], B);
+        ld_states<NS>(&sbc[q][s0 + k][NP + l * NS], C);
+        if constexpr (EXACT) {
+          v[k] = 0.f;
 #pragma unroll
-        for (int n = 0; n < NS; ++n) {
-          S[n] = advance<EXACT>(d.x * A[n], S[n], d.y * B[n]);
-          v[k] = fmaf(S[n], C[n], v[k]);
+          for (int n = 0; n < NS; ++n) {
+            S[n] = advance<true>(d.x * A[n], S[n], d.z * B[n]);
+            v[k] = fmaf(S[n], C[n], v[k]);
+          }
+        } else {
+          const uint64_t dt2 = pack2(d.x, d.y), dx2 = pack2(d.z, d.w);
+          uint64_t y2 = 0;
+#pragma unroll
+          for (int n = 0; n < NS / 2; ++n) {
+            float e0, e1;
+            unpack2(mul2(dt2, A2[n]), e0, e1);
+            asm("ex2.approx.ftz.f32 %0, %0;" : "+f"(e0));
+            asm("ex2.approx.ftz.f32 %0, %0;" : "+f"(e1));
+            S2[n] = fma2(pack2(e0, e1), S2[n], mul2(dx2, pack2(B[2 * n], B[2 * n + 1])));
+            y2 = n == 0 ? mul2(S2[n], pack2(C[0], C[1])) : fma2(S2[n], pack2(C[2 * n], C[2 * n + 1]), y2);
+          }
+          float a, e;
+          unpack2(y2, a, e);
+          v[k] = a + e;
         }
       }
-      // sums over the channel's lanes: every exchange halves the positions a lane still holds, lane l ends with l % 8
+      // sums over the channel's lanes: every exchange halves the positions a lane still holds, lane l ends with position l % G
 #pragma unroll
-      for (int w = 4; w >= 1; w >>= 1) {
+      for (int w = G / 2; w >= 1; w >>= 1) {
         const bool upper = (l & w) != 0;
 #pragma unroll
-        for (int i = 0; i < w; ++i) {
-          const float send = upper ? v[i] : v[i + w], keep = upper ? v[i + w] : v[i];
-          v[i] = keep + __shfl_xor_sync(0xffffffffu, send, w);
+        for (int k = 0; k < w; ++k) {
+          const float send = upper ? v[k] : v[k + w], keep = upper ? v[k + w] : v[k];
+          v[k] = keep + __shfl_xor_sync(0xffffffffu, send, w);
         }
       }
 #pragma unroll
-      for (int o = 8; o < LP; o <<= 1) v[0] += __shfl_xor_sync(0xffffffffu, v[0], o);
-      if (l < 8) sy[s0 + l][ch] = v[0];
-    }
-    __syncthreads();
-#pragma unroll
-    for (int i = 0; i < PAIRS; ++i) {
-      const int s = rs + i * ROWS;
-      if (s < TT && t0 + s < p.t && pair_on) {
-        const float gx = z[i].x * sigmoid_t<EXACT>(z[i].x) * p.scale, gy = z[i].y * sigmoid_t<EXACT>(z[i].y) * p.scale;
-        *reinterpret_cast<Raw *>(p.out + (row0 + t0 + s) * p.out_ld + c0 + cp) =
-            Pair<T>::pack(fmaf(skip.x, u[i].x, sy[s][cp]) * gx, fmaf(skip.y, u[i].y, sy[s][cp + 1]) * gy);
+      for (int o = G; o < LP; o <<= 1) v[0] += __shfl_xor_sync(0xffffffffu, v[0], o);
+      if (l < G && on && t0 + s0 + l < p.t) {
+        const float2 g = sg[q][s0 + l][ch];
+        out[(size_t)(t0 + s0) * p.out_ld] = (T)((v[0] + g.y) * g.x);
       }
     }
+    piece_barrier();
+  }
+  if constexpr (!EXACT) {
+#pragma unroll
+    for (int n = 0; n < NS / 2; ++n) unpack2(S2[n], S[2 * n], S[2 * n + 1]);
   }
   if (on) st_states<NS>(state, S);
 }
@@ -213,61 +281,74 @@ template <typename T> struct Step {
   T *out;
   size_t out_ld;
   float scale;
-  int channels, xr, rp, rows, early;
+  int channels, xr, rp, rows, group, w_shared, early;                // group: sequences of a CTA; w_shared: W_dt columns in shared memory
 };
-constexpr int STEP_ROWS = 4;         // sequences of a CTA
-constexpr int STEP_W = 16;           // step-size weights a thread holds from before the wait
+constexpr int THREADS = 256;
+constexpr int STEP_J = 4;            // sequences per thread in the projection and the element-wise parts
 
-// grid (groups of 256 / LP channels, groups of STEP_ROWS sequences); dynamic shared memory: low | B | C of the sequences
+// grid (groups of 256 / LP channels, groups of `group` sequences).  Dynamic shared memory: dt, dt x [group][CC]; low | B | C
+// [group][xr]; sums over the states [group][CC]; W_dt [rp][CC].
 template <typename T, int LP, int NS>
 __global__ void __launch_bounds__(THREADS)
 selective_step_kernel(Step<T> p) {
   constexpr bool EXACT = sizeof(T) == 4;
-  constexpr int CC = THREADS / LP, NP = LP * NS, KG = THREADS / CC, R = STEP_ROWS;
-  extern __shared__ __align__(16) float xs[];                        // [R][xr]
-  __shared__ float red[KG][R][CC];
-  __shared__ float2 sd[R][CC];                                       // dt, dt x
-  __shared__ float sy[R][CC];
+  constexpr int CC = THREADS / LP, NP = LP * NS, D = NS <= 4 ? 4 : 2;   // D: sequences whose states are in flight per thread
+  extern __shared__ __align__(16) float dyn[];
+  float2 *sd = reinterpret_cast<float2 *>(dyn);                      // [group][CC]
+  float *xs = dyn + 2 * p.group * CC, *sy = xs + p.group * p.xr;
+  T *ws = reinterpret_cast<T *>(sy + p.group * CC);
   const int tid = threadIdx.x, ch = tid / LP, l = tid % LP;
-  const int c0 = blockIdx.x * CC, r0 = blockIdx.y * R, n_rows = min(R, p.rows - r0);
+  const int c0 = blockIdx.x * CC, r0 = blockIdx.y * p.group, n_rows = min(p.group, p.rows - r0);
   if (!p.early) { ugb_pdl_wait(); ugb_pdl_trigger(); }
   const int c = c0 + ch;
   const bool on = c < p.channels;
-  float A[NS], S[R][NS];
+  float A[NS];
 #pragma unroll
   for (int n = 0; n < NS; ++n) A[n] = 0.f;
   if (on) ld_states<NS>(p.a + (size_t)c * NP + l * NS, A);
+  float *state = p.state + ((size_t)r0 * p.channels + c) * NP + l * NS;
+  const size_t next_row = (size_t)p.channels * NP;
+  float S[D][NS], Sn[D][NS];
+  auto load = [&](float (&v)[D][NS], int r) {
 #pragma unroll
-  for (int r = 0; r < R; ++r) {
+    for (int d = 0; d < D; ++d) {
 #pragma unroll
-    for (int n = 0; n < NS; ++n) S[r][n] = 0.f;
-    if (on && r < n_rows) ld_states<NS>(p.state + ((size_t)(r0 + r) * p.channels + c) * NP + l * NS, S[r]);
-  }
-  // (sequence, channel) of this thread in the element-wise parts, and (channel, part of the rank) in the projection
-  const int er = tid / CC, ec = tid % CC;
-  const bool own = er < n_rows && c0 + ec < p.channels;
-  float u = 0.f, z = 0.f, bias = 0.f, skip = 0.f;
-  if (own) {
-    u = (float)p.u[(size_t)(r0 + er) * p.channels + c0 + ec];
-    bias = __ldg(p.dt_bias + c0 + ec);
-    skip = __ldg(p.skip + c0 + ec);
-    for (int q = 0; q < p.z.n; ++q) z += p.z.p[q * p.z.stride + (size_t)(r0 + er) * p.z.ld + c0 + ec];
-  }
-  const int kk = tid / CC;
+      for (int n = 0; n < NS; ++n) v[d][n] = 0.f;
+      if (on && r + d < n_rows) ld_states<NS>(state + (size_t)(r + d) * next_row, v[d]);
+    }
+  };
+  load(S, 0);
+  // channel and sequences of this thread in the projection and the element-wise parts
+  const int ec = tid % CC, er = tid / CC;
   const bool col = c0 + ec < p.channels;
-  float w[STEP_W];
+  float u[STEP_J], z[STEP_J], bias = 0.f, skip = 0.f;
+  if (col) { bias = __ldg(p.dt_bias + c0 + ec); skip = __ldg(p.skip + c0 + ec); }
 #pragma unroll
-  for (int i = 0; i < STEP_W; ++i) w[i] = col && kk + i * KG < p.rp ? (float)p.w_dt[(size_t)(kk + i * KG) * p.channels + c0 + ec] : 0.f;
+  for (int j = 0; j < STEP_J; ++j) {
+    const int r = er + LP * j;
+    u[j] = z[j] = 0.f;
+    if (r < n_rows && col) {
+      u[j] = (float)p.u[(size_t)(r0 + r) * p.channels + c0 + ec];
+      for (int q = 0; q < p.z.n; ++q) z[j] += p.z.p[q * p.z.stride + (size_t)(r0 + r) * p.z.ld + c0 + ec];
+    }
+  }
+  if (p.w_shared)
+    for (int i = tid; i < p.rp * (CC / 8); i += THREADS) {           // channels is a multiple of 8
+      const int k = i / (CC / 8), w = 8 * (i - k * (CC / 8));
+      Row8<T> v{};
+      if (c0 + w < p.channels) v = ld8<T>(p.w_dt + (size_t)k * p.channels + c0 + w);
+      st8<T>(ws + k * CC + w, v);
+    }
   if (p.early) { ugb_pdl_wait(); ugb_pdl_trigger(); }
-  for (int i = tid; i < R * (p.xr / 4); i += THREADS) {
+  for (int i = tid; i < p.group * (p.xr / 4); i += THREADS) {
     const int r = i / (p.xr / 4), k = 4 * (i - r * (p.xr / 4));
     float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
     if (r < n_rows)
-      for (int q = 0; q < p.xdb.n; q += 4) {
+      for (int q = 0; q < p.xdb.n; q += 4) {                         // the partials are added in order
         float4 v[4];
 #pragma unroll
         for (int e = 0; e < 4; ++e)
-          v[e] = q + e < p.xdb.n ? __ldcs(reinterpret_cast<const float4 *>(p.xdb.p + (q + e) * p.xdb.stride + (size_t)(r0 + r) * p.xdb.ld + k))
+          v[e] = q + e < p.xdb.n ? *reinterpret_cast<const float4 *>(p.xdb.p + (q + e) * p.xdb.stride + (size_t)(r0 + r) * p.xdb.ld + k)
                                  : make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
         for (int e = 0; e < 4; ++e) { s.x += v[e].x; s.y += v[e].y; s.z += v[e].z; s.w += v[e].w; }
@@ -275,60 +356,84 @@ selective_step_kernel(Step<T> p) {
     *reinterpret_cast<float4 *>(xs + r * p.xr + k) = s;
   }
   __syncthreads();
-  float acc[R];
+  {
+    float acc[STEP_J];
 #pragma unroll
-  for (int r = 0; r < R; ++r) acc[r] = 0.f;
+    for (int j = 0; j < STEP_J; ++j) acc[j] = bias;
+    auto project = [&](auto weight) {
+      for (int k = 0; k < p.rp; k += 4) {                            // rp is a multiple of 8
+        float w[4];
 #pragma unroll
-  for (int i = 0; i < STEP_W; ++i) {
-    const int k = kk + i * KG;
-    if (k < p.rp) {
+        for (int e = 0; e < 4; ++e) w[e] = weight(k + e);
 #pragma unroll
-      for (int r = 0; r < R; ++r) acc[r] = fmaf(w[i], xs[r * p.xr + k], acc[r]);
+        for (int j = 0; j < STEP_J; ++j) {
+          if (er + LP * j >= p.group) break;
+          const float4 x = *reinterpret_cast<const float4 *>(xs + (er + LP * j) * p.xr + k);
+          acc[j] = fmaf(w[0], x.x, acc[j]); acc[j] = fmaf(w[1], x.y, acc[j]);
+          acc[j] = fmaf(w[2], x.z, acc[j]); acc[j] = fmaf(w[3], x.w, acc[j]);
+        }
+      }
+    };
+    if (p.w_shared) project([&](int k) { return (float)ws[k * CC + ec]; });
+    else project([&](int k) { return col ? (float)p.w_dt[(size_t)k * p.channels + c0 + ec] : 0.f; });
+#pragma unroll
+    for (int j = 0; j < STEP_J; ++j) {
+      if (er + LP * j >= p.group) break;
+      const float d = softplus_t<EXACT>(acc[j]);
+      sd[(er + LP * j) * CC + ec] = make_float2(d, d * u[j]);
     }
   }
-  for (int k = kk + STEP_W * KG; k < p.rp; k += KG) {                // a rank that does not fit the registers
-    const float wk = col ? (float)p.w_dt[(size_t)k * p.channels + c0 + ec] : 0.f;
-#pragma unroll
-    for (int r = 0; r < R; ++r) acc[r] = fmaf(wk, xs[r * p.xr + k], acc[r]);
-  }
-#pragma unroll
-  for (int r = 0; r < R; ++r) red[kk][r][ec] = acc[r];
   __syncthreads();
-  if (er < R) {
-    float s = bias;
+  for (int r = 0; r < n_rows; r += D) {
+    load(Sn, r + D);
+    float y[D];
 #pragma unroll
-    for (int k = 0; k < KG; ++k) s += red[k][er][ec];
-    const float d = softplus_t<EXACT>(s);
-    sd[er][ec] = make_float2(d, d * u);
-  }
-  __syncthreads();
+    for (int d = 0; d < D; ++d) {
+      y[d] = 0.f;
+      if (r + d >= n_rows) continue;                                 // the same for the whole CTA
+      const float2 dt = sd[(r + d) * CC + ch];
+      const float *bc = xs + (r + d) * p.xr + p.rp + l * NS;
+      float B[NS], C[NS];
+      ld_states<NS>(bc, B);
+      ld_states<NS>(bc + NP, C);
 #pragma unroll
-  for (int r = 0; r < R; ++r) {
-    const float2 d = sd[r][ch];
-    const float *bc = xs + r * p.xr + p.rp + l * NS;
-    float y = 0.f;
-#pragma unroll
-    for (int n = 0; n < NS; ++n) {
-      S[r][n] = advance<EXACT>(d.x * A[n], S[r][n], d.y * bc[n]);
-      y = fmaf(S[r][n], bc[NP + n], y);
+      for (int n = 0; n < NS; ++n) {
+        S[d][n] = advance<EXACT>(dt.x * A[n], S[d][n], dt.y * B[n]);
+        y[d] = fmaf(S[d][n], C[n], y[d]);
+      }
+      if (on) st_states<NS>(state + (size_t)(r + d) * next_row, S[d]);
     }
-    if (on && r < n_rows) st_states<NS>(p.state + ((size_t)(r0 + r) * p.channels + c) * NP + l * NS, S[r]);
 #pragma unroll
-    for (int o = 1; o < LP; o <<= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-    if (l == 0) sy[r][ch] = y;
+    for (int o = 1; o < LP; o <<= 1)
+#pragma unroll
+      for (int d = 0; d < D; ++d) y[d] += __shfl_xor_sync(0xffffffffu, y[d], o);
+    if (l == 0) {
+#pragma unroll
+      for (int d = 0; d < D; ++d)
+        if (r + d < n_rows) sy[(r + d) * CC + ch] = y[d];
+    }
+#pragma unroll
+    for (int d = 0; d < D; ++d)
+#pragma unroll
+      for (int n = 0; n < NS; ++n) S[d][n] = Sn[d][n];
   }
   __syncthreads();
-  if (own) p.out[(size_t)(r0 + er) * p.out_ld + c0 + ec] = (T)(fmaf(skip, u, sy[er][ec]) * z * sigmoid_t<EXACT>(z) * p.scale);
+#pragma unroll
+  for (int j = 0; j < STEP_J; ++j) {
+    const int r = er + LP * j;
+    if (r < n_rows && col)
+      p.out[(size_t)(r0 + r) * p.out_ld + c0 + ec] = (T)(fmaf(skip, u[j], sy[r * CC + ec]) * z[j] * sigmoid_t<EXACT>(z[j]) * p.scale);
+  }
 }
 
 template <typename T, int LP, int NS>
 int32_t block_one(ugb_device *dev, const ugb_scan_args &a, const void *dt, const void *xdb, const void *z, size_t z_ld, int b, int t) {
-  constexpr int CC = THREADS / LP;
+  constexpr int CC = SCANNERS / LP;
   Block<T> p;
   p.u = (const T *)a.u; p.dt = (const T *)dt; p.xdb = (const T *)xdb; p.z = (const T *)z; p.a = a.a; p.skip = a.skip; p.dt_bias = a.dt_bias;
   p.state = a.state; p.out = (T *)a.out; p.z_ld = z_ld; p.out_ld = a.out_ld; p.scale = a.scale; p.channels = a.channels; p.xr = a.xr;
   p.rp = a.rp; p.t = t;
-  selective_scan_kernel<T, LP, NS><<<dim3((a.channels + CC - 1) / CC, b), THREADS, 0, dev->stream>>>(p);
+  selective_scan_kernel<T, LP, NS><<<dim3((a.channels + CC - 1) / CC, b), SCANNERS + HELPERS, 0, dev->stream>>>(p);
   return ugb_after_launch(dev, "selective_scan_kernel");
 }
 template <typename T, int LP, int NS>
@@ -338,8 +443,17 @@ int32_t step_one(ugb_device *dev, const ugb_scan_args &a, const void *w_dt, ugb_
   p.u = (const T *)a.u; p.w_dt = (const T *)w_dt; p.xdb = xdb; p.z = z; p.a = a.a; p.skip = a.skip; p.dt_bias = a.dt_bias; p.state = a.state;
   p.out = (T *)a.out; p.out_ld = a.out_ld; p.scale = a.scale; p.channels = a.channels; p.xr = a.xr; p.rp = a.rp; p.rows = rows;
   p.early = early && pdl ? 1 : 0;
-  const cudaError_t e = ugb_launch(selective_step_kernel<T, LP, NS>, dim3((a.channels + CC - 1) / CC, (rows + STEP_ROWS - 1) / STEP_ROWS),
-                                   dim3(THREADS), (size_t)STEP_ROWS * a.xr * 4, dev->stream, pdl, p);
+  // sequences per CTA: enough CTAs for two per SM, no more than a thread's share and the shared memory allow
+  const int groups = (a.channels + CC - 1) / CC, most = std::min(STEP_J * LP, 32);
+  const size_t w_bytes = (size_t)a.rp * CC * sizeof(T), limit = 48 * 1024;
+  p.w_shared = w_bytes <= 24 * 1024;
+  const size_t fixed = p.w_shared ? w_bytes : 0, per_row = (size_t)CC * 12 + (size_t)a.xr * 4;
+  p.group = most;
+  while (p.group > 4 && (long long)groups * ((rows + p.group - 1) / p.group) < 2 * dev->sm_count) p.group /= 2;
+  while (p.group > 1 && fixed + p.group * per_row > limit) p.group /= 2;
+  UGB_REQUIRE(dev, fixed + p.group * per_row <= limit, UGB_ERR_UNSUPPORTED, "selective scan: %d columns of step size, B and C", a.xr);
+  const cudaError_t e = ugb_launch(selective_step_kernel<T, LP, NS>, dim3(groups, (rows + p.group - 1) / p.group), dim3(THREADS),
+                                   fixed + p.group * per_row, dev->stream, pdl, p);
   if (e != cudaSuccess) return ugb_fail(dev, UGB_ERR_CUDA, "launch of selective_step_kernel failed: %s", cudaGetErrorString(e));
   return ugb_after_launch(dev, "selective_step_kernel");
 }
@@ -347,7 +461,7 @@ int32_t step_one(ugb_device *dev, const ugb_scan_args &a, const void *w_dt, ugb_
 // f(LP, NS) for the kernel of a shape
 template <typename F> int32_t with_shape(ugb_device *dev, const ugb_scan_shape &s, F f) {
 #define SHAPE(LP, NS) if (s.lanes == LP && s.per_lane == NS) return f(std::integral_constant<int, LP>(), std::integral_constant<int, NS>())
-  SHAPE(8, 1); SHAPE(8, 2); SHAPE(8, 3); SHAPE(8, 4); SHAPE(8, 6); SHAPE(8, 8); SHAPE(32, 4); SHAPE(32, 8);
+  SHAPE(4, 2); SHAPE(4, 4); SHAPE(4, 6); SHAPE(4, 8); SHAPE(8, 6); SHAPE(8, 8); SHAPE(16, 8); SHAPE(32, 8);
 #undef SHAPE
   return ugb_fail(dev, UGB_ERR_UNSUPPORTED, "selective scan: no kernel for %d states on %d lanes", s.np, s.lanes);
 }
@@ -361,10 +475,12 @@ int32_t check(ugb_device *dev, const ugb_scan_args &a) {
 }  // namespace
 
 ugb_scan_shape ugb_scan_shape_of(int states) {
-  for (int ns : {1, 2, 3, 4, 6, 8})
+  for (int ns : {2, 4, 6, 8})
+    if (states <= 4 * ns) return {4, ns, 4 * ns};
+  for (int ns : {6, 8})
     if (states <= 8 * ns) return {8, ns, 8 * ns};
-  for (int ns : {4, 8})
-    if (states <= 32 * ns) return {32, ns, 32 * ns};
+  for (int lanes : {16, 32})
+    if (states <= 8 * lanes) return {lanes, 8, 8 * lanes};
   return {0, 0, 0};
 }
 
@@ -382,7 +498,6 @@ int32_t ugb_scan_block(ugb_device *dev, const ugb_scan_args &a, const void *dt, 
 int32_t ugb_scan_step(ugb_device *dev, const ugb_scan_args &a, const void *w_dt, ugb_scan_partials xdb, ugb_scan_partials z, int rows, bool pdl, bool early) {
   if (rows == 0) return UGB_OK;
   if (int32_t rc = check(dev, a)) return rc;
-  UGB_REQUIRE(dev, (size_t)STEP_ROWS * a.xr * 4 <= 40 * 1024, UGB_ERR_UNSUPPORTED, "selective scan: %d columns of step size, B and C", a.xr);
   return with_shape(dev, a.shape, [&](auto lp, auto ns) {
     return a.f32 ? step_one<float, lp(), ns()>(dev, a, w_dt, xdb, z, rows, pdl, early) : step_one<__nv_bfloat16, lp(), ns()>(dev, a, w_dt, xdb, z, rows, pdl, early);
   });
