@@ -1,9 +1,9 @@
 // Selective scan (see selective_scan.cuh).
 //
-//   selective_scan_kernel  a block of positions.  A CTA owns 128 / LP channels of one sequence and walks the block in
+//   selective_scan_kernel  a block of positions.  A CTA owns a group of channels of one sequence and walks the block in
 //                          pieces of TT positions: four warps prepare step sizes (softplus), gates, B and C in shared memory,
-//                          four warps advance the states, LP lanes per channel with NS states each in registers, and
-//                          exchange the sums over a channel's lanes several positions at a time.
+//                          the others advance the states, LP lanes per channel pair with NS states of each in registers,
+//                          and exchange the sums over the lanes eight positions at a time.
 //   selective_step_kernel  one position of several sequences: the step-size projection, the state update and the gate in one
 //                          kernel; everything that does not come from the preceding product is fetched ahead of the wait.
 #include "selective_scan.cuh"
@@ -90,7 +90,10 @@ template <typename T> struct Block {
   float scale;
   int channels, xr, rp, t;
 };
-constexpr int SCANNERS = 128, HELPERS = 128;
+constexpr int HELPERS = 128;
+template <int LP, int NS> struct ScanCta {
+  static constexpr int CC = LP * NS <= 64 ? 32 : 256 / LP, SCANNERS = CC / 2 * LP, ALL = SCANNERS + HELPERS;
+};
 
 // two floats at a time (one instruction each on this architecture)
 __device__ __forceinline__ uint64_t pack2(float a, float b) {
@@ -111,55 +114,52 @@ __device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
 }
 
 // The two halves of the CTA meet here from different places of the code: a barrier that is named, not __syncthreads.
-__device__ __forceinline__ void piece_barrier() { asm volatile("bar.sync 1, %0;" ::"n"(SCANNERS + HELPERS) : "memory"); }
+template <int THREADS> __device__ __forceinline__ void piece_barrier() { asm volatile("bar.sync 1, %0;" ::"n"(THREADS) : "memory"); }
 
-// grid (groups of 128 / LP channels, sequences).  128 scanning threads, 128 helping ones, pieces of TT positions in two shared
-// buffers: while the scanners advance the states over piece i, the helpers turn piece i + 1 -- fetched two pieces ahead -- into
-// step sizes, step size times input, output gate and skip term.
-template <typename T, int LP, int NS>
-__global__ void __launch_bounds__(SCANNERS + HELPERS)
+// grid (groups of CC channels, sequences).  A scanning thread has NS states of two neighbouring channels, LP lanes share a pair
+// of channels; 128 threads help.  Pieces of TT positions lie in two shared buffers: while the scanners advance the states over
+// piece i, the helpers turn piece i + 1 -- fetched two pieces ahead -- into step sizes, step size times input, output gate and
+// skip term.  Two channels per thread, because shared memory is what bounds this kernel: a 16-byte read takes four passes
+// whatever its lanes have in common, and B and C are read once for both.
+// CTAS: resident per SM.  Alone on its SM a CTA is bound by its own latencies and takes longer pieces and more registers.
+template <typename T, int LP, int NS, int TT, int CTAS>
+__global__ void __launch_bounds__(ScanCta<LP, NS>::ALL, CTAS)
 selective_scan_kernel(Block<T> p) {
   constexpr bool EXACT = sizeof(T) == 4;
-  constexpr int CC = SCANNERS / LP, TT = LP <= 8 ? 16 : 8, NP = LP * NS, G = LP < 8 ? LP : 8;
+  constexpr int CC = ScanCta<LP, NS>::CC, SCANNERS = ScanCta<LP, NS>::SCANNERS, NP = LP * NS, G = 8;
   constexpr int ROWS = HELPERS / (CC / 2);                           // positions between a helper's channel pairs
   constexpr int PAIRS = (TT + ROWS - 1) / ROWS, BCS = TT * NP / HELPERS;
-  static_assert(NS % 2 == 0 && TT % G == 0 && BCS * HELPERS == TT * NP, "shape");
+  static_assert(TT % G == 0 && BCS * HELPERS == TT * NP, "shape");
   using Raw = typename Pair<T>::Raw;
-  __shared__ __align__(16) float4 sd[2][TT][CC];                     // dt, dt, dt x, dt x
+  __shared__ __align__(16) float4 sd[2][TT][CC / 2];                 // of a channel pair: dt, dt, dt x, dt x
   __shared__ __align__(16) float sbc[2][TT][2 * NP];                 // B | C
-  __shared__ float2 sg[2][TT][CC + 4];                               // gate, skip x; the pitch keeps the scanners' reads conflict-free
+  __shared__ __align__(16) float4 sg[2][TT][CC / 2 + 1];   // gate, gate, skip x, skip x; the pitch avoids conflicts
   const int tid = threadIdx.x, c0 = blockIdx.x * CC, b = blockIdx.y;
   const size_t row0 = (size_t)b * p.t;
   const int pieces = (p.t + TT - 1) / TT;
 
   if (tid >= SCANNERS) {
-    const int h = tid - SCANNERS, cp = (h % (CC / 2)) * 2, rs = h / (CC / 2);
-    const bool on = c0 + cp < p.channels;
-    float2 bias = make_float2(0.f, 0.f), skip = bias;
-    if (on) {
-      bias = *reinterpret_cast<const float2 *>(p.dt_bias + c0 + cp);
-      skip = *reinterpret_cast<const float2 *>(p.skip + c0 + cp);
-    }
-    const Raw zero = Pair<T>::pack(0.f, 0.f);
-    const T *pd = p.dt + row0 * p.channels + c0 + cp, *pu = p.u + row0 * p.channels + c0 + cp, *pz = p.z + row0 * p.z_ld + c0 + cp;
+    // channel pair and first position of this helper; addresses outside the block or the model are brought back inside, what is
+    // loaded from there is not used
+    const int h = tid - SCANNERS, cp = (h % (CC / 2)) * 2, rs = h / (CC / 2), cl = min(c0 + cp, p.channels - 2), last = p.t - 1;
+    const float2 bias = *reinterpret_cast<const float2 *>(p.dt_bias + cl), skip = *reinterpret_cast<const float2 *>(p.skip + cl);
+    const T *pd = p.dt + row0 * p.channels + cl, *pu = p.u + row0 * p.channels + cl, *pz = p.z + row0 * p.z_ld + cl;
     const T *pb = p.xdb + row0 * p.xr + p.rp;
-    struct Fetched { Raw d[PAIRS], u[PAIRS], z[PAIRS], bc[BCS]; } next, after;
+    struct Fetched { Raw d[PAIRS], u[PAIRS], z[PAIRS], bc[BCS]; } even, odd;
     auto fetch = [&](Fetched &f, int piece) {
       const int t0 = piece * TT;
 #pragma unroll
       for (int i = 0; i < PAIRS; ++i) {
-        const int s = rs + i * ROWS, t = t0 + s;
-        f.d[i] = f.u[i] = f.z[i] = zero;
-        if (s < TT && t < p.t && on) {
-          f.d[i] = ld_pair(pd + (size_t)t * p.channels);
-          f.u[i] = ld_pair(pu + (size_t)t * p.channels);
-          f.z[i] = ld_pair(pz + (size_t)t * p.z_ld);
-        }
+        const int t = min(t0 + rs + i * ROWS, last);
+        const size_t at = (size_t)t * p.channels;
+        f.d[i] = ld_pair(pd + at);
+        f.u[i] = ld_pair(pu + at);
+        f.z[i] = ld_pair(pz + (size_t)t * p.z_ld);
       }
 #pragma unroll
       for (int i = 0; i < BCS; ++i) {
-        const int idx = h + i * HELPERS, t = t0 + idx / NP;
-        f.bc[i] = t < p.t ? ld_pair(pb + (size_t)t * p.xr + 2 * (idx % NP)) : zero;
+        const int idx = h + i * HELPERS, t = min(t0 + idx / NP, last);
+        f.bc[i] = ld_pair(pb + (size_t)t * p.xr + 2 * (idx % NP));
       }
     };
     auto stage = [&](const Fetched &f, int piece) {
@@ -167,14 +167,12 @@ selective_scan_kernel(Block<T> p) {
 #pragma unroll
       for (int i = 0; i < PAIRS; ++i) {
         const int s = rs + i * ROWS;
-        if (s >= TT) continue;
-        const bool live = t0 + s < p.t;                              // behind the block: leaves the state alone
+        if (TT % ROWS != 0 && s >= TT) continue;
+        const bool live = t0 + s <= last;                            // behind the block: leaves the state alone
         const float2 d = Pair<T>::wide(f.d[i]), u = Pair<T>::wide(f.u[i]), z = Pair<T>::wide(f.z[i]);
         const float dx = live ? softplus_t<EXACT>(d.x + bias.x) : 0.f, dy = live ? softplus_t<EXACT>(d.y + bias.y) : 0.f;
-        sd[q][s][cp] = make_float4(dx, dx, dx * u.x, dx * u.x);
-        sd[q][s][cp + 1] = make_float4(dy, dy, dy * u.y, dy * u.y);
-        sg[q][s][cp] = make_float2(z.x * sigmoid_t<EXACT>(z.x) * p.scale, skip.x * u.x);
-        sg[q][s][cp + 1] = make_float2(z.y * sigmoid_t<EXACT>(z.y) * p.scale, skip.y * u.y);
+        sd[q][s][cp / 2] = make_float4(dx, dy, dx * u.x, dy * u.y);
+        sg[q][s][cp / 2] = make_float4(z.x * sigmoid_t<EXACT>(z.x) * p.scale, z.y * sigmoid_t<EXACT>(z.y) * p.scale, skip.x * u.x, skip.y * u.y);
       }
 #pragma unroll
       for (int i = 0; i < BCS; ++i) {
@@ -182,94 +180,112 @@ selective_scan_kernel(Block<T> p) {
         *reinterpret_cast<float2 *>(&sbc[q][idx / NP][2 * (idx % NP)]) = Pair<T>::wide(f.bc[i]);
       }
     };
-    fetch(next, 0);
-    fetch(after, 1);
-    stage(next, 0);
-    next = after;
-    fetch(after, 2);
-    piece_barrier();
-    for (int i = 0; i < pieces; ++i) {
+    fetch(even, 0);
+    fetch(odd, 1);
+    stage(even, 0);
+    fetch(even, 2);
+    piece_barrier<ScanCta<LP, NS>::ALL>();
+    for (int i = 0; i < pieces; i += 2) {                            // pieces i + 1 and i + 2 are prepared; a fetch is used two pieces later
       if (i + 1 < pieces) {
-        stage(next, i + 1);
-        next = after;
-        fetch(after, i + 3);
+        stage(odd, i + 1);
+        fetch(odd, i + 3);
       }
-      piece_barrier();
+      piece_barrier<ScanCta<LP, NS>::ALL>();
+      if (i + 1 >= pieces) break;
+      if (i + 2 < pieces) {
+        stage(even, i + 2);
+        fetch(even, i + 4);
+      }
+      piece_barrier<ScanCta<LP, NS>::ALL>();
     }
     return;
   }
 
-  const int ch = tid / LP, l = tid % LP, c = c0 + ch;
-  const bool on = c < p.channels;
-  float S[NS], A[NS];
-#pragma unroll
-  for (int n = 0; n < NS; ++n) S[n] = A[n] = 0.f;
+  const int pair = tid / LP, l = tid % LP, c = c0 + 2 * pair;
+  const bool on = c < p.channels;                                    // channels is even
+  uint64_t S2[NS], A2[NS];                                           // (this channel, the next)
   float *state = p.state + ((size_t)b * p.channels + c) * NP + l * NS;
-  if (on) { ld_states<NS>(state, S); ld_states<NS>(p.a + (size_t)c * NP + l * NS, A); }
-  uint64_t S2[NS / 2], A2[NS / 2];
+  {
+    float s0[NS], s1[NS], a0[NS], a1[NS];
 #pragma unroll
-  for (int n = 0; n < NS / 2; ++n) { S2[n] = pack2(S[2 * n], S[2 * n + 1]); A2[n] = pack2(A[2 * n], A[2 * n + 1]); }
+    for (int n = 0; n < NS; ++n) s0[n] = s1[n] = a0[n] = a1[n] = 0.f;
+    if (on) {
+      const float *a = p.a + (size_t)c * NP + l * NS;
+      ld_states<NS>(state, s0); ld_states<NS>(state + NP, s1); ld_states<NS>(a, a0); ld_states<NS>(a + NP, a1);
+    }
+#pragma unroll
+    for (int n = 0; n < NS; ++n) { S2[n] = pack2(s0[n], s1[n]); A2[n] = pack2(a0[n], a1[n]); }
+  }
   T *out = p.out + (row0 + l % G) * p.out_ld + c;
-  piece_barrier();
+  piece_barrier<ScanCta<LP, NS>::ALL>();
   for (int i = 0; i < pieces; ++i) {
     const int q = i & 1, t0 = i * TT;
-#pragma unroll(G < 8 ? 2 : 1)
+    float2 y[TT / G];                                                // stored after the piece: a store would hold up the next reads
+#pragma unroll
     for (int s0 = 0; s0 < TT; s0 += G) {
-      float v[G];
+      float v[G], w[G];                                              // sums of the two channels
 #pragma unroll
       for (int k = 0; k < G; ++k) {
-        const float4 d = sd[q][s0 + k][ch];
+        const float4 d = sd[q][s0 + k][pair];
         float B[NS], C[NS];
         ld_states<NS>(&sbc[q][s0 + k][l * NS], B);
         ld_states<NS>(&sbc[q][s0 + k][NP + l * NS], C);
-        if constexpr (EXACT) {
-          v[k] = 0.f;
+        v[k] = w[k] = 0.f;
+        const uint64_t dt2 = pack2(d.x, d.y);
 #pragma unroll
-          for (int n = 0; n < NS; ++n) {
-            S[n] = advance<true>(d.x * A[n], S[n], d.z * B[n]);
-            v[k] = fmaf(S[n], C[n], v[k]);
+        for (int n = 0; n < NS; ++n) {
+          float x0, x1, s0v, s1v;
+          unpack2(mul2(dt2, A2[n]), x0, x1);
+          if constexpr (EXACT) {
+            unpack2(S2[n], s0v, s1v);
+            s0v = advance<true>(x0, s0v, d.z * B[n]);
+            s1v = advance<true>(x1, s1v, d.w * B[n]);
+            S2[n] = pack2(s0v, s1v);
+          } else {
+            asm("ex2.approx.ftz.f32 %0, %0;" : "+f"(x0));
+            asm("ex2.approx.ftz.f32 %0, %0;" : "+f"(x1));
+            S2[n] = fma2(pack2(x0, x1), S2[n], pack2(d.z * B[n], d.w * B[n]));
+            unpack2(S2[n], s0v, s1v);
           }
-        } else {
-          const uint64_t dt2 = pack2(d.x, d.y), dx2 = pack2(d.z, d.w);
-          uint64_t y2 = 0;
-#pragma unroll
-          for (int n = 0; n < NS / 2; ++n) {
-            float e0, e1;
-            unpack2(mul2(dt2, A2[n]), e0, e1);
-            asm("ex2.approx.ftz.f32 %0, %0;" : "+f"(e0));
-            asm("ex2.approx.ftz.f32 %0, %0;" : "+f"(e1));
-            S2[n] = fma2(pack2(e0, e1), S2[n], mul2(dx2, pack2(B[2 * n], B[2 * n + 1])));
-            y2 = n == 0 ? mul2(S2[n], pack2(C[0], C[1])) : fma2(S2[n], pack2(C[2 * n], C[2 * n + 1]), y2);
-          }
-          float a, e;
-          unpack2(y2, a, e);
-          v[k] = a + e;
+          v[k] = fmaf(s0v, C[n], v[k]);
+          w[k] = fmaf(s1v, C[n], w[k]);
         }
       }
-      // sums over the channel's lanes: every exchange halves the positions a lane still holds, lane l ends with position l % G
+      // sums over the lanes of a pair: every exchange halves the positions a lane still holds, lane l ends with position l % G
 #pragma unroll
-      for (int w = G / 2; w >= 1; w >>= 1) {
-        const bool upper = (l & w) != 0;
+      for (int h = G / 2; h >= 1; h >>= 1) {
+        const bool upper = (l & h) != 0;
 #pragma unroll
-        for (int k = 0; k < w; ++k) {
-          const float send = upper ? v[k] : v[k + w], keep = upper ? v[k + w] : v[k];
-          v[k] = keep + __shfl_xor_sync(0xffffffffu, send, w);
+        for (int k = 0; k < h; ++k) {
+          const float sv = upper ? v[k] : v[k + h], kv = upper ? v[k + h] : v[k], sw = upper ? w[k] : w[k + h], kw = upper ? w[k + h] : w[k];
+          v[k] = kv + __shfl_xor_sync(0xffffffffu, sv, h);
+          w[k] = kw + __shfl_xor_sync(0xffffffffu, sw, h);
         }
       }
 #pragma unroll
-      for (int o = G; o < LP; o <<= 1) v[0] += __shfl_xor_sync(0xffffffffu, v[0], o);
-      if (l < G && on && t0 + s0 + l < p.t) {
-        const float2 g = sg[q][s0 + l][ch];
-        out[(size_t)(t0 + s0) * p.out_ld] = (T)((v[0] + g.y) * g.x);
+      for (int o = G; o < LP; o <<= 1) {
+        v[0] += __shfl_xor_sync(0xffffffffu, v[0], o);
+        w[0] += __shfl_xor_sync(0xffffffffu, w[0], o);
+      }
+      y[s0 / G] = make_float2(v[0], w[0]);
+    }
+    if (l < G && on) {
+#pragma unroll
+      for (int s0 = 0; s0 < TT; s0 += G) {
+        const float4 g = sg[q][s0 + l][pair];
+        const float2 v = y[s0 / G];
+        if (t0 + s0 + l < p.t) *reinterpret_cast<Raw *>(out + (size_t)(t0 + s0) * p.out_ld) = Pair<T>::pack((v.x + g.z) * g.x, (v.y + g.w) * g.y);
       }
     }
-    piece_barrier();
+    piece_barrier<ScanCta<LP, NS>::ALL>();
   }
-  if constexpr (!EXACT) {
+  if (on) {
+    float s0[NS], s1[NS];
 #pragma unroll
-    for (int n = 0; n < NS / 2; ++n) unpack2(S2[n], S[2 * n], S[2 * n + 1]);
+    for (int n = 0; n < NS; ++n) unpack2(S2[n], s0[n], s1[n]);
+    st_states<NS>(state, s0);
+    st_states<NS>(state + NP, s1);
   }
-  if (on) st_states<NS>(state, S);
 }
 
 // ----------------------------------------------------------------- a step ----
@@ -428,12 +444,19 @@ selective_step_kernel(Step<T> p) {
 
 template <typename T, int LP, int NS>
 int32_t block_one(ugb_device *dev, const ugb_scan_args &a, const void *dt, const void *xdb, const void *z, size_t z_ld, int b, int t) {
-  constexpr int CC = SCANNERS / LP;
+  using Cta = ScanCta<LP, NS>;
   Block<T> p;
   p.u = (const T *)a.u; p.dt = (const T *)dt; p.xdb = (const T *)xdb; p.z = (const T *)z; p.a = a.a; p.skip = a.skip; p.dt_bias = a.dt_bias;
   p.state = a.state; p.out = (T *)a.out; p.z_ld = z_ld; p.out_ld = a.out_ld; p.scale = a.scale; p.channels = a.channels; p.xr = a.xr;
   p.rp = a.rp; p.t = t;
-  selective_scan_kernel<T, LP, NS><<<dim3((a.channels + CC - 1) / CC, b), SCANNERS + HELPERS, 0, dev->stream>>>(p);
+  const dim3 grid((a.channels + Cta::CC - 1) / Cta::CC, b);
+  constexpr int TT = LP * NS <= 64 ? 16 : 8, CTAS = sizeof(T) == 2 && NS <= 4 ? 3 : 1;
+  bool alone = false;
+  if constexpr (LP * NS <= 16) {
+    alone = (long long)grid.x * grid.y <= dev->sm_count;
+    if (alone) selective_scan_kernel<T, LP, NS, 2 * TT, 1><<<grid, Cta::ALL, 0, dev->stream>>>(p);
+  }
+  if (!alone) selective_scan_kernel<T, LP, NS, TT, CTAS><<<grid, Cta::ALL, 0, dev->stream>>>(p);
   return ugb_after_launch(dev, "selective_scan_kernel");
 }
 template <typename T, int LP, int NS>
@@ -458,7 +481,7 @@ int32_t step_one(ugb_device *dev, const ugb_scan_args &a, const void *w_dt, ugb_
   return ugb_after_launch(dev, "selective_step_kernel");
 }
 
-// f(LP, NS) for the kernel of a shape
+// f(LP, NS) for the step kernel of a shape
 template <typename F> int32_t with_shape(ugb_device *dev, const ugb_scan_shape &s, F f) {
 #define SHAPE(LP, NS) if (s.lanes == LP && s.per_lane == NS) return f(std::integral_constant<int, LP>(), std::integral_constant<int, NS>())
   SHAPE(4, 2); SHAPE(4, 4); SHAPE(4, 6); SHAPE(4, 8); SHAPE(8, 6); SHAPE(8, 8); SHAPE(16, 8); SHAPE(32, 8);
@@ -490,9 +513,12 @@ int32_t ugb_scan_block(ugb_device *dev, const ugb_scan_args &a, const void *dt, 
   if (b == 0 || t == 0) return UGB_OK;
   if (int32_t rc = check(dev, a)) return rc;
   UGB_REQUIRE(dev, z_ld % 8 == 0 && b <= 65535, UGB_ERR_SHAPE, "selective scan: %d sequences, gate rows %zu apart", b, z_ld);
-  return with_shape(dev, a.shape, [&](auto lp, auto ns) {
-    return a.f32 ? block_one<float, lp(), ns()>(dev, a, dt, xdb, z, z_ld, b, t) : block_one<__nv_bfloat16, lp(), ns()>(dev, a, dt, xdb, z, z_ld, b, t);
-  });
+#define BLOCK(NP, LP) \
+  if (a.shape.np == NP) \
+    return a.f32 ? block_one<float, LP, NP / LP>(dev, a, dt, xdb, z, z_ld, b, t) : block_one<__nv_bfloat16, LP, NP / LP>(dev, a, dt, xdb, z, z_ld, b, t)
+  BLOCK(8, 8); BLOCK(16, 8); BLOCK(24, 8); BLOCK(32, 8); BLOCK(48, 8); BLOCK(64, 8); BLOCK(128, 16); BLOCK(256, 32);
+#undef BLOCK
+  return ugb_fail(dev, UGB_ERR_UNSUPPORTED, "selective scan: no kernel for %d states", a.shape.np);
 }
 
 int32_t ugb_scan_step(ugb_device *dev, const ugb_scan_args &a, const void *w_dt, ugb_scan_partials xdb, ugb_scan_partials z, int rows, bool pdl, bool early) {

@@ -5,8 +5,8 @@
 
 #include "ugb_internal.h"
 
-// How the states of a channel are dealt to threads: `lanes` neighbouring lanes with `per_lane` states each.  A channel
-// takes np = lanes * per_lane states in memory; the ones behind the model's count have B = C = 0 and stay zero.
+// A channel takes np states in memory; the ones behind the model's count have B = C = 0 and stay zero.  In a step they are
+// dealt to `lanes` neighbouring lanes with `per_lane` states each.
 struct ugb_scan_shape { int lanes, per_lane, np; };
 // lanes = 0 when there is no kernel for so many states
 ugb_scan_shape ugb_scan_shape_of(int states);
