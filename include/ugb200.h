@@ -716,7 +716,7 @@ UGB_API int32_t ugb_selective_scan(ugb_device *dev, const ugb_slice *x, const ug
                                    const ugb_slice *a_log, const ugb_slice *skip, const ugb_slice *dt_bias, ugb_slice *state,
                                    ugb_slice *out, size_t b, size_t t, size_t channels, size_t states, float scale);
 /* One position of every sequence: low_bc F32 [rows, rank + 2 states], w_dt T [rank, channels], z F32 [rows, channels]; dt =
- * softplus(w_dt^T low + dt_bias); the rest as above with t = 1. */
+ * softplus(w_dt^T low + dt_bias), low rounded to T; the rest as above with t = 1. */
 UGB_API int32_t ugb_selective_step(ugb_device *dev, const ugb_slice *x, const ugb_slice *low_bc, const ugb_slice *w_dt,
                                    const ugb_slice *z, const ugb_slice *a_log, const ugb_slice *skip, const ugb_slice *dt_bias,
                                    ugb_slice *state, ugb_slice *out, size_t rows, size_t channels, size_t rank, size_t states,

@@ -181,6 +181,8 @@ def test_selective_step(dev, bf16, channels, states, rank, rows, steps):
     for i in range(steps):
         x, _, _, z, a_log, skip, bias = scan_inputs(1, rows, channels, states)
         low = synth.normal(25 + i, (rows, rank + 2 * states))
+        if bf16:                                            # the projection's operand is rounded, B and C are not
+            low[:, :rank] = synth.bf16_bits_to_f32(synth.to_bf16_bits(low[:, :rank]))
         xs, xv = B.act(x[:, 0])
         out = B.out(rows * channels)
         dev.selective_step(xs, B.f32(low), w, B.f32(z[:, 0]), B.f32(a_log), B.f32(skip), B.f32(bias), state, out, rows, channels, rank, states, 1.2)

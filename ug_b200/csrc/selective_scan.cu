@@ -11,6 +11,7 @@
 #include <algorithm>
 #include <type_traits>
 
+#include "decode_kernels.cuh"
 #include "hybrid_kernels.cuh"
 
 namespace {
@@ -301,18 +302,23 @@ template <typename T> struct Step {
 };
 constexpr int THREADS = 256;
 constexpr int STEP_J = 4;            // sequences per thread in the projection and the element-wise parts
+// sequences of a CTA at most: a thread holds its states of all of them in registers from before the wait
+template <int NS> struct StepRows { static constexpr int D = NS <= 4 ? 16 : 8; };
 
 // grid (groups of 256 / LP channels, groups of `group` sequences).  Dynamic shared memory: dt, dt x [group][CC]; low | B | C
-// [group][xr]; sums over the states [group][CC]; W_dt [rp][CC].
+// [group][xr]; sums over the states [group][CC]; with w_shared W_dt [rk][CC + 8], and low [16][rk + 8] in T for the tensor cores,
+// rk = rp rounded up to 16.
 template <typename T, int LP, int NS>
 __global__ void __launch_bounds__(THREADS)
 selective_step_kernel(Step<T> p) {
   constexpr bool EXACT = sizeof(T) == 4;
-  constexpr int CC = THREADS / LP, NP = LP * NS, D = NS <= 4 ? 4 : 2;   // D: sequences whose states are in flight per thread
+  constexpr int CC = THREADS / LP, NP = LP * NS, D = StepRows<NS>::D;
   extern __shared__ __align__(16) float dyn[];
   float2 *sd = reinterpret_cast<float2 *>(dyn);                      // [group][CC]
   float *xs = dyn + 2 * p.group * CC, *sy = xs + p.group * p.xr;
-  T *ws = reinterpret_cast<T *>(sy + p.group * CC);
+  constexpr int WLD = CC + 8;                                        // pitches that ldmatrix reads without conflicts
+  const int rk = (p.rp + 15) / 16 * 16, xld = rk + 8;
+  T *ws = reinterpret_cast<T *>(sy + p.group * CC), *xl = ws + rk * WLD;
   const int tid = threadIdx.x, ch = tid / LP, l = tid % LP;
   const int c0 = blockIdx.x * CC, r0 = blockIdx.y * p.group, n_rows = min(p.group, p.rows - r0);
   if (!p.early) { ugb_pdl_wait(); ugb_pdl_trigger(); }
@@ -324,16 +330,13 @@ selective_step_kernel(Step<T> p) {
   if (on) ld_states<NS>(p.a + (size_t)c * NP + l * NS, A);
   float *state = p.state + ((size_t)r0 * p.channels + c) * NP + l * NS;
   const size_t next_row = (size_t)p.channels * NP;
-  float S[D][NS], Sn[D][NS];
-  auto load = [&](float (&v)[D][NS], int r) {
+  float S[D][NS];
 #pragma unroll
-    for (int d = 0; d < D; ++d) {
+  for (int d = 0; d < D; ++d) {
 #pragma unroll
-      for (int n = 0; n < NS; ++n) v[d][n] = 0.f;
-      if (on && r + d < n_rows) ld_states<NS>(state + (size_t)(r + d) * next_row, v[d]);
-    }
-  };
-  load(S, 0);
+    for (int n = 0; n < NS; ++n) S[d][n] = 0.f;
+    if (on && d < n_rows) ld_states<NS>(state + (size_t)d * next_row, S[d]);
+  }
   // channel and sequences of this thread in the projection and the element-wise parts
   const int ec = tid % CC, er = tid / CC;
   const bool col = c0 + ec < p.channels;
@@ -348,90 +351,110 @@ selective_step_kernel(Step<T> p) {
       for (int q = 0; q < p.z.n; ++q) z[j] += p.z.p[q * p.z.stride + (size_t)(r0 + r) * p.z.ld + c0 + ec];
     }
   }
-  if (p.w_shared)
-    for (int i = tid; i < p.rp * (CC / 8); i += THREADS) {           // channels is a multiple of 8
+  if (p.w_shared) {
+    for (int i = tid; i < rk * (CC / 8); i += THREADS) {             // channels is a multiple of 8
       const int k = i / (CC / 8), w = 8 * (i - k * (CC / 8));
       Row8<T> v{};
-      if (c0 + w < p.channels) v = ld8<T>(p.w_dt + (size_t)k * p.channels + c0 + w);
-      st8<T>(ws + k * CC + w, v);
+      if (k < p.rp && c0 + w < p.channels) v = ld8<T>(p.w_dt + (size_t)k * p.channels + c0 + w);
+      st8<T>(ws + k * WLD + w, v);
     }
+    if (!EXACT && rk > p.rp && tid < 16) st8<T>(xl + tid * xld + p.rp, Row8<T>{});
+  }
   if (p.early) { ugb_pdl_wait(); ugb_pdl_trigger(); }
   for (int i = tid; i < p.group * (p.xr / 4); i += THREADS) {
     const int r = i / (p.xr / 4), k = 4 * (i - r * (p.xr / 4));
     float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
     if (r < n_rows)
-      for (int q = 0; q < p.xdb.n; q += 4) {                         // the partials are added in order
-        float4 v[4];
+      for (int q = 0; q < p.xdb.n; q += 8) {                         // the partials are added in order
+        float4 v[8];
 #pragma unroll
-        for (int e = 0; e < 4; ++e)
+        for (int e = 0; e < 8; ++e)
           v[e] = q + e < p.xdb.n ? *reinterpret_cast<const float4 *>(p.xdb.p + (q + e) * p.xdb.stride + (size_t)(r0 + r) * p.xdb.ld + k)
                                  : make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-        for (int e = 0; e < 4; ++e) { s.x += v[e].x; s.y += v[e].y; s.z += v[e].z; s.w += v[e].w; }
+        for (int e = 0; e < 8; ++e) { s.x += v[e].x; s.y += v[e].y; s.z += v[e].z; s.w += v[e].w; }
       }
+    if (!EXACT && p.w_shared && k < p.rp) Act<T>::st4(xl + r * xld + k, s);
     *reinterpret_cast<float4 *>(xs + r * p.xr + k) = s;
   }
   __syncthreads();
-  {
-    float acc[STEP_J];
-#pragma unroll
-    for (int j = 0; j < STEP_J; ++j) acc[j] = bias;
-    auto project = [&](auto weight) {
-      for (int k = 0; k < p.rp; k += 4) {                            // rp is a multiple of 8
-        float w[4];
-#pragma unroll
-        for (int e = 0; e < 4; ++e) w[e] = weight(k + e);
-#pragma unroll
-        for (int j = 0; j < STEP_J; ++j) {
-          if (er + LP * j >= p.group) break;
-          const float4 x = *reinterpret_cast<const float4 *>(xs + (er + LP * j) * p.xr + k);
-          acc[j] = fmaf(w[0], x.x, acc[j]); acc[j] = fmaf(w[1], x.y, acc[j]);
-          acc[j] = fmaf(w[2], x.z, acc[j]); acc[j] = fmaf(w[3], x.w, acc[j]);
-        }
+  // step sizes before bias and softplus: on the tensor cores (a 16-row tile of sequences, a warp per 8 channels), or one by one
+  float pre[STEP_J];
+  bool done = false;
+  if constexpr (!EXACT) {
+    done = p.w_shared != 0;
+    const int warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
+    if (done && warp * 8 < CC) {
+      float acc[4] = {0.f, 0.f, 0.f, 0.f};
+      for (int k = 0; k < rk; k += 16) {
+        uint32_t a[4], b0, b1;
+        asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+                     : "=r"(a[0]), "=r"(a[1]), "=r"(a[2]), "=r"(a[3])
+                     : "r"(ugb_tc::smem_u32(xl + (lane & 15) * xld + k + 8 * (lane >> 4))));
+        asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];"
+                     : "=r"(b0), "=r"(b1) : "r"(ugb_tc::smem_u32(ws + (k + (lane & 15)) * WLD + 8 * warp)));
+        ugb_decode::mma_bf16_16x8x16(acc, a[0], a[1], a[2], a[3], b0, b1);
       }
-    };
-    if (p.w_shared) project([&](int k) { return (float)ws[k * CC + ec]; });
-    else project([&](int k) { return col ? (float)p.w_dt[(size_t)k * p.channels + c0 + ec] : 0.f; });
 #pragma unroll
-    for (int j = 0; j < STEP_J; ++j) {
-      if (er + LP * j >= p.group) break;
-      const float d = softplus_t<EXACT>(acc[j]);
-      sd[(er + LP * j) * CC + ec] = make_float2(d, d * u[j]);
+      for (int h = 0; h < 2; ++h)
+        if (g + 8 * h < p.group) {
+          sd[(g + 8 * h) * CC + 8 * warp + 2 * tq].x = acc[2 * h];
+          sd[(g + 8 * h) * CC + 8 * warp + 2 * tq + 1].x = acc[2 * h + 1];
+        }
+    }
+    if (done) {
+      __syncthreads();
+#pragma unroll
+      for (int j = 0; j < STEP_J; ++j) pre[j] = er + LP * j < p.group ? sd[(er + LP * j) * CC + ec].x : 0.f;
     }
   }
-  __syncthreads();
-  for (int r = 0; r < n_rows; r += D) {
-    load(Sn, r + D);
-    float y[D];
+  if (!done) {
 #pragma unroll
-    for (int d = 0; d < D; ++d) {
-      y[d] = 0.f;
-      if (r + d >= n_rows) continue;                                 // the same for the whole CTA
-      const float2 dt = sd[(r + d) * CC + ch];
-      const float *bc = xs + (r + d) * p.xr + p.rp + l * NS;
+    for (int j = 0; j < STEP_J; ++j) pre[j] = 0.f;
+    for (int k = 0; k < p.rp; ++k) {
+      const float w = p.w_shared ? (float)ws[k * WLD + ec] : (col ? (float)p.w_dt[(size_t)k * p.channels + c0 + ec] : 0.f);
+#pragma unroll
+      for (int j = 0; j < STEP_J; ++j)
+        if (er + LP * j < p.group) pre[j] = fmaf(w, xs[(er + LP * j) * p.xr + k], pre[j]);
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < STEP_J; ++j) {
+    if (er + LP * j >= p.group) break;
+    const float d = softplus_t<EXACT>(pre[j] + bias);
+    sd[(er + LP * j) * CC + ec] = make_float2(d, d * u[j]);
+  }
+  __syncthreads();
+#pragma unroll
+  for (int d0 = 0; d0 < D; d0 += 4) {                                // the sums of four sequences are exchanged together
+    if (d0 >= n_rows) break;                                         // the same for the whole CTA
+    float y[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int d = d0 + e;
+      y[e] = 0.f;
+      if (d >= n_rows) continue;
+      const float2 dt = sd[d * CC + ch];
+      const float *bc = xs + d * p.xr + p.rp + l * NS;
       float B[NS], C[NS];
       ld_states<NS>(bc, B);
       ld_states<NS>(bc + NP, C);
 #pragma unroll
       for (int n = 0; n < NS; ++n) {
         S[d][n] = advance<EXACT>(dt.x * A[n], S[d][n], dt.y * B[n]);
-        y[d] = fmaf(S[d][n], C[n], y[d]);
+        y[e] = fmaf(S[d][n], C[n], y[e]);
       }
-      if (on) st_states<NS>(state + (size_t)(r + d) * next_row, S[d]);
+      if (on) st_states<NS>(state + (size_t)d * next_row, S[d]);
     }
 #pragma unroll
     for (int o = 1; o < LP; o <<= 1)
 #pragma unroll
-      for (int d = 0; d < D; ++d) y[d] += __shfl_xor_sync(0xffffffffu, y[d], o);
+      for (int e = 0; e < 4; ++e) y[e] += __shfl_xor_sync(0xffffffffu, y[e], o);
     if (l == 0) {
 #pragma unroll
-      for (int d = 0; d < D; ++d)
-        if (r + d < n_rows) sy[(r + d) * CC + ch] = y[d];
+      for (int e = 0; e < 4; ++e)
+        if (d0 + e < n_rows) sy[(d0 + e) * CC + ch] = y[e];
     }
-#pragma unroll
-    for (int d = 0; d < D; ++d)
-#pragma unroll
-      for (int n = 0; n < NS; ++n) S[d][n] = Sn[d][n];
   }
   __syncthreads();
 #pragma unroll
@@ -467,9 +490,10 @@ int32_t step_one(ugb_device *dev, const ugb_scan_args &a, const void *w_dt, ugb_
   p.out = (T *)a.out; p.out_ld = a.out_ld; p.scale = a.scale; p.channels = a.channels; p.xr = a.xr; p.rp = a.rp; p.rows = rows;
   p.early = early && pdl ? 1 : 0;
   // sequences per CTA: enough CTAs for two per SM, no more than a thread's share and the shared memory allow
-  const int groups = (a.channels + CC - 1) / CC, most = std::min(STEP_J * LP, 32);
-  const size_t w_bytes = (size_t)a.rp * CC * sizeof(T), limit = 48 * 1024;
-  p.w_shared = w_bytes <= 24 * 1024;
+  const int groups = (a.channels + CC - 1) / CC, most = std::min(STEP_J * LP, StepRows<NS>::D);
+  const int rk = (a.rp + 15) / 16 * 16;
+  const size_t w_bytes = ((size_t)rk * (CC + 8) + 16 * (rk + 8)) * sizeof(T), limit = 48 * 1024;
+  p.w_shared = w_bytes <= 26 * 1024;
   const size_t fixed = p.w_shared ? w_bytes : 0, per_row = (size_t)CC * 12 + (size_t)a.xr * 4;
   p.group = most;
   while (p.group > 4 && (long long)groups * ((rows + p.group - 1) / p.group) < 2 * dev->sm_count) p.group /= 2;
