@@ -77,11 +77,6 @@ int32_t ugb_hybrid_matmul(ugb_hybrid *m, const Mat &x) {
   g.splits = x.splits; g.bn = x.bn; g.b_static = x.groups == nullptr; g.pdl = m->pdl != 0; g.late_trigger = true;
   g.groups = x.groups; g.n_groups = x.n_groups; g.tile_m = x.tile;
   g.smem_kib = x.m <= 64 || (x.groups && x.tile == 64) ? 144 : 0;
-  if (g.bn == 0 && !x.groups && x.batch == 1 && x.m > 128) {
-    // narrow products of a block: tiles small enough to occupy the SMs
-    const size_t sms = dev->sm_count, tiles_m = (x.m + 127) / 128;
-    if (tiles_m * ((x.n + 255) / 256) < sms * 3 / 4) g.bn = tiles_m * ((x.n + 127) / 128) >= sms * 3 / 4 ? 128 : 64;
-  }
   if (!x.f32_out && !x.groups && x.batch == 1 && x.nk && x.m <= 64 && x.k >= 256) {
     // a T result cannot be split into partials: the two k halves of a tile on a pair of CTAs, with the narrowest tile that fits the SMs
     for (int bn : {64, 96, 128, 160})
