@@ -489,14 +489,15 @@ int32_t step_one(ugb_device *dev, const ugb_scan_args &a, const void *w_dt, ugb_
   p.u = (const T *)a.u; p.w_dt = (const T *)w_dt; p.xdb = xdb; p.z = z; p.a = a.a; p.skip = a.skip; p.dt_bias = a.dt_bias; p.state = a.state;
   p.out = (T *)a.out; p.out_ld = a.out_ld; p.scale = a.scale; p.channels = a.channels; p.xr = a.xr; p.rp = a.rp; p.rows = rows;
   p.early = early && pdl ? 1 : 0;
-  // sequences per CTA: enough CTAs for two per SM, no more than a thread's share and the shared memory allow
+  // sequences per CTA: two CTAs are resident per SM, so one wave of at least 1.5 per SM; no more than a thread's share and the
+  // shared memory allow
   const int groups = (a.channels + CC - 1) / CC, most = std::min(STEP_J * LP, StepRows<NS>::D);
   const int rk = (a.rp + 15) / 16 * 16;
   const size_t w_bytes = ((size_t)rk * (CC + 8) + 16 * (rk + 8)) * sizeof(T), limit = 48 * 1024;
   p.w_shared = w_bytes <= 26 * 1024;
   const size_t fixed = p.w_shared ? w_bytes : 0, per_row = (size_t)CC * 12 + (size_t)a.xr * 4;
   p.group = most;
-  while (p.group > 4 && (long long)groups * ((rows + p.group - 1) / p.group) < 2 * dev->sm_count) p.group /= 2;
+  while (p.group > 4 && 2ll * groups * ((rows + p.group - 1) / p.group) < 3 * dev->sm_count) p.group /= 2;
   while (p.group > 1 && fixed + p.group * per_row > limit) p.group /= 2;
   UGB_REQUIRE(dev, fixed + p.group * per_row <= limit, UGB_ERR_UNSUPPORTED, "selective scan: %d columns of step size, B and C", a.xr);
   const cudaError_t e = ugb_launch(selective_step_kernel<T, LP, NS>, dim3(groups, (rows + p.group - 1) / p.group), dim3(THREADS),
