@@ -1204,16 +1204,27 @@ class KabidraWorkload:
 
 class ZidevikWorkload(KabidraWorkload):
     """The Zidevik decoder at the layer sizes of the 1.1B Llama benchmark model, beside Kabidra and Llama at those sizes: the
-    decode steps, prompts and single kernels of KabidraWorkload for all three in one process."""
+    decode steps, prompts and single kernels of KabidraWorkload for all three in one process; then eight layers of width 4096
+    beside Kabidra's."""
     metric = "tokens/s, Zidevik decode (64 sequences, 2048 cached positions)"
     name = ("Zidevik, width 2048, 22 layers of which 6 run twice (attention with 32 heads of 64 on 4 beside a scan of 4096 channels "
             "with 16 states; feed-forwards alternately dense with 5632 columns and 2 of 16 experts of 1408 beside a shared one of "
             "2816; token input of 256), vocab 32000, bf16; beside Kabidra and the Llama-1.1B shape")
     SFU_PER_CLOCK = 16           # special functions per clock and SM
 
-    def __init__(self, rank=0):
+    def __init__(self, rank=0, wide=False):
+        from ug_b200.kabidra_config import Config as KabidraConfig
+        from ug_b200.kabidra_config import Layer
         from ug_b200.zidevik_config import Config
-        self.cfg = Config.like_llama_1b()
+        self.sms = 148
+        self.other = KabidraWorkload()
+        if wide:
+            self.cfg = Config.like_llama(4096, 8, 128, 8, 11264)
+            att = dict(heads=32, dim=128, vdim=128, q_rank=1536, kv_rank=512, scale=128 ** -0.5)
+            self.other.cfg = KabidraConfig(vocab=32000, width=4096, eps=1e-5, taps=4, layers=[
+                Layer("latent_attention", dict(att), 11264) if i % 4 == 3 else Layer("mingru", {"width": 4096}, 11264) for i in range(8)])
+        else:
+            self.cfg = Config.like_llama()
 
     def setup(self, dev):
         import re
@@ -1229,9 +1240,7 @@ class ZidevikWorkload(KabidraWorkload):
         with ThreadPoolExecutor(max_workers=min(16, os.cpu_count() or 1)) as ex:
             made = dict(zip(first, ex.map(lambda n: synth.zidevik_tensor(500, n, shapes[n]), first.values())))
         self.weights = {n: made[kind(n)] for n in shapes}
-        self.other = KabidraWorkload()
         self.other.setup(dev)
-        self.sms = 148
 
     def splits(self, n, k, decode, batch):
         """k splits of a step's product, as the engine chooses them."""
@@ -1311,19 +1320,16 @@ class ZidevikWorkload(KabidraWorkload):
             out["scan"]["frac_of_special_functions"] = round(1e3 * n / (self.SFU_PER_CLOCK * self.sms * 1.965e9) / out["scan"]["ms"], 3)
         return out
 
-    def record(self, dev, warmup, steps, peaks):
-        from ug_b200 import kabidra, llama, synth, zidevik
-        from ug_b200.llama_config import Config as LlamaConfig
-        lc = LlamaConfig.llama_1b()
-        lw = _weights(lc)
-        made = {"zidevik": (self, lambda b, t: zidevik.Model.new(self.cfg, self.weights, dev, b, t)),
-                "kabidra": (self.other, lambda b, t: kabidra.Model.new(self.other.cfg, self.other.weights, dev, b, t)),
-                "llama": (None, lambda b, t: llama.Model.new(lc, lw, dev, b, t))}
-        sampler = ClockSampler(0)
-        sampler.start()
-        rec = {"workload": self.name, "metric": self.metric, "unit": self.unit, "dtype": self.dtype, "steps": steps,
-               "data": "synthetic (random weights and tokens)", "peak_source": peaks["source"], "decode": {}, "prefill": {}}
-        for batch, depth in self.DECODE:
+    def pair(self, dev):
+        """Name -> (workload that knows the model's kernels, constructor of (sequences, positions))."""
+        from ug_b200 import kabidra, zidevik
+        return {"zidevik": (self, lambda b, t: zidevik.Model.new(self.cfg, self.weights, dev, b, t)),
+                "kabidra": (self.other, lambda b, t: kabidra.Model.new(self.other.cfg, self.other.weights, dev, b, t))}
+
+    def cases(self, dev, made, warmup, steps, peaks, decode, prefill):
+        from ug_b200 import synth
+        rec = {"decode": {}, "prefill": {}}
+        for batch, depth in decode:
             prompts, r = synth.tokens(8, (batch, depth), self.cfg.vocab), {}
             for key, (wl, make) in made.items():
                 m = make(batch, depth + warmup + steps + 64)
@@ -1336,11 +1342,12 @@ class ZidevikWorkload(KabidraWorkload):
                     r[key]["kernels"] = wl.kernels(m, batch, batch, 1, at, peaks)
                     r[key]["kernels"]["head"] = {"ms": round(m.time_kernel("head"), 4), "launches": 1}
                 else:
-                    kv = 2 * lc.num_hidden_layers * 2 * lc.num_key_value_heads * lc.head_dim() * at * batch
+                    c = m.cfg
+                    kv = 2 * c.num_hidden_layers * 2 * c.num_key_value_heads * c.head_dim() * at * batch
                     r[key]["attention_frac"] = round(kv / peaks["hbm"] / 1e6 / m.time_kernel("decode_attention", 20), 3)
                 m.close()
             rec["decode"]["%d x %d" % (batch, depth)] = r
-        for batch, t in self.PREFILL:
+        for batch, t in prefill:
             prompts, r = dev.slice_from_values(synth.tokens(9, (batch, t), self.cfg.vocab).reshape(-1)), {}
             for key, (wl, make) in made.items():
                 m = make(batch, t + (32 if wl else 0))
@@ -1358,6 +1365,22 @@ class ZidevikWorkload(KabidraWorkload):
                     r[key]["kernels"] = wl.kernels(m, batch * t, batch, t, 0, peaks)
                 m.close()
             rec["prefill"]["%d x %d" % (batch, t)] = r
+        return rec
+
+    def record(self, dev, warmup, steps, peaks):
+        from ug_b200 import llama
+        from ug_b200.llama_config import Config as LlamaConfig
+        lc = LlamaConfig.llama_1b()
+        lw = _weights(lc)
+        sampler = ClockSampler(0)
+        sampler.start()
+        made = {**self.pair(dev), "llama": (None, lambda b, t: llama.Model.new(lc, lw, dev, b, t))}
+        rec = {"workload": self.name, "metric": self.metric, "unit": self.unit, "dtype": self.dtype, "steps": steps,
+               "data": "synthetic (random weights and tokens)", "peak_source": peaks["source"],
+               **self.cases(dev, made, warmup, steps, peaks, self.DECODE, self.PREFILL)}
+        wide = ZidevikWorkload(wide=True)
+        wide.setup(dev)
+        rec["width 4096, 8 layers"] = wide.cases(dev, wide.pair(dev), warmup, steps, peaks, self.DECODE[:1], self.PREFILL)
         rec["clocks"] = sampler.stop()
         rec["value"] = rec["decode"]["64 x 2048"]["zidevik"]["tokens_per_s"]
         return rec

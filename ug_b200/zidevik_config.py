@@ -110,14 +110,15 @@ class Config:
         return out
 
     @staticmethod
-    def like_llama_1b(layers=22, vocab=32000):
-        """Layers of the size of the 1.1B Llama benchmark model: width 2048, 32 heads of 64 on 4, a scan of 4096 channels with
-        16 states; every other feed-forward dense with 5632 columns, the others 16 experts of 1408 of which a token uses 2
-        beside a shared one of 2816.  Layers 8 .. 13 run twice."""
-        left = Attention(heads=32, kv_heads=4, dim=64, vdim=64, rot_dims=64, rot_base=10000.0, scale=0.125)
-        right = Scan(inner=4096, state=16, conv=4, dt_rank=128)
-        return Config(vocab=vocab, width=2048, eps=1e-5, loop=Loop(8, 14, 2), side_dim=256, logit_softcap=30.0,
-                      layers=[Layer(left, right, 1.0, 1.0, 5632 if i % 2 == 0 else Experts(16, 2, 1408, 2816)) for i in range(layers)])
+    def like_llama(width=2048, layers=22, head=64, kv_heads=4, ff=5632, vocab=32000):
+        """Layers of the size of a Llama benchmark model (the 1.1B one by default): as many heads as the width holds, a scan of
+        twice the width with 16 states; every other feed-forward dense, the others 16 experts of a quarter of its columns, of
+        which a token uses 2, beside a shared one of half.  A quarter of the layers, from the third eighth on, runs twice."""
+        left = Attention(heads=width // head, kv_heads=kv_heads, dim=head, vdim=head, rot_dims=head, rot_base=10000.0, scale=head ** -0.5)
+        right = Scan(inner=2 * width, state=16, conv=4, dt_rank=width // 16)
+        lo = 3 * layers // 8
+        return Config(vocab=vocab, width=width, eps=1e-5, loop=Loop(lo, lo + max(1, (layers + 2) // 4), 2), side_dim=256, logit_softcap=30.0,
+                      layers=[Layer(left, right, 1.0, 1.0, ff if i % 2 == 0 else Experts(16, 2, ff // 4, ff // 2)) for i in range(layers)])
 
 
 def _read_mlp(i, mlp):
