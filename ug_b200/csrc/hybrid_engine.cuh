@@ -59,11 +59,11 @@ struct ugb_hybrid_work {
   void *xs = nullptr, *xx = nullptr;                       // the stream in T; stream | embedding output for a loop's input
   void *xdb = nullptr, *dt = nullptr;                      // step-size latent | B | C; step sizes before their bias
   float *gu = nullptr;                                     // f32 model: (gate, up) products
-  float *side = nullptr;
+  float *side = nullptr, *part = nullptr;                  // part: narrow products of a block, before they are summed
   void *side_h = nullptr;
   // mixture of experts: token rows grouped by expert in tiles of `tile` rows
   int tile = 0, tiles = 0;
-  float *router = nullptr, *xout = nullptr;
+  float *xout = nullptr;
   void *xin = nullptr, *xmid = nullptr;
   int *count = nullptr, *map = nullptr, *slot = nullptr;   // rows per expert, expert of a tile, row of (token, choice)
   float4 *choice = nullptr;                                // {expert, place, weight}

@@ -40,6 +40,18 @@ static size_t up8(size_t n) { return ugb_up8(n); }
 
 namespace {
 
+// Narrow products of a block have few tiles and a long k loop that one CTA walks in order: k splits that fill the SMs with
+// 128 x 256 tiles, four k blocks or more each.  Their f32 partials take at most narrow_rows() rows.
+int narrow_splits(const ugb_hybrid *m, int rows, size_t n, size_t k) {
+  if (m->f32) return 1;
+  const int tiles = (rows + 127) / 128 * (int)((n + 255) / 256), kb = (int)((k + 63) / 64);
+  const int s = std::min({UGB_HYBRID_MAX_SPLITS, m->dev->sm_count / tiles, kb / 4});
+  return s > 1 ? ugb_tc_gemm_effective_splits(k, s) : 1;
+}
+size_t narrow_rows(const ugb_hybrid *m, size_t rows) {
+  return m->f32 ? rows : std::max(rows, std::min(rows * UGB_HYBRID_MAX_SPLITS, (size_t)m->dev->sm_count * 128));
+}
+
 // tiles of `tile` rows that hold `rows` rows grouped into `groups`
 int group_tiles(size_t rows, int groups, int tile) { return (int)(rows / tile) + groups; }
 
@@ -173,14 +185,22 @@ int32_t run(ugb_hybrid *m, ugb_hybrid_work &w, const int *tok, int t_block, int 
     // ---- scan
     const size_t n_cat = L.n_cat(), cat_s = (size_t)d.heads * L.vp, cat_f = cat_s + L.ci;
     const int xr = L.rp + 2 * L.np;
-    const Tiling x_t = decode ? ugb_hybrid_tile(m, xr, L.ci) : Tiling{0, 1};
+    const Tiling x_t = decode ? ugb_hybrid_tile(m, xr, L.ci) : Tiling{0, narrow_splits(m, rows, xr, L.ci)};
     if (m->on(UGB_HYBRID_K_SCAN_IN)) {
-      Mat g{w.xdb, w.hc, L.w_x, (size_t)rows, (size_t)xr, (size_t)L.ci};
-      g.splits = x_t.splits; g.bn = x_t.bn; g.f32_out = decode || m->f32;
+      const bool sum = !decode && x_t.splits > 1;            // a block's split product is summed and rounded to T
+      Mat g{sum ? (void *)w.part : w.xdb, w.hc, L.w_x, (size_t)rows, (size_t)xr, (size_t)L.ci};
+      g.splits = x_t.splits; g.bn = sum ? 256 : x_t.bn; g.f32_out = decode || m->f32 || sum;
       if ((rc = ugb_hybrid_matmul(m, g))) return rc;
+      if (sum) {
+        const size_t n4 = (size_t)rows * xr / 4;
+        e = ugb_launch(sum_partials_kernel<T>, dim3((unsigned)((n4 + 255) / 256)), dim3(256), 0, dev->stream, pdl, w.part, x_t.splits, (size_t)rows * xr, n4, (T *)w.xdb);
+        if (e != cudaSuccess) return ugb_fail(dev, UGB_ERR_CUDA, "launch of sum_partials_kernel failed: %s", cudaGetErrorString(e));
+        if ((rc = ugb_after_launch(dev, "sum_partials_kernel"))) return rc;
+      }
       if (!decode) {
         Mat h{w.dt, w.xdb, L.w_dt, (size_t)rows, (size_t)L.ci, (size_t)L.rp};
         h.a_ld = xr; h.nk = false; h.f32_out = m->f32;
+        h.bn = 128;                                          // few k blocks: the epilogues are the work, and small ones overlap better
         if ((rc = ugb_hybrid_matmul(m, h))) return rc;
       }
     }
@@ -225,10 +245,11 @@ int32_t run(ugb_hybrid *m, ugb_hybrid_work &w, const int *tok, int t_block, int 
       if (m->on(UGB_HYBRID_K_ROUTE)) {
         if (!decode) {
           const size_t es = m->es();
-          Mat g{w.router, w.h, (const char *)L.w_in + n_in * wl * es, (size_t)rows, (size_t)L.ep, (size_t)wl};
+          Mat g{w.part, w.h, (const char *)L.w_in + n_in * wl * es, (size_t)rows, (size_t)L.ep, (size_t)wl};
+          g.splits = narrow_splits(m, rows, L.ep, wl); g.bn = g.splits > 1 ? 256 : 0;
           if ((rc = ugb_hybrid_matmul(m, g))) return rc;
           if (!whole) UGB_CUDA(dev, cudaMemsetAsync(w.count, 0, d.experts * sizeof(int), dev->stream));
-          route_kernel<<<(rows + ROUTE_ROWS - 1) / ROUTE_ROWS, 256, 0, dev->stream>>>(w.router, L.ep, rows, d.experts, d.top, w.choice, w.count);
+          route_kernel<<<(rows + ROUTE_ROWS - 1) / ROUTE_ROWS, 256, 0, dev->stream>>>(w.part, g.splits, L.ep, rows, d.experts, d.top, w.choice, w.count);
           if ((rc = ugb_after_launch(dev, "route_kernel"))) return rc;
         }
         e = ugb_launch(expert_rows_kernel<T>, dim3(rows), dim3(256), 0, dev->stream, pdl, (const T *)w.h, w.choice, w.count, d.experts, d.top, tile, tiles,
@@ -260,10 +281,10 @@ int32_t run(ugb_hybrid *m, ugb_hybrid_work &w, const int *tok, int t_block, int 
 
     // ---- input of the token
     if (side) {
-      const Tiling g_t = decode ? ugb_hybrid_tile(m, m->sl, wl) : Tiling{0, 1}, p_t = decode ? ugb_hybrid_tile(m, wl, m->sl) : Tiling{0, 1};
+      const Tiling g_t = decode ? ugb_hybrid_tile(m, m->sl, wl) : Tiling{0, narrow_splits(m, rows, m->sl, wl)}, p_t = decode ? ugb_hybrid_tile(m, wl, m->sl) : Tiling{0, 1};
       if (m->on(UGB_HYBRID_K_SIDE)) {
         Mat g{w.side, w.xs, L.side_gate, (size_t)rows, (size_t)m->sl, (size_t)wl};
-        g.splits = g_t.splits; g.bn = g_t.bn;
+        g.splits = g_t.splits; g.bn = !decode && g_t.splits > 1 ? 256 : g_t.bn;
         if ((rc = ugb_hybrid_matmul(m, g))) return rc;
       }
       if (m->on(UGB_HYBRID_K_SIDE_GATE)) {
@@ -422,8 +443,8 @@ int32_t ugb_parallel_work(ugb_hybrid *m, ugb_hybrid_work &w, int rows, bool deco
       (rc = ugb_hybrid_alloc(m, &w.cat, R * cat * es, false)) || (rc = ugb_hybrid_alloc(m, &w.xs, R * wl * es, false)) ||
       (rc = ugb_hybrid_alloc(m, &w.xx, m->cfg.loop_times ? R * 2 * wl * es : 0, false)) ||
       (rc = ugb_hybrid_alloc(m, &w.xdb, parts * R * xr * (decode ? 4 : es), false)) || (rc = ugb_hybrid_alloc(m, &w.dt, decode ? 0 : R * ci * es, false)) ||
-      (rc = dmalloc(m, &w.gu, gu)) || (rc = dmalloc(m, &w.side, parts * R * m->sl)) || (rc = ugb_hybrid_alloc(m, &w.side_h, R * m->sl * es, false)) ||
-      (rc = dmalloc(m, &w.router, decode ? 0 : R * ep)) || (rc = dmalloc(m, &w.choice, R * top, true)) || (rc = dmalloc(m, &w.slot, R * top, true)) ||
+      (rc = dmalloc(m, &w.gu, gu)) || (rc = dmalloc(m, &w.side, (decode ? parts * R : narrow_rows(m, R)) * m->sl)) || (rc = ugb_hybrid_alloc(m, &w.side_h, R * m->sl * es, false)) ||
+      (rc = dmalloc(m, &w.part, decode ? 0 : narrow_rows(m, R) * std::max(xr, ep))) || (rc = dmalloc(m, &w.choice, R * top, true)) || (rc = dmalloc(m, &w.slot, R * top, true)) ||
       (rc = dmalloc(m, &w.count, E, true)) || (rc = dmalloc(m, &w.map, w.tiles)) || (rc = ugb_hybrid_alloc(m, &w.xin, xrows * wl * es, true)) ||
       (rc = ugb_hybrid_alloc(m, &w.xmid, xrows * ef * es, true)) || (rc = dmalloc(m, &w.xout, xrows * wl)))
     return rc;

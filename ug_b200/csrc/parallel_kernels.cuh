@@ -218,12 +218,12 @@ mixer_inputs_kernel(MixerIn<TI, T> a, int rows) {
 }
 
 // ---------------------------------------------------------------- experts ----
-// Router logits [rows][ld] of a block -> choice [rows][top] = {expert, place among the expert's rows, sigmoid score}.  32
+// Router logits [n_part][rows][ld] of a block, to be summed -> choice [rows][top] = {expert, place among the expert's rows, sigmoid score}.  32
 // rows per CTA: places are handed out per CTA in shared memory, one global counter update per expert and CTA.  Which place
 // a row gets depends on the order of the CTAs; nothing that is computed does.
 constexpr int ROUTE_ROWS = 32;
 static __global__ void __launch_bounds__(256)
-route_kernel(const float *__restrict__ logits, int ld, int rows, int experts, int top, float4 *__restrict__ choice, int *__restrict__ count) {
+route_kernel(const float *__restrict__ logits, int n_part, int ld, int rows, int experts, int top, float4 *__restrict__ choice, int *__restrict__ count) {
   __shared__ int n[32 * ROUTER_PER_LANE], base[32 * ROUTER_PER_LANE];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r0 = blockIdx.x * ROUTE_ROWS;
   n[threadIdx.x] = 0;
@@ -231,7 +231,12 @@ route_kernel(const float *__restrict__ logits, int ld, int rows, int experts, in
   for (int r = r0 + warp; r < min(rows, r0 + ROUTE_ROWS); r += 8) {
     float z[ROUTER_PER_LANE];
 #pragma unroll
-    for (int j = 0; j < ROUTER_PER_LANE; ++j) z[j] = lane + 32 * j < experts ? logits[(size_t)r * ld + lane + 32 * j] : -INFINITY;
+    for (int j = 0; j < ROUTER_PER_LANE; ++j) {
+      const int e = lane + 32 * j;
+      z[j] = e < experts ? 0.f : -INFINITY;
+      if (e < experts)
+        for (int p = 0; p < n_part; ++p) z[j] += logits[((size_t)p * rows + r) * ld + e];
+    }
     top_experts(z, experts, top, [&](int k, int e, float zk) {
       if (lane == 0) choice[(size_t)r * top + k] = make_float4(__int_as_float(e), __int_as_float(atomicAdd(n + e, 1)), sigmoid_f(zk), 0.f);
     });
@@ -304,6 +309,24 @@ static __global__ void silu_mul_kernel(const float *__restrict__ gu, float *__re
     const float2 v = *reinterpret_cast<const float2 *>(gu + r * in_ld + 2 * c);
     out[r * out_ld + c] = silu_f(v.x) * v.y;
   }
+}
+
+// out = sum of n_part f32 partials, rounded to T; n4 groups of four values
+template <typename T>
+__global__ void __launch_bounds__(256)
+sum_partials_kernel(const float *__restrict__ part, int n_part, size_t part_stride, size_t n4, T *__restrict__ out) {
+  ugb_pdl_wait();
+  ugb_pdl_trigger();
+  const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= n4) return;
+  float4 v[8], s = make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int p = 0; p < n_part; p += 8) {                    // the partials are added in order
+#pragma unroll
+    for (int k = 0; k < 8; ++k) v[k] = p + k < n_part ? __ldcs(reinterpret_cast<const float4 *>(part + (size_t)(p + k) * part_stride) + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int k = 0; k < 8; ++k) { s.x += v[k].x; s.y += v[k].y; s.z += v[k].z; s.w += v[k].w; }
+  }
+  Act<T>::st4(out + 4 * i, s);
 }
 
 // ------------------------------------------------------------- token input ---

@@ -493,15 +493,21 @@ int32_t step_one(ugb_device *dev, const ugb_scan_args &a, const void *w_dt, ugb_
   // shared memory allow
   const int groups = (a.channels + CC - 1) / CC, most = std::min(STEP_J * LP, StepRows<NS>::D);
   const int rk = (a.rp + 15) / 16 * 16;
-  const size_t w_bytes = ((size_t)rk * (CC + 8) + 16 * (rk + 8)) * sizeof(T), limit = 48 * 1024;
-  p.w_shared = w_bytes <= 26 * 1024;
+  const size_t w_bytes = ((size_t)rk * (CC + 8) + 16 * (rk + 8)) * sizeof(T), limit = 100 * 1024;   // two CTAs per SM
+  p.w_shared = w_bytes <= 64 * 1024;
   const size_t fixed = p.w_shared ? w_bytes : 0, per_row = (size_t)CC * 12 + (size_t)a.xr * 4;
   p.group = most;
   while (p.group > 4 && 2ll * groups * ((rows + p.group - 1) / p.group) < 3 * dev->sm_count) p.group /= 2;
   while (p.group > 1 && fixed + p.group * per_row > limit) p.group /= 2;
   UGB_REQUIRE(dev, fixed + p.group * per_row <= limit, UGB_ERR_UNSUPPORTED, "selective scan: %d columns of step size, B and C", a.xr);
-  const cudaError_t e = ugb_launch(selective_step_kernel<T, LP, NS>, dim3(groups, (rows + p.group - 1) / p.group), dim3(THREADS),
-                                   fixed + p.group * per_row, dev->stream, pdl, p);
+  static size_t allowed[64] = {};                            // by device; a size is met by an eager step before any capture
+  size_t &most_smem = allowed[dev->ordinal & 63];
+  const size_t smem = fixed + p.group * per_row;
+  if (smem > std::max<size_t>(most_smem, 48 * 1024)) {
+    UGB_CUDA(dev, cudaFuncSetAttribute(selective_step_kernel<T, LP, NS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    most_smem = smem;
+  }
+  const cudaError_t e = ugb_launch(selective_step_kernel<T, LP, NS>, dim3(groups, (rows + p.group - 1) / p.group), dim3(THREADS), smem, dev->stream, pdl, p);
   if (e != cudaSuccess) return ugb_fail(dev, UGB_ERR_CUDA, "launch of selective_step_kernel failed: %s", cudaGetErrorString(e));
   return ugb_after_launch(dev, "selective_step_kernel");
 }
