@@ -151,9 +151,9 @@ def scan_want(xv, dtv, bcv, zv, a_log, skip, bias, s0, scale):
 @pytest.mark.parametrize("bf16", [False, True])
 @pytest.mark.parametrize("channels,states,batch,cuts", [
     (8, 8, 2, (2, 3, 7)), (40, 16, 1, (31, 32, 33, 2)), (200, 24, 2, (64, 5)), (72, 32, 1, (9, 40)), (16, 48, 1, (70,)), (32, 64, 2, (33, 2)),
-    (24, 128, 1, (2, 17, 8)), (8, 256, 1, (40,)), (264, 16, 1, (700, 2))])
+    (24, 128, 1, (2, 17, 8)), (8, 256, 1, (40,)), (264, 16, 1, (700, 2)), (512, 16, 10, (37, 3)), (264, 8, 20, (19, 2))])
 def test_selective_scan(dev, bf16, channels, states, batch, cuts):
-    """Blocks that continue one another from a given state, for every dealing of states to lanes."""
+    """Blocks that continue one another from a given state, for every dealing of states to lanes, with few CTAs and with many."""
     B, t = Buf(dev, bf16), sum(cuts)
     x, dt, bc, z, a_log, skip, bias = scan_inputs(t, batch, channels, states)
     s0 = synth.normal(22, (batch, channels, states))
@@ -172,7 +172,7 @@ def test_selective_scan(dev, bf16, channels, states, batch, cuts):
 
 @pytest.mark.parametrize("bf16", [False, True])
 @pytest.mark.parametrize("channels,states,rank,rows,steps", [
-    (8, 8, 8, 1, 5), (40, 16, 24, 3, 4), (200, 24, 8, 4, 3), (72, 32, 136, 5, 3), (16, 48, 16, 2, 3), (32, 64, 200, 9, 2), (24, 128, 40, 6, 3), (8, 256, 8, 1, 3)])
+    (8, 8, 8, 1, 5), (40, 16, 24, 3, 4), (200, 24, 8, 4, 3), (72, 32, 136, 5, 3), (16, 48, 16, 2, 3), (32, 64, 200, 9, 2), (24, 128, 40, 6, 3), (8, 256, 8, 1, 3), (40, 16, 520, 3, 2), (72, 16, 136, 40, 2)])
 def test_selective_step(dev, bf16, channels, states, rank, rows, steps):
     B = Buf(dev, bf16)
     w, wv = B.act(synth.normal(23, (rank, channels), rank ** -0.5))
